@@ -889,6 +889,70 @@ int nerva_b200_session_attach_peers(NervaCudaHfDecodeSequenceSession *session,
  * the bounded-wait path on one GPU without faulting or hanging anything. */
 int nerva_b200_session_attach_loopback(NervaCudaHfDecodeSequenceSession *session);
 
+/* ---- parallel-block decoders (no counterpart in the reference) ----
+ * A decoder whose layers are described one by one: one norm in front of both sublayers,
+ * x += ls1 * attention(norm(x)) + ls2 * mlp(norm(x)), sliding-window grouped-query attention with
+ * a rotation of part of each head (optionally YaRN-scaled) and a weightless RMS norm of q and k
+ * after it, a range of layers that runs several times with the same weights (each pass with its
+ * own cache), a scaled embedding and soft-capped logits.  Every size is per layer.
+ *
+ * The session is an ordinary one: start / advance / run / append / fork / batch_advance_one /
+ * read_logits work on it as on any other.  The create request carries the planned weight
+ * descriptors (required) and the scalars that are common to the model (hidden, vocab_size,
+ * layer_count, max_context_tokens, rms_eps; heads, kv_heads, head_dim and intermediate hold the
+ * largest of any layer; every chain layer is FULL / DENSE).  Descriptor order: embeddings,
+ * loop vectors (when loop_times != 0), per layer {norm, w_q, w_k, w_v, w_o, w_gate, w_up, w_down
+ * (the last three when intermediate != 0), attention scale, mlp scale (when intermediate != 0)},
+ * final norm, head. */
+typedef struct NervaB200ParallelLayer {
+  uint32_t heads;
+  uint32_t kv_heads;
+  uint32_t qk_dim;           /* per-head query / key size, at most 256 */
+  uint32_t v_dim;            /* per-head value size, at most 256 */
+  uint32_t intermediate;     /* 0: the layer has no feed-forward */
+  uint32_t window;           /* keys a query sees, itself included; 0: all before it */
+  uint32_t rotary_dims;      /* leading dimensions of a head that are rotated (even; 0: none) */
+  uint32_t qk_norm;          /* 1: q and k divided by their root mean square after the rotation */
+  double rotary_base;
+  double yarn_factor;        /* 0: no scaling of the frequencies */
+  double yarn_original;
+  double yarn_fast;
+  double yarn_slow;
+  float score_scale;
+  uint32_t layer_scale;      /* 1: per-channel scales ls1 / ls2 follow the layer's weights */
+} NervaB200ParallelLayer;
+typedef struct NervaB200ParallelModel {
+  uint32_t layer_count;
+  uint32_t compute;          /* NERVA_DTYPE_BF16, or NERVA_DTYPE_F32: activations, cache and products in fp32 */
+  uint32_t loop_start;       /* layers [loop_start, loop_stop) run loop_times times; loop_times 0: no loop */
+  uint32_t loop_stop;
+  uint32_t loop_times;
+  float embedding_scale;
+  float logit_softcap;       /* 0: none */
+  uint32_t reserved;
+  const NervaB200ParallelLayer *layers;
+} NervaB200ParallelModel;
+int nerva_b200_session_create_parallel(const NervaCudaHfDecodeSequenceSessionCreateRequest *request,
+                                       const NervaB200ParallelModel *model,
+                                       NervaCudaHfDecodeSequenceSessionCreateResult *out,
+                                       NervaCudaHfDecodeSequenceSession **session_out);
+
+/* Runs `count` given tokens after the positions the session has already run (a fresh or reset
+ * session begins at position 0) and samples after the last of them, so that advance can follow.
+ * Several tokens go through the block step where the model has one, a single token through the
+ * decode step.  want[i] (i < want_count): places among these tokens whose logits are copied to
+ * logits[i * vocab_size] (host memory).  `reset` != 0 first drops what the session holds.  Works
+ * for every single-GPU session. */
+int nerva_b200_session_append(NervaCudaHfDecodeSequenceSession *session, const uint32_t *tokens,
+                              uint32_t count, uint32_t reset, const uint32_t *want,
+                              uint32_t want_count, float *logits);
+
+/* The residual stream after each layer run of the next appended blocks (a diagnostic): `stream`
+ * is host memory of [layer runs][capacity_rows][hidden] floats, filled for the rows of the append
+ * calls that follow until it is set to NULL.  Parallel-block sessions only. */
+int nerva_b200_session_capture_stream(NervaCudaHfDecodeSequenceSession *session, float *stream,
+                                      uint32_t capacity_rows);
+
 /* Tuning aid of the per-operator engine: nanosecond stamps (%globaltimer) of the
  * last step, 8 per launch, launches ordered [layer][QKV, attention, O, gate/up,
  * down] then lm_head.  Slots 0..3: first block at kernel entry, after the wait

@@ -33,8 +33,9 @@ __device__ __forceinline__ uint32_t row_token(const BlockTokenRow &r) {
   return r.position < *r.prompt_count ? r.prompt[r.position] : r.slots[r.position - 1u].token;
 }
 
-// h[row][:] = embedding row of the row's token, as f32.
-__global__ void block_embed_kernel(const BlockTokenRow *rows, const uint16_t *embeddings, uint32_t hidden, float *h) {
+// h[row][:] = embedding row of the row's token, as f32, times scale; rows of `padded` values, zero beyond hidden.
+__global__ void block_embed_kernel(const BlockTokenRow *rows, const uint16_t *embeddings, uint32_t hidden, float *h,
+                                   float scale, uint32_t padded) {
   pdl_trigger();
   const BlockTokenRow r = rows[blockIdx.x];
   uint32_t token = row_token(r);
@@ -43,22 +44,25 @@ __global__ void block_embed_kernel(const BlockTokenRow *rows, const uint16_t *em
     token = 0;
   }
   const uint16_t *src = embeddings + static_cast<uint64_t>(token) * hidden;
-  float *dst = h + static_cast<uint64_t>(blockIdx.x) * hidden;
-  for (uint32_t i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = bf16_bits_to_f32(src[i]);
+  float *dst = h + static_cast<uint64_t>(blockIdx.x) * padded;
+  for (uint32_t i = threadIdx.x; i < padded; i += blockDim.x) dst[i] = i < hidden ? bf16_bits_to_f32(src[i]) * scale : 0.0f;
 }
 
 // x[row][:] = bf16(h[row][:] * rsqrt(mean(h^2) + eps) * w): the arithmetic, thread mapping and
 // summation order of the single-token prologue (step_device.cuh norm_single_*), so a token
-// normalises to the same bits whichever path carries it.
+// normalises to the same bits whichever path carries it.  row_index (optional): block i takes row
+// row_index[i] of h.
 __global__ void __launch_bounds__(kNormThreads) block_norm_kernel(const float *h, const uint16_t *w, float eps,
-                                                                  uint32_t cols, uint16_t *x, uint32_t x_stride) {
+                                                                  uint32_t cols, uint16_t *x, uint32_t x_stride,
+                                                                  const uint32_t *row_index) {
   __shared__ float scratch[40];
   pdl_trigger();
   NormWeightRegs weights;
   norm_weights_preload(weights, w, cols);
   pdl_wait();
   NormValueRegs values;
-  norm_single_load(values, h + static_cast<uint64_t>(blockIdx.x) * cols, cols);
+  const uint32_t source = row_index != nullptr ? row_index[blockIdx.x] : blockIdx.x;
+  norm_single_load(values, h + static_cast<uint64_t>(source) * cols, cols);
   norm_single_finish(x + static_cast<uint64_t>(blockIdx.x) * x_stride, values, weights, eps, cols, scratch);
 }
 
@@ -189,6 +193,29 @@ bool plan_workspace(const Session *s, BlockWorkspace *ws, StaticArena &arena, vo
   const ModelDims &d = s->dims;
   const uint64_t ah = d.attention_hidden(), kvh = d.kv_hidden(), qkv_rows = ah + 2 * kvh;
   const uint64_t rows = ws->max_rows, sample = ws->sample_rows;
+  if (s->parallel) {
+    const ParallelPlan &plan = *s->parallel;
+    const uint64_t words = plan.element_bytes() / 2u;
+    const uint64_t slots = rows * plan.max_heads * kWindowMaxSplits;
+    bool ok = carve(arena, base, rows * plan.width_pad * words, &ws->x_bf16);
+    ok = ok && carve(arena, base, rows * plan.max_qkv_pad, &ws->qkv);
+    ok = ok && carve(arena, base, rows * plan.max_attn_pad * words, &ws->attn);
+    ok = ok && carve(arena, base, rows * plan.width_pad, &ws->h_b);
+    ok = ok && carve(arena, base, rows * std::max<uint64_t>(plan.max_ff_pad, 8u) * words, &ws->ff);
+    ok = ok && carve(arena, base, sample * d.vocab, &ws->logits);
+    ok = ok && carve(arena, base, slots * plan.max_v_pad, &ws->partial_acc);
+    ok = ok && carve(arena, base, slots, &ws->partial_m);
+    ok = ok && carve(arena, base, slots, &ws->partial_l);
+    ok = ok && carve(arena, base, rows * plan.max_heads, &ws->attn_tickets);
+    ok = ok && carve(arena, base, gemm_tc_workspace_bytes(ws->max_rows, s->sm_count) / sizeof(float), &ws->gemm_workspace);
+    ok = ok && carve(arena, base, sample * kBlockArgmaxChunks, &ws->best_value);
+    ok = ok && carve(arena, base, sample * kBlockArgmaxChunks, &ws->best_index);
+    ok = ok && carve(arena, base, rows, &ws->attn_rows);
+    ok = ok && carve(arena, base, rows, &ws->token_rows);
+    ok = ok && carve(arena, base, sample, &ws->sample_rows_dev);
+    ok = ok && carve(arena, base, sample, &ws->head_rows);
+    return ok;
+  }
   const uint64_t max_x = std::max<uint64_t>(std::max<uint64_t>(d.hidden, d.intermediate), ah);
   const uint32_t max_out = std::max(std::max<uint32_t>(static_cast<uint32_t>(qkv_rows), 2u * d.intermediate),
                                     std::max(d.hidden, d.vocab));
@@ -210,6 +237,7 @@ bool plan_workspace(const Session *s, BlockWorkspace *ws, StaticArena &arena, vo
   ok = ok && carve(arena, base, rows, &ws->attn_rows);
   ok = ok && carve(arena, base, rows, &ws->token_rows);
   ok = ok && carve(arena, base, sample, &ws->sample_rows_dev);
+  ok = ok && carve(arena, base, sample, &ws->head_rows);
   return ok;
 }
 
@@ -228,6 +256,7 @@ struct BlockPlan {
   // the tensor maps of the caches the rows live in (rows[r].map_index), or empty for the fused kernel.
   std::vector<TensorMapStorage> k_maps, v_maps;
   uint32_t longest = 0;  // longest context among the rows
+  uint32_t capture_row = 0;  // where the block's rows begin in the session's stream capture
 };
 
 cudaError_t block_gemm(const BlockPlan &b, const uint16_t *weight, uint32_t rows, uint32_t cols, const uint16_t *x,
@@ -262,13 +291,20 @@ cudaError_t enqueue_block_layers(const BlockPlan &b, uint64_t *launches) {
   const uint32_t qkv_rows = ah + 2u * kvh;
   uint64_t n = 0;
   cudaError_t err = launch_with_pdl(block_embed_kernel, dim3(b.rows), dim3(256), 0, b.stream, false, ws.token_rows,
-                                    arena_at(s, s->layout.embeddings), d.hidden, ws.h_b);
+                                    arena_at(s, s->layout.embeddings), d.hidden, ws.h_b,
+                                    s->parallel ? s->parallel->embedding_scale : 1.0f,
+                                    s->parallel ? s->parallel->width_pad : d.hidden);
   n += 1;
+  if (s->parallel) {
+    if (launches != nullptr) *launches += n;
+    if (err != cudaSuccess) return err;
+    return enqueue_parallel_block_layers(s, ParallelBlock{b.stream, b.rows, b.longest, b.publish, b.capture_row}, launches);
+  }
   for (uint32_t l = 0; err == cudaSuccess && l < d.layers; ++l) {
     const LayerLayout &L = s->layout.layers[l];
     // attention half
     err = launch_with_pdl(block_norm_kernel, dim3(b.rows), dim3(kNormThreads), 0, b.stream, b.pdl, ws.h_b,
-                          arena_at(s, L.rms_attn), s->rms_eps, d.hidden, ws.x_bf16, d.hidden);
+                          arena_at(s, L.rms_attn), s->rms_eps, d.hidden, ws.x_bf16, d.hidden, nullptr);
     if (err == cudaSuccess)
       err = block_gemm(b, s->weights->qkv_packed + static_cast<uint64_t>(l) * qkv_rows * d.hidden, qkv_rows, d.hidden,
                        ws.x_bf16, d.hidden, kEpilogueStore, nullptr, ws.qkv, nullptr);
@@ -333,7 +369,7 @@ cudaError_t enqueue_block_layers(const BlockPlan &b, uint64_t *launches) {
     // MLP half
     if (err == cudaSuccess)
       err = launch_with_pdl(block_norm_kernel, dim3(b.rows), dim3(kNormThreads), 0, b.stream, b.pdl, ws.h_a,
-                            arena_at(s, L.rms_mlp), s->rms_eps, d.hidden, ws.x_bf16, d.hidden);
+                            arena_at(s, L.rms_mlp), s->rms_eps, d.hidden, ws.x_bf16, d.hidden, nullptr);
     if (err == cudaSuccess)
       err = block_gemm(b, s->weights->gate_up_packed + gate_up_packed_offset(s, l),
                        2u * d.intermediate, d.hidden, ws.x_bf16, d.hidden, kEpilogueSwiglu, nullptr, nullptr, ws.ff);
@@ -344,6 +380,25 @@ cudaError_t enqueue_block_layers(const BlockPlan &b, uint64_t *launches) {
     n += 4;
   }
   if (launches != nullptr) *launches += n;
+  return err;
+}
+
+// Final norm and lm_head of `count` rows of the block into ws.logits; row_index (device) names the
+// rows, null: the first `count`.
+cudaError_t enqueue_block_head(const BlockPlan &b, uint32_t count, const uint32_t *row_index, uint64_t *launches) {
+  Session *s = b.model;
+  const ModelDims &d = s->dims;
+  const BlockWorkspace &ws = s->weights->block_ws;
+  if (s->parallel) return enqueue_parallel_block_head(s, b.stream, count, row_index, launches);
+  BlockPlan head = b;
+  head.rows = count;
+  cudaError_t err = launch_with_pdl(block_norm_kernel, dim3(count), dim3(kNormThreads), 0, b.stream, b.pdl, ws.h_b,
+                                    arena_at(s, s->layout.final_norm), s->rms_eps, d.hidden, ws.x_bf16, d.hidden,
+                                    row_index);
+  if (err == cudaSuccess)
+    err = block_gemm(head, arena_at(s, s->layout.lm_head), d.vocab, d.hidden, ws.x_bf16, d.hidden, kEpilogueStore,
+                     nullptr, ws.logits, nullptr);
+  if (launches != nullptr) *launches += 2;
   return err;
 }
 
@@ -404,6 +459,7 @@ cudaError_t upload_rows(const BlockWorkspace &ws, const std::vector<FusedAttenti
 
 bool block_step_supported(const NervaCudaHfDecodeSequenceSession *s) {
   const ModelDims &d = s->dims;
+  if (s->parallel) return s->parallel->f32 || tensor_map_available();
   if (s->tp_world > 1 || s->has_moe || d.mla() || !s->fused_attention || d.dtype != NERVA_DTYPE_BF16) return false;
   const uint64_t ah = d.attention_hidden();
   if (d.hidden % 64u != 0 || ah % 64u != 0 || d.intermediate % 64u != 0) return false;
@@ -412,6 +468,12 @@ bool block_step_supported(const NervaCudaHfDecodeSequenceSession *s) {
     if (L.mlp_kind != NERVA_MLP_KIND_DENSE || L.o_bias != kMissingOffset) return false;
   }
   return tensor_map_available();
+}
+
+cudaError_t launch_argmax_partials(cudaStream_t stream, const float *logits, uint32_t vocab, uint32_t rows, uint32_t chunks,
+                                   float *best_value, uint32_t *best_index, bool pdl) {
+  return launch_with_pdl(block_argmax_partials_kernel, dim3(chunks, rows), dim3(256), 0, stream, pdl, logits, vocab,
+                         best_value, best_index);
 }
 
 cudaError_t allocate_block_workspace(NervaCudaHfDecodeSequenceSession *s) {
@@ -427,6 +489,11 @@ cudaError_t allocate_block_workspace(NervaCudaHfDecodeSequenceSession *s) {
   StaticArena arena(ws.bytes);
   if (!plan_workspace(s, &ws, arena, ws.block)) return cudaErrorMemoryAllocation;
   const ModelDims &d = s->dims;
+  if (s->parallel) {
+    // tickets begin at zero; the padding of the activation rows has to be finite
+    err = cudaMemsetAsync(ws.block, 0, ws.bytes, s->stream);
+    return err == cudaSuccess ? configure_gemm_tc_kernel() : err;
+  }
   const uint32_t max_out = std::max(std::max<uint32_t>(static_cast<uint32_t>(d.attention_hidden() + 2 * d.kv_hidden()),
                                                       2u * d.intermediate),
                                     std::max(d.hidden, d.vocab));
@@ -474,16 +541,10 @@ cudaError_t enqueue_block_decode(NervaCudaHfDecodeSequenceSession *const *sessio
   uint64_t n = 0;
   err = enqueue_block_layers(b, &n);
   // final norm, lm_head, arg-max: per row
+  if (err == cudaSuccess) err = enqueue_block_head(b, count, nullptr, &n);
   if (err == cudaSuccess)
-    err = launch_with_pdl(block_norm_kernel, dim3(count), dim3(kNormThreads), 0, stream, b.pdl, ws.h_b,
-                          arena_at(model, model->layout.final_norm), model->rms_eps, d.hidden, ws.x_bf16, d.hidden);
-  if (err == cudaSuccess)
-    err = block_gemm(b, arena_at(model, model->layout.lm_head), d.vocab, d.hidden, ws.x_bf16, d.hidden, kEpilogueStore,
-                     nullptr, ws.logits, nullptr);
-  if (err == cudaSuccess)
-    err = launch_with_pdl(block_argmax_partials_kernel, dim3(kBlockArgmaxChunks, count), dim3(256), 0, stream, b.pdl,
-                          ws.logits, d.vocab, ws.best_value, ws.best_index);
-  n += 3;
+    err = launch_argmax_partials(stream, ws.logits, d.vocab, count, kBlockArgmaxChunks, ws.best_value, ws.best_index, b.pdl);
+  n += 1;
   // every row's token into its own session's ring, and its logits into the session's own buffer
   // (nerva_b200_session_read_logits), in one launch
   std::vector<BlockSampleRow> sample(count);
@@ -510,14 +571,14 @@ cudaError_t enqueue_block_decode(NervaCudaHfDecodeSequenceSession *const *sessio
   return err;
 }
 
-cudaError_t enqueue_chunked_prefill(NervaCudaHfDecodeSequenceSession *s, uint32_t prompt_count, uint32_t sample_kind,
-                                    uint64_t *launches) {
-  (void)sample_kind;
+cudaError_t enqueue_chunked_prefill(NervaCudaHfDecodeSequenceSession *s, uint32_t first, uint32_t prompt_count,
+                                    const WantedLogits &wanted, uint64_t *launches) {
   const BlockWorkspace &ws = s->weights->block_ws;
-  if (ws.block == nullptr || prompt_count == 0) return cudaErrorNotSupported;
+  if (ws.block == nullptr || first >= prompt_count) return cudaErrorNotSupported;
   const ModelDims &d = s->dims;
+  const uint64_t width = s->parallel ? s->parallel->width_pad : d.hidden;
   cudaError_t err = cudaSuccess;
-  for (uint32_t begin = 0; err == cudaSuccess && begin < prompt_count; begin += ws.max_rows) {
+  for (uint32_t begin = first; err == cudaSuccess && begin < prompt_count; begin += ws.max_rows) {
     const uint32_t rows = std::min(ws.max_rows, prompt_count - begin);
     std::vector<FusedAttentionRow> attn(rows);
     std::vector<BlockTokenRow> tokens(rows);
@@ -529,6 +590,7 @@ cudaError_t enqueue_chunked_prefill(NervaCudaHfDecodeSequenceSession *s, uint32_
     if (err != cudaSuccess) break;
     BlockPlan b{s, s->stream, rows, block_attention_splits(s, rows, begin + rows), true, s->use_pdl};
     b.longest = begin + rows;
+    b.capture_row = begin - first;
     if (ws.paged_rows && s->kv_maps) {
       b.k_maps.push_back(s->kv_map_k);  // all rows of a chunk live in this session's cache (map_index 0)
       b.v_maps.push_back(s->kv_map_v);
@@ -536,8 +598,25 @@ cudaError_t enqueue_chunked_prefill(NervaCudaHfDecodeSequenceSession *s, uint32_
     err = enqueue_block_layers(b, launches);
     if (err == cudaSuccess && begin + rows == prompt_count) {
       // the last position's residual stream becomes the session's own, where the head expects it
-      err = cudaMemcpyAsync(s->h_b, ws.h_b + static_cast<uint64_t>(rows - 1u) * d.hidden,
-                            static_cast<uint64_t>(d.hidden) * sizeof(float), cudaMemcpyDeviceToDevice, s->stream);
+      err = cudaMemcpyAsync(s->h_b, ws.h_b + static_cast<uint64_t>(rows - 1u) * width, width * sizeof(float),
+                            cudaMemcpyDeviceToDevice, s->stream);
+    }
+    // the wanted positions of this chunk, up to sample_rows of them per head launch
+    std::vector<uint32_t> place, row;
+    for (uint32_t i = 0; i < wanted.count; ++i) {
+      const uint32_t at = first + wanted.places[i];
+      if (at < begin || at >= begin + rows) continue;
+      place.push_back(i);
+      row.push_back(at - begin);
+    }
+    for (size_t i = 0; err == cudaSuccess && i < row.size(); i += ws.sample_rows) {
+      const uint32_t count = static_cast<uint32_t>(std::min<size_t>(ws.sample_rows, row.size() - i));
+      err = cudaMemcpyAsync(ws.head_rows, row.data() + i, count * sizeof(uint32_t), cudaMemcpyHostToDevice, s->stream);
+      if (err == cudaSuccess) err = enqueue_block_head(b, count, ws.head_rows, launches);
+      for (uint32_t k = 0; err == cudaSuccess && k < count; ++k)
+        err = cudaMemcpyAsync(wanted.logits + static_cast<uint64_t>(place[i + k]) * d.vocab,
+                              ws.logits + static_cast<uint64_t>(k) * d.vocab,
+                              static_cast<uint64_t>(d.vocab) * sizeof(float), cudaMemcpyDeviceToHost, s->stream);
     }
   }
   return err;

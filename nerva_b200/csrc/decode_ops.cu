@@ -21,7 +21,7 @@ __device__ __forceinline__ uint32_t current_token(const StepState &st, uint32_t 
 }
 
 __global__ void embed_kernel(StepState st, const uint16_t *embeddings, uint32_t hidden,
-                             float *input) {
+                             float *input, float scale, uint32_t padded) {
   pdl_trigger();  // the first projection may start prefetching its weights now
   const uint32_t position = *st.cursor;
   if (position >= st.max_context) {
@@ -34,7 +34,8 @@ __global__ void embed_kernel(StepState st, const uint16_t *embeddings, uint32_t 
     token = 0;
   }
   const uint16_t *row = embeddings + static_cast<uint64_t>(token) * hidden;
-  for (uint32_t i = threadIdx.x; i < hidden; i += blockDim.x) input[i] = bf16_bits_to_f32(row[i]);
+  for (uint32_t i = threadIdx.x; i < padded; i += blockDim.x)
+    input[i] = i < hidden ? bf16_bits_to_f32(row[i]) * scale : 0.0f;
 }
 
 // One block per head: blocks [0, heads) are query heads, [heads, heads+kv_heads)
@@ -303,6 +304,16 @@ __global__ void pack_gate_up_kernel(const uint16_t *gate, const uint16_t *up, ui
   }
 }
 
+__global__ void pack_rows_kernel(const uint16_t *src, uint32_t rows, uint32_t cols, uint16_t *dst, uint32_t dst_cols,
+                                 uint32_t row_step, uint32_t row_first) {
+  const uint64_t total = static_cast<uint64_t>(rows) * cols;
+  const uint64_t stride = static_cast<uint64_t>(gridDim.x) * blockDim.x;
+  for (uint64_t i = static_cast<uint64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
+    const uint64_t row = i / cols;
+    dst[(row * row_step + row_first) * dst_cols + (i - row * cols)] = src[i];
+  }
+}
+
 __global__ void identity_table_kernel(uint32_t *table, uint32_t count) {
   const uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i < count) table[i] = i;
@@ -324,8 +335,8 @@ uint32_t grid_for(uint64_t count) {
 }  // namespace
 
 cudaError_t launch_embed(cudaStream_t stream, const StepState &st, const uint16_t *embeddings,
-                         uint32_t hidden, float *input) {
-  embed_kernel<<<1, 256, 0, stream>>>(st, embeddings, hidden, input);
+                         uint32_t hidden, float *input, float scale, uint32_t padded) {
+  embed_kernel<<<1, 256, 0, stream>>>(st, embeddings, hidden, input, scale, padded == 0 ? hidden : padded);
   return cudaGetLastError();
 }
 
@@ -408,6 +419,13 @@ cudaError_t launch_pack_gate_up(cudaStream_t stream, const uint16_t *gate, const
                                 uint16_t *packed, uint32_t intermediate, uint32_t hidden) {
   pack_gate_up_kernel<<<grid_for(static_cast<uint64_t>(intermediate) * hidden), 256, 0, stream>>>(
       gate, up, packed, intermediate, hidden);
+  return cudaGetLastError();
+}
+
+cudaError_t launch_pack_rows(cudaStream_t stream, const uint16_t *src, uint32_t rows, uint32_t cols, uint16_t *dst,
+                             uint32_t dst_cols, uint32_t row_step, uint32_t row_first) {
+  pack_rows_kernel<<<grid_for(static_cast<uint64_t>(rows) * cols), 256, 0, stream>>>(src, rows, cols, dst, dst_cols,
+                                                                                   row_step, row_first);
   return cudaGetLastError();
 }
 

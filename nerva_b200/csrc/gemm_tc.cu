@@ -69,7 +69,10 @@ struct GemmKernelParams {
   uint32_t stages;
   uint32_t tmem_columns;  // allocation: two accumulator buffers of tmem_columns / 2 fp32 columns
   uint32_t epilogue;
+  uint32_t split_row;         // kEpilogueStoreSwiglu: first row of the gate/up pairs (a multiple of 32)
   const float *resid_in;
+  const uint16_t *row_scale;  // kEpilogueStore, optional: y is multiplied by row_scale[row] before the residual add
+  float softcap;              // kEpilogueStore: 0, or y becomes softcap * tanh(y / softcap)
   float *out_f32;
   uint16_t *out_bf16;
   float *workspace;
@@ -217,26 +220,35 @@ __device__ __forceinline__ uint32_t instr_desc_bf16(uint32_t n) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((kTileRows >> 4) << 24);
 }
 
-// Epilogue of 16 tokens (g .. g + 15) of accumulator row `row`, values in v.  Called by all 32 lanes
-// of a warp whose lanes hold 32 consecutive rows.
-__device__ __forceinline__ void tile_epilogue(const GemmKernelParams &p, const float (&v)[kGroup], uint32_t row,
-                                              uint32_t g, uint32_t lane) {
-  if (p.epilogue == kEpilogueSwiglu) {
+// N consecutive tokens m0 .. m0 + N - 1 of accumulator row `row`, values in v.  Called by all 32 lanes
+// of a warp whose lanes hold 32 consecutive rows (the first a multiple of 32).
+template <uint32_t N>
+__device__ __forceinline__ void row_epilogue(const GemmKernelParams &p, const float (&v)[N], uint32_t row, uint32_t m0,
+                                             uint32_t lane) {
+  const bool pairs = p.epilogue == kEpilogueSwiglu || (p.epilogue == kEpilogueStoreSwiglu && row >= p.split_row);
+  if (pairs) {
     // rows interleaved (gate, up): the neighbouring lane holds the other half of the pair
+    const uint32_t base = p.epilogue == kEpilogueStoreSwiglu ? p.split_row : 0u;
+    const uint32_t width = (p.rows - base) / 2u;
 #pragma unroll
-    for (uint32_t j = 0; j < kGroup; ++j) {
+    for (uint32_t j = 0; j < N; ++j) {
       const float other = __shfl_xor_sync(0xffffffffu, v[j], 1);
-      const uint32_t m = g + j;
+      const uint32_t m = m0 + j;
       if ((lane & 1u) == 0 && row + 1u < p.rows && m < p.tokens)
-        p.out_bf16[static_cast<uint64_t>(m) * (p.rows / 2u) + row / 2u] = f32_to_bf16_bits(silu(v[j]) * other);
+        p.out_bf16[static_cast<uint64_t>(m) * width + (row - base) / 2u] = f32_to_bf16_bits(silu(v[j]) * other);
     }
   } else if (row < p.rows) {
+    const uint32_t width = p.epilogue == kEpilogueStoreSwiglu ? p.split_row : p.rows;
+    const float scale = p.row_scale != nullptr ? bf16_bits_to_f32(p.row_scale[row]) : 1.0f;
 #pragma unroll
-    for (uint32_t j = 0; j < kGroup; ++j) {
-      const uint32_t m = g + j;
+    for (uint32_t j = 0; j < N; ++j) {
+      const uint32_t m = m0 + j;
       if (m < p.tokens) {
-        const uint64_t at = static_cast<uint64_t>(m) * p.rows + row;
-        p.out_f32[at] = p.resid_in != nullptr ? v[j] + __ldcg(p.resid_in + at) : v[j];
+        const uint64_t at = static_cast<uint64_t>(m) * width + row;
+        float y = v[j];
+        if (p.row_scale != nullptr) y *= scale;
+        if (p.softcap > 0.0f) y = p.softcap * tanhf(y / p.softcap);
+        p.out_f32[at] = p.resid_in != nullptr ? y + __ldcg(p.resid_in + at) : y;
       }
     }
   }
@@ -249,29 +261,6 @@ __device__ __forceinline__ void tile_epilogue(const GemmKernelParams &p, const f
 // written them itself) leave at once.
 constexpr uint32_t kFixupMaxListed = 320;  // contributors whose slots are looked up once, in shared memory
 constexpr uint32_t kFixupBatch = 8;
-
-__device__ __forceinline__ void fixup_epilogue(const GemmKernelParams &p, const float4 &v, uint32_t row, uint32_t m0) {
-  const float vals[4] = {v.x, v.y, v.z, v.w};
-  if (p.epilogue == kEpilogueSwiglu) {
-    // rows interleaved (gate, up): the neighbouring lane holds the other half of the pair
-#pragma unroll
-    for (uint32_t j = 0; j < 4u; ++j) {
-      const float other = __shfl_xor_sync(0xffffffffu, vals[j], 1);
-      const uint32_t m = m0 + j;
-      if ((threadIdx.x & 1u) == 0 && row + 1u < p.rows && m < p.tokens)
-        p.out_bf16[static_cast<uint64_t>(m) * (p.rows / 2u) + row / 2u] = f32_to_bf16_bits(silu(vals[j]) * other);
-    }
-  } else if (row < p.rows) {
-#pragma unroll
-    for (uint32_t j = 0; j < 4u; ++j) {
-      const uint32_t m = m0 + j;
-      if (m < p.tokens) {
-        const uint64_t at = static_cast<uint64_t>(m) * p.rows + row;
-        p.out_f32[at] = p.resid_in != nullptr ? vals[j] + __ldcg(p.resid_in + at) : vals[j];
-      }
-    }
-  }
-}
 
 __global__ void __launch_bounds__(4 * kTileRows) gemm_fixup_kernel(GemmKernelParams p, uint32_t gemm_blocks) {
   __shared__ uint32_t range[2];
@@ -321,7 +310,8 @@ __global__ void __launch_bounds__(4 * kTileRows) gemm_fixup_kernel(GemmKernelPar
       }
     }
   }
-  fixup_epilogue(p, v, tile * kTileRows + row_in_tile, m0);
+  const float vals[4] = {v.x, v.y, v.z, v.w};
+  row_epilogue<4>(p, vals, tile * kTileRows + row_in_tile, m0, threadIdx.x & 31u);
 }
 
 __global__ void __launch_bounds__(kGemmThreads, 2)
@@ -473,7 +463,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         for (uint32_t g = 0; g < p.n_pad; g += kGroup) {
           float v[kGroup];
           tmem_load16(taddr + g, v);
-          tile_epilogue(p, v, row, g, lane);
+          row_epilogue<kGroup>(p, v, row, g, lane);
         }
       }
       tcgen05_fence_before();
@@ -579,7 +569,8 @@ bool gemm_tc_eligible(const GemmParams &g) {
   return g.tokens >= 1 && g.tokens <= kGemmMaxTokens && g.cols % kSliceK == 0 && g.cols != 0 && g.rows != 0 &&
          reinterpret_cast<uintptr_t>(g.weight) % 16u == 0 && reinterpret_cast<uintptr_t>(g.x) % 16u == 0 &&
          (g.epilogue != kEpilogueSwiglu || g.rows % 2u == 0) &&
-         (g.epilogue == kEpilogueStore || g.epilogue == kEpilogueSwiglu);
+         (g.epilogue != kEpilogueStoreSwiglu || (g.rows % 2u == 0 && g.split_row % 32u == 0 && g.split_row <= g.rows)) &&
+         (g.epilogue == kEpilogueStore || g.epilogue == kEpilogueSwiglu || g.epilogue == kEpilogueStoreSwiglu);
 }
 
 uint64_t gemm_tc_workspace_bytes(uint32_t tokens, uint32_t sm_count) {
@@ -603,7 +594,10 @@ cudaError_t launch_gemm_tc(cudaStream_t stream, const GemmParams &g, uint32_t sm
   p.stages = stages_for(p.n_pad);
   p.tmem_columns = tmem_columns_for(p.n_pad);
   p.epilogue = g.epilogue;
+  p.split_row = g.split_row;
   p.resid_in = g.resid_in;
+  p.row_scale = g.row_scale;
+  p.softcap = g.softcap;
   p.out_f32 = g.out_f32;
   p.out_bf16 = g.out_bf16;
   p.workspace = g.workspace;

@@ -44,6 +44,7 @@ enum ProjectionEpilogue : uint32_t {
   kEpilogueStore = 0,     // out_f32[row] = y
   kEpilogueSwiglu = 1,    // rows interleaved (gate, up): out_bf16[row/2] = bf16(silu(gate) * up)
   kEpilogueArgmax = 2,    // out_f32[row] = y and per-block (best value, lowest index)
+  kEpilogueStoreSwiglu = 3,  // block projection: rows below split_row as kEpilogueStore, the rest as kEpilogueSwiglu
 };
 
 // ---- tensor-parallel exchange of a row-parallel projection (O, down) ----
@@ -110,7 +111,11 @@ struct GemmParams {
   uint32_t tokens;
   uint32_t epilogue;       // kEpilogueStore: out_f32[token][row] = y (+ resid_in[token][row])
                            // kEpilogueSwiglu: rows interleaved (gate, up): out_bf16[token][row/2]
-  const float *resid_in;   // optional [tokens][rows]
+                           // kEpilogueStoreSwiglu: out_f32[token][split_row], out_bf16[token][(rows - split_row)/2]
+  uint32_t split_row;
+  const uint16_t *row_scale;  // optional bf16 [rows], kEpilogueStore: y * row_scale[row] is what is stored / added
+  float softcap;           // kEpilogueStore: 0, or softcap * tanh(y / softcap) is stored
+  const float *resid_in;   // optional [tokens][rows]; may be out_f32
   float *out_f32;          // [tokens][rows]
   uint16_t *out_bf16;      // [tokens][rows/2]
   float *workspace;        // gemm_tc_workspace_bytes(tokens, sm_count)
@@ -149,8 +154,9 @@ struct StepState {
 };
 
 // input[h] = embedding[token(cursor)][h] as f32.
+// scale: multiplies every element (1: as stored); padded (0: hidden): elements of `input`, zero beyond hidden.
 cudaError_t launch_embed(cudaStream_t stream, const StepState &st, const uint16_t *embeddings,
-                         uint32_t hidden, float *input);
+                         uint32_t hidden, float *input, float scale = 1.0f, uint32_t padded = 0);
 
 struct QkvPrepareParams {
   float *qkv;  // [heads*d | kv_heads*d | kv_heads*d] f32, q is normalised/rotated in place
@@ -319,6 +325,97 @@ cudaError_t configure_moe_kernels();
 // Two launches: routing + gate/up of the chosen experts, then SwiGLU + down and the weighted sum.
 cudaError_t launch_moe_experts(cudaStream_t stream, const MoeExpertParams &p, uint32_t sm_count, bool pdl);
 
+// ---- parallel-block layers (parallel_projection.cu) ----
+// Several weight matrices in one launch for one token: the projections of a layer whose mixer and
+// feed-forward read the same normalised vector, and the two output projections that are summed into
+// the residual stream.  All vectors are padded to multiples of 64 with zeros, matrices have zero
+// columns (and rows) there.
+enum ParallelProjectionKind : uint32_t {
+  kParallelIn = 0,    // x = norm(h + step); matrix 0 -> out_f32 (fp32), matrix 1 (gate/up rows interleaved) -> out_act
+  kParallelOut = 1,   // h_out = (h + step) + scale0 * (matrix 0 . x0) + scale1 * (matrix 1 . x1)
+  kParallelHead = 2,  // x = norm(h); matrix 0 -> soft-capped out_f32 and per-block arg-max partials
+};
+struct ParallelProjectionParams {
+  const uint16_t *w0, *w1;       // [rows][cols] bf16
+  uint32_t rows0, cols0, rows1, cols1;  // rows1 == 0: no second matrix
+  const float *h;                // [cols0 or rows0] residual stream
+  const uint16_t *step;          // optional bf16 vector added to h (a looped layer's pass vector)
+  const uint16_t *norm;          // bf16 [cols0], zero beyond width
+  uint32_t width;                // elements the norm's mean is taken over
+  float eps;
+  const void *x0, *x1;           // kParallelOut: activation vectors
+  const uint16_t *scale0, *scale1;  // kParallelOut: optional bf16 [rows0]
+  float *h_out;                  // kParallelOut; may be h
+  float *out_f32;
+  void *out_act;                 // kParallelIn: [rows1 / 2]
+  float softcap;
+  float *best_value;             // kParallelHead [blocks]
+  uint32_t *best_index;
+  uint32_t *error_word;
+  uint32_t pdl;
+};
+// bf16 activations, weights through the TMA ring (row_stream.cuh).  Shapes it cannot hold go to the plain form.
+bool parallel_stream_eligible(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count);
+uint32_t parallel_stream_blocks(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count);
+cudaError_t launch_parallel_projection(cudaStream_t stream, uint32_t kind, const ParallelProjectionParams &p,
+                                       uint32_t sm_count);
+cudaError_t configure_parallel_projection();
+// The plain form: any number of tokens, activations fp32 (f32 = true: true fp32 throughout) or bf16,
+// no norm and no pass vector in front (x0 is the activation block of kParallelIn / kParallelHead).
+// Row strides are cols0 / cols1 for x, rows0 for h, h_out and out_f32, rows1 / 2 for out_act.
+cudaError_t launch_parallel_projection_plain(cudaStream_t stream, uint32_t kind, const ParallelProjectionParams &p,
+                                             uint32_t tokens, bool f32);
+// x[row] = norm(h[source] + step) for `rows` rows; source = row_index[row] when given.  step is also added
+// to h itself (then no row_index).  x is fp32 or bf16 [rows][padded].
+cudaError_t launch_stream_norm(cudaStream_t stream, float *h, const uint16_t *step, const uint16_t *norm, float eps,
+                               uint32_t width, uint32_t padded, void *x, bool f32, uint32_t rows,
+                               const uint32_t *row_index, bool pdl);
+
+// ---- sliding-window grouped-query attention (window_attention.cu) ----
+// Head sizes are arbitrary up to 256; cached rows are [kv_heads][qk_pad] and [kv_heads][v_pad] elements
+// (sizes rounded up to 16, zeros behind the head), bf16 or fp32, in the session's 16-token pages.
+struct WindowAttentionShape {
+  uint32_t heads, kv_heads, qk_dim, v_dim, qk_pad, v_pad;
+  uint32_t window;         // keys a query sees, itself included; 0: all
+  uint32_t rotary_pairs;   // pairs (i, i + rotary_pairs) of a head that are rotated
+  uint32_t qk_norm;        // weightless RMS norm of q and k after the rotation
+  float rotary_magnitude;  // factor on cos and sin
+  float scale, eps;
+  const float *frequency;  // [rotary_pairs] angle per position
+};
+struct WindowAttentionParams {
+  WindowAttentionShape s;
+  float *qkv;              // [rows][qkv_stride]: q | k | v of the projection; prepared queries are written back
+  uint32_t qkv_stride;
+  void *out;               // [rows][out_stride] bf16 or fp32
+  uint32_t out_stride;
+  uint64_t key_offset, value_offset;  // elements from the start of a session's cache to this layer run's pages
+  uint32_t splits;
+  float *partial_acc, *partial_m, *partial_l;  // [rows][heads][splits][...]
+  uint32_t *tickets;       // [rows][heads], zero between launches
+  uint32_t f32;            // cache and output in fp32
+  uint32_t pdl;
+  // one token of one session
+  const uint32_t *cursor;
+  uint32_t max_context, page_count;
+  void *keys, *values;
+  const uint32_t *page_table;
+  uint32_t *error_word;
+  // block step: the rows' positions and caches; queries prepared and K/V cached by launch_window_publish
+  const struct FusedAttentionRow *rows;
+  uint32_t row_count;
+};
+constexpr uint32_t kWindowMaxSplits = 16;
+bool window_attention_supported(const WindowAttentionShape &s, bool f32);
+uint32_t window_attention_splits(uint32_t target_context, uint32_t window);
+cudaError_t configure_window_attention();
+// q/k rotation and norm, K/V rows into the cache, for the rows of a block step.
+cudaError_t launch_window_publish(cudaStream_t stream, const WindowAttentionParams &p);
+// One token per row: the lone decode step (rows == nullptr: prepares q and appends K/V itself) or block rows.
+cudaError_t launch_window_attention(cudaStream_t stream, const WindowAttentionParams &p);
+// Consecutive positions of one session on the tensor pipe (bf16 cache only).
+cudaError_t launch_window_prefill(cudaStream_t stream, const WindowAttentionParams &p);
+
 // ---- greedy sampling ----
 // Reduces per-block (value, index) partials, writes the token slot at the
 // cursor and advances the cursor.  sample == 0: only advances the cursor.
@@ -334,6 +431,9 @@ struct TpSample {
 cudaError_t launch_sample_greedy(cudaStream_t stream, const StepState &st, const float *best_value,
                                  const uint32_t *best_index, uint32_t partials, uint32_t sample,
                                  bool pdl = false, const TpSample *tp = nullptr);
+// Arg-max candidates of `chunks` slices of each row's logits: best_value / best_index [rows][chunks].
+cudaError_t launch_argmax_partials(cudaStream_t stream, const float *logits, uint32_t vocab, uint32_t rows, uint32_t chunks,
+                                   float *best_value, uint32_t *best_index, bool pdl);
 // One row of a packed step for the batched sampler: the row's session (cursor, token ring, ...) and
 // where that session keeps the logits it sampled from (nullable).
 struct BlockSampleRow {
@@ -369,6 +469,10 @@ cudaError_t launch_pack_qkv(cudaStream_t stream, const uint16_t *wq, const uint1
                             uint64_t kv_elems);
 cudaError_t launch_pack_gate_up(cudaStream_t stream, const uint16_t *gate, const uint16_t *up,
                                 uint16_t *packed, uint32_t intermediate, uint32_t hidden);
+// Copies a [rows][cols] matrix to dst row r * row_step + row_first with dst_cols columns per row
+// (columns beyond cols are left as they are).
+cudaError_t launch_pack_rows(cudaStream_t stream, const uint16_t *src, uint32_t rows, uint32_t cols, uint16_t *dst,
+                             uint32_t dst_cols, uint32_t row_step, uint32_t row_first);
 cudaError_t launch_identity_table(cudaStream_t stream, uint32_t *table, uint32_t count);
 cudaError_t launch_fill_normal_bf16(cudaStream_t stream, uint16_t *out, uint64_t count,
                                     uint64_t seed, uint64_t tensor_id, float std);

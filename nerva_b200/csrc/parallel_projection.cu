@@ -1,0 +1,368 @@
+// Projections of a parallel-block layer (one norm in front of mixer and feed-forward, both results
+// summed into the residual stream) for one token, and the plain any-shape form of the same for a
+// block of tokens.
+//
+// The streaming form puts two weight matrices into one launch on the row-stream core
+// (row_stream.cuh): its ring runs across a job list, so the second matrix's bytes follow the first's
+// without a gap.
+//   kParallelIn    [Q; K; V] and the interleaved gate/up matrix behind one norm prologue
+//   kParallelOut   O and down, dealt to the blocks by the same row ranges, so the block that owns a
+//                  row of the stream has both sums and writes h + scale0 * O + scale1 * down once
+//   kParallelHead  the head behind the final norm, logits soft-capped before the arg-max
+// A layer is three launches with the attention in between, and the residual stream is read and
+// written once.
+#include "kernels.cuh"
+#include "row_stream.cuh"
+#include "step_device.cuh"
+
+namespace nb {
+namespace {
+
+constexpr uint32_t kNoIndex = 0xffffffffu;
+constexpr uint32_t kPrewaitSlots = kStreamSlots - 1;  // ring slots filled ahead of a norm prologue's loads
+
+__device__ __forceinline__ bool candidate_better(float v, uint32_t i, float best_v, uint32_t best_i) {
+  return v > best_v || (v == best_v && i < best_i);
+}
+__device__ __forceinline__ float soft_cap(float y, float cap) { return cap > 0.0f ? cap * tanhf(y / cap) : y; }
+
+struct ParallelShared {
+  StreamShared first, second;  // the ring's barriers are first's; each job has its own edge records
+  JobDesc jobs[2];
+  float scratch[40];
+  float best_v[kStreamWarps];
+  uint32_t best_i[kStreamWarps];
+};
+
+__host__ __device__ inline uint32_t round128(uint32_t v) { return (v + 127u) & ~127u; }
+
+template <uint32_t KIND>
+__global__ void __launch_bounds__(kStreamThreads, 1) parallel_stream_kernel(ParallelProjectionParams p) {
+  extern __shared__ __align__(128) uint8_t smem[];
+  uint8_t *ring = smem;
+  uint16_t *x0 = reinterpret_cast<uint16_t *>(smem + kRingBytes);
+  uint16_t *x1 = reinterpret_cast<uint16_t *>(smem + kRingBytes + round128(p.cols0 * 2u));
+  const uint32_t x_bytes = round128(p.cols0 * 2u) + (KIND == kParallelOut && p.rows1 != 0 ? round128(p.cols1 * 2u) : 0u);
+  ParallelShared &sh = *reinterpret_cast<ParallelShared *>(smem + kRingBytes + x_bytes);
+  float *total0 = reinterpret_cast<float *>(smem + kRingBytes + x_bytes + round128(sizeof(ParallelShared)));
+  const bool second = KIND != kParallelHead && p.rows1 != 0;
+  const uint32_t unit1 = KIND == kParallelIn ? 2u : 1u;
+
+  pdl_trigger();
+  if (threadIdx.x == 0) {
+    sh.jobs[0] = JobDesc{p.w0, p.rows0, p.cols0, 1, 0};
+    sh.jobs[1] = JobDesc{p.w1, p.rows1, KIND == kParallelIn ? p.cols0 : p.cols1, unit1, 0};
+  }
+  __syncthreads();
+  RowStream rs;
+  stream_init(rs, ring, sh.first, sh.jobs, second ? 2u : 1u);
+  stream_fill(rs, KIND == kParallelOut ? kStreamSlots : kPrewaitSlots);
+
+  uint32_t begin0, end0, begin1 = 0, end1 = 0;
+  block_row_range(p.rows0, 1, blockIdx.x, gridDim.x, &begin0, &end0);
+  if (second) block_row_range(p.rows1, unit1, blockIdx.x, gridDim.x, &begin1, &end1);
+  const uint32_t rows0 = end0 - begin0, rows1 = end1 - begin1;
+  float *total1 = total0 + rows0;
+  for (uint32_t r = threadIdx.x; r < rows0 + rows1; r += blockDim.x) total0[r] = 0.0f;
+
+  float resid_first = 0.0f;
+  if (KIND == kParallelOut) {
+    pdl_wait();
+    if (threadIdx.x < rows0) resid_first = __ldcg(p.h + begin0 + threadIdx.x);
+    const uint4 *src0 = reinterpret_cast<const uint4 *>(p.x0);
+    for (uint32_t i = threadIdx.x; i < p.cols0 / 8u; i += blockDim.x) reinterpret_cast<uint4 *>(x0)[i] = __ldcg(src0 + i);
+    if (second) {
+      const uint4 *src1 = reinterpret_cast<const uint4 *>(p.x1);
+      for (uint32_t i = threadIdx.x; i < p.cols1 / 8u; i += blockDim.x) reinterpret_cast<uint4 *>(x1)[i] = __ldcg(src1 + i);
+    }
+  } else {
+    NormWeightRegs weights, step;
+    norm_weights_preload(weights, p.norm, p.cols0);
+    if (p.step != nullptr) norm_weights_preload(step, p.step, p.cols0);
+    pdl_wait();
+    NormValueRegs values;
+    norm_single_load(values, p.h, p.cols0);
+    stream_fill(rs);  // the ring slot held back, now behind the activation loads
+    if (p.step != nullptr) {
+#pragma unroll
+      for (uint32_t k = 0; k < kNormRegIters; ++k) {
+        values.v[k].x += bf16x2_lo(step.w[k].x);
+        values.v[k].y += bf16x2_hi(step.w[k].x);
+        values.v[k].z += bf16x2_lo(step.w[k].y);
+        values.v[k].w += bf16x2_hi(step.w[k].y);
+      }
+    }
+    norm_single_finish(x0, values, weights, p.eps, p.cols0, sh.scratch, p.width);
+  }
+  __syncthreads();
+
+  stream_consume(rs, sh.first, 0, x0, total0, p.error_word);
+  if (second) stream_consume(rs, sh.second, 1, KIND == kParallelOut ? x1 : x0, total1, p.error_word);
+  __syncthreads();
+
+  if (KIND == kParallelIn) {
+    for (uint32_t r = threadIdx.x; r < rows0; r += blockDim.x)
+      p.out_f32[begin0 + r] = stream_row_total(sh.first, total0, r);
+    uint16_t *act = reinterpret_cast<uint16_t *>(p.out_act);
+    for (uint32_t i = threadIdx.x; i < rows1 / 2u; i += blockDim.x) {
+      const float gate = stream_row_total(sh.second, total1, 2u * i);
+      const float up = stream_row_total(sh.second, total1, 2u * i + 1u);
+      act[begin1 / 2u + i] = f32_to_bf16_bits(silu(gate) * up);
+    }
+  } else if (KIND == kParallelOut) {
+    for (uint32_t r = threadIdx.x; r < rows0; r += blockDim.x) {
+      const uint32_t row = begin0 + r;
+      float resid = r == threadIdx.x ? resid_first : __ldcg(p.h + row);
+      if (p.step != nullptr) resid += bf16_bits_to_f32(p.step[row]);
+      float y = stream_row_total(sh.first, total0, r);
+      if (p.scale0 != nullptr) y *= bf16_bits_to_f32(p.scale0[row]);
+      if (second) {
+        float z = stream_row_total(sh.second, total1, r);
+        if (p.scale1 != nullptr) z *= bf16_bits_to_f32(p.scale1[row]);
+        y += z;
+      }
+      p.h_out[row] = resid + y;
+    }
+  } else {
+    float bv = -INFINITY;
+    uint32_t bi = kNoIndex;
+    for (uint32_t r = threadIdx.x; r < rows0; r += blockDim.x) {
+      const float v = soft_cap(stream_row_total(sh.first, total0, r), p.softcap);
+      p.out_f32[begin0 + r] = v;
+      if (isfinite(v) && candidate_better(v, begin0 + r, bv, bi)) {
+        bv = v;
+        bi = begin0 + r;
+      }
+    }
+    for (int offset = 16; offset > 0; offset >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, offset);
+      const uint32_t oi = __shfl_xor_sync(0xffffffffu, bi, offset);
+      if (oi != kNoIndex && candidate_better(ov, oi, bv, bi)) {
+        bv = ov;
+        bi = oi;
+      }
+    }
+    if ((threadIdx.x & 31u) == 0) {
+      sh.best_v[threadIdx.x >> 5] = bv;
+      sh.best_i[threadIdx.x >> 5] = bi;
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+      bv = -INFINITY;
+      bi = kNoIndex;
+      for (uint32_t w = 0; w < kStreamWarps; ++w) {
+        if (sh.best_i[w] != kNoIndex && candidate_better(sh.best_v[w], sh.best_i[w], bv, bi)) {
+          bv = sh.best_v[w];
+          bi = sh.best_i[w];
+        }
+      }
+      p.best_value[blockIdx.x] = bv;
+      p.best_index[blockIdx.x] = bi;
+    }
+  }
+  stream_drain(rs);
+}
+
+uint32_t stream_blocks(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count) {
+  // one block per SM; fewer when the matrices are too small to give every warp of every block 4 KiB
+  uint64_t bytes = static_cast<uint64_t>(p.rows0) * p.cols0 * 2u;
+  if (kind != kParallelHead)
+    bytes += static_cast<uint64_t>(p.rows1) * (kind == kParallelIn ? p.cols0 : p.cols1) * 2u;
+  uint64_t blocks = bytes / (static_cast<uint64_t>(kStreamWarps) * 4096u);
+  if (blocks > p.rows0) blocks = p.rows0;
+  if (blocks > sm_count) blocks = sm_count;
+  return blocks == 0 ? 1u : static_cast<uint32_t>(blocks);
+}
+
+uint32_t stream_smem_bytes(uint32_t kind, const ParallelProjectionParams &p, uint32_t blocks) {
+  const bool second = kind != kParallelHead && p.rows1 != 0;
+  uint32_t rows = max_rows_per_block(p.rows0, 1, blocks);
+  if (second) rows += max_rows_per_block(p.rows1, kind == kParallelIn ? 2u : 1u, blocks);
+  return kRingBytes + round128(p.cols0 * 2u) + (kind == kParallelOut && second ? round128(p.cols1 * 2u) : 0u) +
+         round128(sizeof(ParallelShared)) + round128(rows * 4u + 16u);
+}
+
+// ---------------------------------------------------------------- plain form ----
+// One warp per output row (or gate/up pair) and up to kPlainTokens tokens; lane l takes elements
+// 2l, 2l+1 of every 64.  The form every shape and the fp32 sessions run.
+constexpr uint32_t kPlainTokens = 4;
+constexpr uint32_t kPlainWarps = 8;
+
+__device__ __forceinline__ float2 load_pair(const float *x) { return __ldcg(reinterpret_cast<const float2 *>(x)); }
+__device__ __forceinline__ float2 load_pair(const uint16_t *x) {
+  const uint32_t w = __ldcg(reinterpret_cast<const uint32_t *>(x));
+  return make_float2(bf16x2_lo(w), bf16x2_hi(w));
+}
+__device__ __forceinline__ void store_act(float *out, float v) { *out = v; }
+__device__ __forceinline__ void store_act(uint16_t *out, float v) { *out = f32_to_bf16_bits(v); }
+
+template <class X>
+__device__ __forceinline__ void plain_dots(const uint16_t *w, const X *x, uint32_t cols, uint32_t tokens,
+                                           float (&acc)[kPlainTokens]) {
+#pragma unroll
+  for (uint32_t m = 0; m < kPlainTokens; ++m) acc[m] = 0.0f;
+  for (uint32_t k = 2u * (threadIdx.x & 31u); k < cols; k += 64u) {
+    const uint32_t wk = __ldg(reinterpret_cast<const uint32_t *>(w + k));
+#pragma unroll
+    for (uint32_t m = 0; m < kPlainTokens; ++m) {
+      if (m < tokens) {
+        const float2 xk = load_pair(x + static_cast<uint64_t>(m) * cols + k);
+        acc[m] = fmaf(bf16x2_lo(wk), xk.x, acc[m]);
+        acc[m] = fmaf(bf16x2_hi(wk), xk.y, acc[m]);
+      }
+    }
+  }
+#pragma unroll
+  for (uint32_t m = 0; m < kPlainTokens; ++m) acc[m] = warp_sum(acc[m]);
+}
+
+template <class X, uint32_t KIND>
+__global__ void __launch_bounds__(kPlainWarps * 32) parallel_plain_kernel(ParallelProjectionParams p, uint32_t tokens) {
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t lane = threadIdx.x & 31u;
+  const uint32_t unit = blockIdx.x * kPlainWarps + (threadIdx.x >> 5);
+  const uint32_t m0 = blockIdx.y * kPlainTokens;
+  const uint32_t count = tokens - m0 < kPlainTokens ? tokens - m0 : kPlainTokens;
+  const X *x0 = reinterpret_cast<const X *>(p.x0) + static_cast<uint64_t>(m0) * p.cols0;
+  if (KIND == kParallelIn && unit >= p.rows0) {
+    const uint32_t pair = unit - p.rows0;
+    if (pair >= p.rows1 / 2u) return;
+    float gate[kPlainTokens], up[kPlainTokens];
+    plain_dots(p.w1 + static_cast<uint64_t>(2u * pair) * p.cols0, x0, p.cols0, count, gate);
+    plain_dots(p.w1 + static_cast<uint64_t>(2u * pair + 1u) * p.cols0, x0, p.cols0, count, up);
+    if (lane != 0) return;
+    for (uint32_t m = 0; m < count; ++m)
+      store_act(reinterpret_cast<X *>(p.out_act) + static_cast<uint64_t>(m0 + m) * (p.rows1 / 2u) + pair, silu(gate[m]) * up[m]);
+    return;
+  }
+  if (unit >= p.rows0) return;
+  float y[kPlainTokens];
+  plain_dots(p.w0 + static_cast<uint64_t>(unit) * p.cols0, x0, p.cols0, count, y);
+  if (KIND == kParallelOut) {
+    float z[kPlainTokens];
+    if (p.rows1 != 0)
+      plain_dots(p.w1 + static_cast<uint64_t>(unit) * p.cols1,
+                 reinterpret_cast<const X *>(p.x1) + static_cast<uint64_t>(m0) * p.cols1, p.cols1, count, z);
+    if (lane != 0) return;
+    const float s0 = p.scale0 != nullptr ? bf16_bits_to_f32(p.scale0[unit]) : 1.0f;
+    const float s1 = p.scale1 != nullptr ? bf16_bits_to_f32(p.scale1[unit]) : 1.0f;
+    for (uint32_t m = 0; m < count; ++m) {
+      const uint64_t at = static_cast<uint64_t>(m0 + m) * p.rows0 + unit;
+      p.h_out[at] = __ldcg(p.h + at) + (p.rows1 != 0 ? y[m] * s0 + z[m] * s1 : y[m] * s0);
+    }
+    return;
+  }
+  if (lane != 0) return;
+  for (uint32_t m = 0; m < count; ++m)
+    p.out_f32[static_cast<uint64_t>(m0 + m) * p.rows0 + unit] = KIND == kParallelHead ? soft_cap(y[m], p.softcap) : y[m];
+}
+
+constexpr uint32_t kNormThreads = 256;
+
+// One block per row; any width (values are read twice: they sit in L1 or L2).
+template <class X>
+__global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(float *h, const uint16_t *step, const uint16_t *norm,
+                                                                   float eps, uint32_t width, uint32_t padded, X *x,
+                                                                   const uint32_t *row_index) {
+  __shared__ float scratch[40];
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t source = row_index != nullptr ? row_index[blockIdx.x] : blockIdx.x;
+  float *row = h + static_cast<uint64_t>(source) * padded;
+  X *out = x + static_cast<uint64_t>(blockIdx.x) * padded;
+  float sumsq = 0.0f;
+  for (uint32_t i = threadIdx.x * 4u; i < padded; i += kNormThreads * 4u) {
+    float4 v = *reinterpret_cast<const float4 *>(row + i);
+    if (step != nullptr) {
+      const uint2 s = *reinterpret_cast<const uint2 *>(step + i);
+      v.x += bf16x2_lo(s.x);
+      v.y += bf16x2_hi(s.x);
+      v.z += bf16x2_lo(s.y);
+      v.w += bf16x2_hi(s.y);
+      *reinterpret_cast<float4 *>(row + i) = v;  // read back below by the same thread
+    }
+    sumsq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  const float total = block_sum(sumsq, scratch);
+  const float scale = 1.0f / sqrtf(total / static_cast<float>(width) + eps);
+  for (uint32_t i = threadIdx.x * 4u; i < padded; i += kNormThreads * 4u) {
+    const float4 v = *reinterpret_cast<const float4 *>(row + i);
+    const uint2 w = *reinterpret_cast<const uint2 *>(norm + i);
+    store_act(out + i, v.x * scale * bf16x2_lo(w.x));
+    store_act(out + i + 1u, v.y * scale * bf16x2_hi(w.x));
+    store_act(out + i + 2u, v.z * scale * bf16x2_lo(w.y));
+    store_act(out + i + 3u, v.w * scale * bf16x2_hi(w.y));
+  }
+}
+
+}  // namespace
+
+cudaError_t configure_parallel_projection() {
+  const int max_smem = 227 * 1024;
+  cudaError_t err = cudaFuncSetAttribute(parallel_stream_kernel<kParallelIn>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
+  if (err == cudaSuccess)
+    err = cudaFuncSetAttribute(parallel_stream_kernel<kParallelOut>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
+  if (err == cudaSuccess)
+    err = cudaFuncSetAttribute(parallel_stream_kernel<kParallelHead>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
+  return err;
+}
+
+bool parallel_stream_eligible(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count) {
+  auto aligned = [](const void *q) { return reinterpret_cast<uintptr_t>(q) % 16u == 0; };
+  if (p.rows0 == 0 || p.cols0 == 0 || p.cols0 % 8u != 0 || !aligned(p.w0)) return false;
+  if (p.rows1 != 0 && (!aligned(p.w1) || p.cols1 % 8u != 0 || (kind == kParallelIn && p.rows1 % 2u != 0))) return false;
+  if (kind == kParallelOut) {
+    if (!aligned(p.x0) || (p.rows1 != 0 && (!aligned(p.x1) || p.rows1 != p.rows0))) return false;
+  } else if (p.cols0 / 4u > kNormRegIters * kStreamThreads || !aligned(p.h) ||
+             reinterpret_cast<uintptr_t>(p.norm) % 8u != 0 || reinterpret_cast<uintptr_t>(p.step) % 8u != 0) {
+    return false;
+  }
+  return stream_smem_bytes(kind, p, stream_blocks(kind, p, sm_count)) <= 227u * 1024u;
+}
+
+uint32_t parallel_stream_blocks(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count) {
+  return stream_blocks(kind, p, sm_count);
+}
+
+cudaError_t launch_parallel_projection(cudaStream_t stream, uint32_t kind, const ParallelProjectionParams &p,
+                                       uint32_t sm_count) {
+  if (!parallel_stream_eligible(kind, p, sm_count)) return cudaErrorInvalidValue;
+  const uint32_t blocks = stream_blocks(kind, p, sm_count);
+  void (*kernel)(ParallelProjectionParams) = kind == kParallelIn    ? parallel_stream_kernel<kParallelIn>
+                                             : kind == kParallelOut ? parallel_stream_kernel<kParallelOut>
+                                                                    : parallel_stream_kernel<kParallelHead>;
+  return launch_with_pdl(kernel, dim3(blocks), dim3(kStreamThreads), stream_smem_bytes(kind, p, blocks), stream,
+                         p.pdl != 0, p);
+}
+
+cudaError_t launch_parallel_projection_plain(cudaStream_t stream, uint32_t kind, const ParallelProjectionParams &p,
+                                             uint32_t tokens, bool f32) {
+  if (tokens == 0 || p.rows0 == 0 || p.cols0 % 64u != 0 || p.cols1 % 64u != 0) return cudaErrorInvalidValue;
+  const uint32_t units = p.rows0 + (kind == kParallelIn ? p.rows1 / 2u : 0u);
+  const dim3 grid((units + kPlainWarps - 1u) / kPlainWarps, (tokens + kPlainTokens - 1u) / kPlainTokens);
+  void (*kernel)(ParallelProjectionParams, uint32_t);
+  if (f32)
+    kernel = kind == kParallelIn    ? parallel_plain_kernel<float, kParallelIn>
+             : kind == kParallelOut ? parallel_plain_kernel<float, kParallelOut>
+                                    : parallel_plain_kernel<float, kParallelHead>;
+  else
+    kernel = kind == kParallelIn    ? parallel_plain_kernel<uint16_t, kParallelIn>
+             : kind == kParallelOut ? parallel_plain_kernel<uint16_t, kParallelOut>
+                                    : parallel_plain_kernel<uint16_t, kParallelHead>;
+  return launch_with_pdl(kernel, grid, dim3(kPlainWarps * 32), 0, stream, p.pdl != 0, p, tokens);
+}
+
+cudaError_t launch_stream_norm(cudaStream_t stream, float *h, const uint16_t *step, const uint16_t *norm, float eps,
+                               uint32_t width, uint32_t padded, void *x, bool f32, uint32_t rows,
+                               const uint32_t *row_index, bool pdl) {
+  if (rows == 0 || padded % 4u != 0 || (step != nullptr && row_index != nullptr)) return cudaErrorInvalidValue;
+  if (f32)
+    return launch_with_pdl(stream_norm_kernel<float>, dim3(rows), dim3(kNormThreads), 0, stream, pdl, h, step, norm, eps,
+                           width, padded, static_cast<float *>(x), row_index);
+  return launch_with_pdl(stream_norm_kernel<uint16_t>, dim3(rows), dim3(kNormThreads), 0, stream, pdl, h, step, norm, eps,
+                         width, padded, static_cast<uint16_t *>(x), row_index);
+}
+
+}  // namespace nb

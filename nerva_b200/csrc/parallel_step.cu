@@ -1,0 +1,500 @@
+// Decoders made of parallel blocks: x += ls1 * attention(norm(x)) + ls2 * mlp(norm(x)), every size per
+// layer, a range of layers run several times with the same weights (NervaB200ParallelModel).  This
+// file turns the description into a plan (padded weights, layer runs, cache offsets) and enqueues the
+// layers for the session's two step functions: the decode step (session.cu) and the block step
+// (block_step.cu).  Token fetch, embedding, sampler, token ring, graphs, page table and forks are the
+// session's own.
+//
+// Decode step, per layer run: norm + [Q; K; V | gate/up] -> attention -> [O | down] + residual: three
+// launches.  Block step: norm, one projection for all five input matrices, q/k preparation + cache
+// append, attention, O and down with the residual add in their epilogues.
+#include <math.h>
+
+#include <algorithm>
+#include <vector>
+
+#include "session.h"
+
+namespace nb {
+namespace {
+
+typedef NervaCudaHfDecodeSequenceSession Session;
+
+uint32_t round_up(uint32_t v, uint32_t m) { return (v + m - 1u) / m * m; }
+
+// Angle per position of every rotated pair.  Scaled (YaRN): pairs that turn more than `fast` times over
+// the original length keep their frequency, pairs that turn less than `slow` times have it divided by
+// `factor`, with a linear ramp over the pair index in between, and cos and sin grow by 0.1 ln(factor) + 1.
+void rotary_table(const NervaB200ParallelLayer &l, std::vector<float> *out, float *magnitude) {
+  const uint32_t pairs = l.rotary_dims / 2u;
+  const double dims = l.rotary_dims;
+  const bool scaled = l.yarn_factor != 0.0 && pairs != 0;
+  double lo = 0.0, hi = 0.0;
+  if (scaled) {
+    auto dim_of = [&](double turns) {
+      return dims * log(l.yarn_original / (2.0 * M_PI * turns)) / (2.0 * log(l.rotary_base));
+    };
+    lo = std::max(floor(dim_of(l.yarn_fast)), 0.0);
+    hi = std::min(ceil(dim_of(l.yarn_slow)), dims - 1.0);
+  }
+  out->clear();
+  for (uint32_t i = 0; i < pairs; ++i) {
+    double f = pow(l.rotary_base, -2.0 * i / dims);
+    if (scaled) {
+      const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+      f = f / l.yarn_factor * ramp + f * (1.0 - ramp);
+    }
+    out->push_back(static_cast<float>(f));
+  }
+  *magnitude = scaled ? static_cast<float>(0.1 * log(l.yarn_factor) + 1.0) : 1.0f;
+}
+
+const uint16_t *arena_at(const Session *s, uint64_t offset) {
+  return offset == kMissingOffset ? nullptr : s->weights->arena + offset;
+}
+
+const uint16_t *step_vector(const ParallelPlan &plan, const ParallelRun &run) {
+  return run.step < 0 ? nullptr : plan.loop_vectors + static_cast<uint64_t>(run.step) * plan.width_pad;
+}
+
+// The matrices and sizes of a layer's two projection launches; activations and outputs are the caller's.
+ParallelProjectionParams layer_in(const ParallelPlan &plan, const ParallelLayerPlan &l, float eps) {
+  ParallelProjectionParams p{};
+  p.w0 = l.w_in;
+  p.rows0 = l.qkv_pad;
+  p.cols0 = plan.width_pad;
+  p.w1 = l.w_in + static_cast<uint64_t>(l.qkv_pad) * plan.width_pad;
+  p.rows1 = 2u * l.ff_pad;
+  p.norm = l.norm;
+  p.width = plan.width;
+  p.eps = eps;
+  return p;
+}
+ParallelProjectionParams layer_out(const ParallelPlan &plan, const ParallelLayerPlan &l) {
+  ParallelProjectionParams p{};
+  p.w0 = l.w_o;
+  p.rows0 = plan.width_pad;
+  p.cols0 = l.attn_pad;
+  if (l.ff_pad != 0) {
+    p.w1 = l.w_down;
+    p.rows1 = plan.width_pad;
+    p.cols1 = l.ff_pad;
+  }
+  if (l.layer_scale) {
+    p.scale0 = l.ls_attn;
+    p.scale1 = l.ls_mlp;
+  }
+  return p;
+}
+// The two halves of an output launch, for shapes whose vectors do not fit one block together.
+ParallelProjectionParams first_matrix(ParallelProjectionParams p) {
+  p.w1 = nullptr;
+  p.rows1 = p.cols1 = 0;
+  return p;
+}
+ParallelProjectionParams second_matrix(ParallelProjectionParams p) {
+  p.w0 = p.w1;
+  p.rows0 = p.rows1;
+  p.cols0 = p.cols1;
+  p.x0 = p.x1;
+  p.scale0 = p.scale1;
+  p.step = nullptr;  // added by the first
+  return first_matrix(p);
+}
+WindowAttentionParams layer_attention(const ParallelPlan &plan, const ParallelLayerPlan &l, const ParallelRun &run) {
+  WindowAttentionParams p{};
+  p.s = l.shape;
+  p.qkv_stride = l.qkv_pad;
+  p.out_stride = l.attn_pad;
+  p.key_offset = run.key_offset;
+  p.value_offset = run.value_offset;
+  p.f32 = plan.f32 ? 1u : 0u;
+  return p;
+}
+
+cudaError_t block_gemm(Session *s, cudaStream_t stream, GemmParams g, uint32_t tokens) {
+  const BlockWorkspace &ws = s->weights->block_ws;
+  g.tokens = tokens;
+  g.workspace = ws.gemm_workspace;
+  g.error_word = s->device_error;
+  g.pdl = s->use_pdl ? 1u : 0u;
+  return launch_gemm_tc(stream, g, s->sm_count);
+}
+
+// Rows below which a block's attention is one query per thread block: a tile of the tensor-pipe kernel
+// would be mostly empty and walk its keys alone.
+constexpr uint32_t kPrefillTileMinRows = 8;
+
+}  // namespace
+
+std::shared_ptr<ParallelPlan> make_parallel_plan(const NervaB200ParallelModel &m, uint32_t width, uint32_t vocab, float eps) {
+  auto refuse = [](const char *why) {
+    set_last_error(std::string("parallel-block model not supported: ") + why);
+    return std::shared_ptr<ParallelPlan>();
+  };
+  auto plan = std::make_shared<ParallelPlan>();
+  if (m.compute != NERVA_DTYPE_BF16 && m.compute != NERVA_DTYPE_F32) return refuse("compute type");
+  plan->f32 = m.compute == NERVA_DTYPE_F32;
+  plan->width = width;
+  plan->width_pad = round_up(width, 64);
+  plan->vocab = vocab;
+  plan->embedding_scale = m.embedding_scale;
+  plan->softcap = m.logit_softcap;
+  plan->loop_times = m.loop_times;
+  if (m.loop_times != 0 && (m.loop_start >= m.loop_stop || m.loop_stop > m.layer_count)) return refuse("loop range");
+  for (uint32_t i = 0; i < m.layer_count; ++i) {
+    const NervaB200ParallelLayer &in = m.layers[i];
+    if (in.heads == 0 || in.kv_heads == 0 || in.heads % in.kv_heads != 0 || in.qk_dim == 0 || in.v_dim == 0 ||
+        in.qk_dim > 256u || in.v_dim > 256u)
+      return refuse("needs heads divisible by kv_heads and head sizes of 1 to 256");
+    if (in.rotary_dims % 2u != 0 || in.rotary_dims > in.qk_dim ||
+        (in.rotary_dims != 0 && !(in.rotary_base > 0.0 && in.rotary_base != 1.0)) ||
+        (in.yarn_factor != 0.0 && !(in.yarn_factor > 0.0 && in.yarn_original > 0.0 && in.yarn_fast > 0.0 && in.yarn_slow > 0.0)))
+      return refuse("rotation");
+    ParallelLayerPlan l;
+    WindowAttentionShape &a = l.shape;
+    a.heads = in.heads;
+    a.kv_heads = in.kv_heads;
+    a.qk_dim = in.qk_dim;
+    a.v_dim = in.v_dim;
+    a.qk_pad = round_up(in.qk_dim, 16);
+    a.v_pad = round_up(in.v_dim, 16);
+    a.window = in.window;
+    a.rotary_pairs = in.rotary_dims / 2u;
+    a.qk_norm = in.qk_norm;
+    a.scale = in.score_scale;
+    a.eps = eps;
+    rotary_table(in, &l.frequencies, &a.rotary_magnitude);
+    if (!window_attention_supported(a, plan->f32)) return refuse("attention shape");
+    l.intermediate = in.intermediate;
+    l.ff_pad = round_up(in.intermediate, 64);
+    l.qkv_rows = in.heads * in.qk_dim + in.kv_heads * (in.qk_dim + in.v_dim);
+    l.qkv_pad = round_up(l.qkv_rows, 64);
+    l.attn_width = in.heads * in.v_dim;
+    l.attn_pad = round_up(l.attn_width, 64);
+    l.layer_scale = in.layer_scale != 0;
+    plan->max_heads = std::max(plan->max_heads, in.heads);
+    plan->max_qkv_pad = std::max(plan->max_qkv_pad, l.qkv_pad);
+    plan->max_attn_pad = std::max(plan->max_attn_pad, l.attn_pad);
+    plan->max_ff_pad = std::max(plan->max_ff_pad, l.ff_pad);
+    plan->max_v_pad = std::max(plan->max_v_pad, a.v_pad);
+    plan->layers.push_back(l);
+  }
+  auto run = [&](uint32_t layer, int32_t step) {
+    ParallelRun r;
+    r.layer = layer;
+    r.step = step;
+    plan->runs.push_back(r);
+  };
+  const uint32_t start = m.loop_times != 0 ? m.loop_start : m.layer_count;
+  for (uint32_t i = 0; i < start; ++i) run(i, -1);
+  for (uint32_t t = 0; t < m.loop_times; ++t)
+    for (uint32_t i = start; i < m.loop_stop; ++i) run(i, i == start ? static_cast<int32_t>(t) : -1);
+  for (uint32_t i = m.loop_times != 0 ? m.loop_stop : start; i < m.layer_count; ++i) run(i, -1);
+  return plan;
+}
+
+void place_parallel_cache(ParallelPlan *plan, uint32_t pages) {
+  const uint64_t tokens = static_cast<uint64_t>(pages) * NERVA_KV_CACHE_BLOCK_TOKENS;
+  plan->key_elems = plan->value_elems = 0;
+  for (ParallelRun &r : plan->runs) {
+    const WindowAttentionShape &a = plan->layers[r.layer].shape;
+    r.key_offset = plan->key_elems;
+    r.value_offset = plan->value_elems;
+    plan->key_elems += tokens * a.kv_heads * a.qk_pad;
+    plan->value_elems += tokens * a.kv_heads * a.v_pad;
+  }
+}
+
+cudaError_t pack_parallel_weights(Session *s) {
+  const ParallelPlan &plan = *s->parallel;
+  const uint32_t width = plan.width, pad = plan.width_pad;
+  cudaError_t err = cudaSuccess;
+  auto clear = [&](void *p, uint64_t bytes) {
+    if (err == cudaSuccess && bytes != 0) err = cudaMemsetAsync(p, 0, bytes, s->stream);
+  };
+  auto pack = [&](uint64_t offset, uint32_t rows, uint32_t cols, uint16_t *dst, uint32_t dst_cols, uint32_t step,
+                  uint32_t first) {
+    if (err == cudaSuccess && rows != 0)
+      err = launch_pack_rows(s->stream, arena_at(s, offset), rows, cols, dst, dst_cols, step, first);
+  };
+  clear(plan.loop_vectors, static_cast<uint64_t>(std::max(plan.loop_times, 1u)) * pad * 2u);
+  pack(s->layout.loop_vectors, plan.loop_times, width, plan.loop_vectors, pad, 1, 0);
+  for (size_t i = 0; i < plan.layers.size(); ++i) {
+    const ParallelLayerPlan &l = plan.layers[i];
+    const LayerLayout &L = s->layout.layers[i];
+    const WindowAttentionShape &a = l.shape;
+    clear(l.w_in, (l.qkv_pad + 2ull * l.ff_pad) * pad * 2u);
+    clear(l.w_o, static_cast<uint64_t>(pad) * l.attn_pad * 2u);
+    clear(l.w_down, static_cast<uint64_t>(pad) * std::max(l.ff_pad, 8u) * 2u);
+    clear(l.norm, pad * 2u);
+    clear(l.ls_attn, pad * 2u);
+    clear(l.ls_mlp, pad * 2u);
+    const uint32_t q_rows = a.heads * a.qk_dim, k_rows = a.kv_heads * a.qk_dim, v_rows = a.kv_heads * a.v_dim;
+    pack(L.w_q, q_rows, width, l.w_in, pad, 1, 0);
+    pack(L.w_k, k_rows, width, l.w_in, pad, 1, q_rows);
+    pack(L.w_v, v_rows, width, l.w_in, pad, 1, q_rows + k_rows);
+    pack(L.w_o, width, l.attn_width, l.w_o, l.attn_pad, 1, 0);
+    pack(L.rms_attn, 1, width, l.norm, pad, 1, 0);
+    if (l.intermediate != 0) {
+      pack(L.w_gate, l.intermediate, width, l.w_in, pad, 2, l.qkv_pad);
+      pack(L.w_up, l.intermediate, width, l.w_in, pad, 2, l.qkv_pad + 1u);
+      pack(L.w_down, width, l.intermediate, l.w_down, l.ff_pad, 1, 0);
+    }
+    if (l.layer_scale) {
+      pack(L.ls_attn, 1, width, l.ls_attn, pad, 1, 0);
+      if (l.intermediate != 0) pack(L.ls_mlp, 1, width, l.ls_mlp, pad, 1, 0);
+    }
+    if (err == cudaSuccess && !l.frequencies.empty())
+      err = cudaMemcpyAsync(l.frequency, l.frequencies.data(), l.frequencies.size() * sizeof(float),
+                            cudaMemcpyHostToDevice, s->stream);
+    s->parallel->layers[i].shape.frequency = l.frequency;
+  }
+  clear(plan.final_norm, pad * 2u);
+  clear(plan.head, static_cast<uint64_t>(plan.vocab) * pad * 2u);
+  pack(s->layout.final_norm, 1, width, plan.final_norm, pad, 1, 0);
+  pack(s->layout.lm_head, plan.vocab, width, plan.head, pad, 1, 0);
+  return err;
+}
+
+uint32_t parallel_attention_splits(const ParallelPlan &plan, uint32_t target_context) {
+  uint32_t most = 1;
+  for (const ParallelLayerPlan &l : plan.layers)
+    most = std::max(most, window_attention_splits(target_context, l.shape.window));
+  return most;
+}
+
+cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launches, StepProfile *prof, ProfileMark mark) {
+  const ParallelPlan &plan = *s->parallel;
+  const uint32_t pdl = s->use_pdl ? 1u : 0u;
+  uint64_t n = 0;
+  cudaError_t err = cudaSuccess;
+  for (const ParallelRun &run : plan.runs) {
+    const ParallelLayerPlan &l = plan.layers[run.layer];
+    const uint16_t *step = step_vector(plan, run);
+    ParallelProjectionParams in = layer_in(plan, l, s->rms_eps);
+    in.pdl = pdl;
+    in.error_word = s->device_error;
+    in.h = s->h_b;
+    in.step = step;
+    in.out_f32 = s->qkv;
+    in.out_act = s->ff_bf16;
+    ParallelProjectionParams out = layer_out(plan, l);
+    out.pdl = pdl;
+    out.error_word = s->device_error;
+    out.h = out.h_out = s->h_b;
+    out.step = step;
+    out.x0 = s->attn_bf16;
+    out.x1 = s->ff_bf16;
+    const bool streamed = !plan.f32 && parallel_stream_eligible(kParallelIn, in, s->sm_count) &&
+                          parallel_stream_eligible(kParallelOut, first_matrix(out), s->sm_count) &&
+                          (out.rows1 == 0 || parallel_stream_eligible(kParallelOut, second_matrix(out), s->sm_count));
+    if (streamed) {
+      err = launch_parallel_projection(s->stream, kParallelIn, in, s->sm_count);
+      n += 1;
+    } else {
+      err = launch_stream_norm(s->stream, s->h_b, step, l.norm, s->rms_eps, plan.width, plan.width_pad, s->x_scratch,
+                               plan.f32, 1, nullptr, pdl != 0);
+      out.step = nullptr;  // it is part of the stream now
+      in.x0 = s->x_scratch;
+      if (err == cudaSuccess) err = launch_parallel_projection_plain(s->stream, kParallelIn, in, 1, plan.f32);
+      n += 2;
+    }
+    mark(s, prof, kBucketQkv);
+    if (err != cudaSuccess) break;
+
+    WindowAttentionParams a = layer_attention(plan, l, run);
+    a.pdl = pdl;
+    a.qkv = s->qkv;
+    a.out = s->attn_bf16;
+    a.splits = std::min(splits, window_attention_splits(UINT32_MAX / 2u, l.shape.window));
+    a.partial_acc = s->partial_acc;
+    a.partial_m = s->partial_m;
+    a.partial_l = s->partial_l;
+    a.tickets = s->attn_tickets;
+    a.cursor = s->device_cursor;
+    a.max_context = s->max_context;
+    a.page_count = s->kv_pages;
+    a.keys = s->kv_keys;
+    a.values = s->kv_values;
+    a.page_table = s->page_table;
+    a.error_word = s->device_error;
+    err = launch_window_attention(s->stream, a);
+    n += 1;
+    mark(s, prof, kBucketAttention);
+    if (err != cudaSuccess) break;
+
+    if (!streamed) {
+      err = launch_parallel_projection_plain(s->stream, kParallelOut, out, 1, plan.f32);
+      n += 1;
+    } else if (parallel_stream_eligible(kParallelOut, out, s->sm_count)) {
+      err = launch_parallel_projection(s->stream, kParallelOut, out, s->sm_count);
+      n += 1;
+    } else {
+      // both activation vectors do not fit beside the weight ring: one matrix after the other
+      err = launch_parallel_projection(s->stream, kParallelOut, first_matrix(out), s->sm_count);
+      if (err == cudaSuccess) err = launch_parallel_projection(s->stream, kParallelOut, second_matrix(out), s->sm_count);
+      n += 2;
+    }
+    mark(s, prof, kBucketDown);
+    if (err != cudaSuccess) break;
+  }
+  if (launches != nullptr) *launches += n;
+  return err;
+}
+
+cudaError_t enqueue_parallel_head(Session *s, uint32_t *partials, uint64_t *launches) {
+  const ParallelPlan &plan = *s->parallel;
+  ParallelProjectionParams p{};
+  p.w0 = plan.head;
+  p.rows0 = plan.vocab;
+  p.cols0 = plan.width_pad;
+  p.h = s->h_b;
+  p.norm = plan.final_norm;
+  p.width = plan.width;
+  p.eps = s->rms_eps;
+  p.out_f32 = s->logits;
+  p.softcap = plan.softcap;
+  p.best_value = s->best_value;
+  p.best_index = s->best_index;
+  p.error_word = s->device_error;
+  p.pdl = s->use_pdl ? 1u : 0u;
+  if (!plan.f32 && parallel_stream_eligible(kParallelHead, p, s->sm_count)) {
+    *partials = parallel_stream_blocks(kParallelHead, p, s->sm_count);
+    if (launches != nullptr) *launches += 1;
+    return launch_parallel_projection(s->stream, kParallelHead, p, s->sm_count);
+  }
+  cudaError_t err = launch_stream_norm(s->stream, s->h_b, nullptr, plan.final_norm, s->rms_eps, plan.width,
+                                       plan.width_pad, s->x_scratch, plan.f32, 1, nullptr, p.pdl != 0);
+  p.x0 = s->x_scratch;
+  if (err == cudaSuccess) err = launch_parallel_projection_plain(s->stream, kParallelHead, p, 1, plan.f32);
+  *partials = std::min(kBlockArgmaxChunks, s->sm_count);
+  if (err == cudaSuccess)
+    err = launch_argmax_partials(s->stream, s->logits, plan.vocab, 1, *partials, s->best_value, s->best_index, p.pdl != 0);
+  if (launches != nullptr) *launches += 3;
+  return err;
+}
+
+cudaError_t enqueue_parallel_block_layers(Session *s, const ParallelBlock &b, uint64_t *launches) {
+  const ParallelPlan &plan = *s->parallel;
+  const BlockWorkspace &ws = s->weights->block_ws;
+  const uint32_t pdl = s->use_pdl ? 1u : 0u;
+  uint64_t n = 0;
+  cudaError_t err = cudaSuccess;
+  for (size_t index = 0; err == cudaSuccess && index < plan.runs.size(); ++index) {
+    const ParallelRun &run = plan.runs[index];
+    const ParallelLayerPlan &l = plan.layers[run.layer];
+    err = launch_stream_norm(b.stream, ws.h_b, step_vector(plan, run), l.norm, s->rms_eps, plan.width, plan.width_pad,
+                             ws.x_bf16, plan.f32, b.rows, nullptr, pdl != 0);
+    ParallelProjectionParams in = layer_in(plan, l, s->rms_eps);
+    if (err == cudaSuccess && plan.f32) {
+      in.x0 = ws.x_bf16;
+      in.out_f32 = ws.qkv;
+      in.out_act = ws.ff;
+      in.pdl = pdl;
+      err = launch_parallel_projection_plain(b.stream, kParallelIn, in, b.rows, true);
+    } else if (err == cudaSuccess) {
+      GemmParams g{};
+      g.weight = l.w_in;
+      g.rows = l.qkv_pad + 2u * l.ff_pad;
+      g.cols = plan.width_pad;
+      g.x = ws.x_bf16;
+      g.epilogue = l.ff_pad != 0 ? kEpilogueStoreSwiglu : kEpilogueStore;
+      g.split_row = l.qkv_pad;
+      g.out_f32 = ws.qkv;
+      g.out_bf16 = ws.ff;
+      err = block_gemm(s, b.stream, g, b.rows);
+    }
+
+    WindowAttentionParams a = layer_attention(plan, l, run);
+    a.pdl = pdl;
+    a.qkv = ws.qkv;
+    a.out = ws.attn;
+    a.partial_acc = ws.partial_acc;
+    a.partial_m = ws.partial_m;
+    a.partial_l = ws.partial_l;
+    a.tickets = ws.attn_tickets;
+    a.rows = ws.attn_rows;
+    a.row_count = b.rows;
+    if (err == cudaSuccess) err = launch_window_publish(b.stream, a);
+    if (err == cudaSuccess) {
+      if (b.one_session && b.rows >= kPrefillTileMinRows && !plan.f32) {
+        err = launch_window_prefill(b.stream, a);
+      } else {
+        // rows x KV heads fill the machine already: as few spans as keep about four blocks per SM
+        const uint32_t machine = 4u * s->sm_count / (b.rows * l.shape.kv_heads);
+        a.splits = std::min(window_attention_splits(b.longest, l.shape.window), std::max(machine, 1u));
+        err = launch_window_attention(b.stream, a);
+      }
+    }
+
+    ParallelProjectionParams out = layer_out(plan, l);
+    if (err == cudaSuccess && plan.f32) {
+      out.h = out.h_out = ws.h_b;
+      out.x0 = ws.attn;
+      out.x1 = ws.ff;
+      out.pdl = pdl;
+      err = launch_parallel_projection_plain(b.stream, kParallelOut, out, b.rows, true);
+      n += 5;
+    } else if (err == cudaSuccess) {
+      GemmParams g{};
+      g.rows = plan.width_pad;
+      g.epilogue = kEpilogueStore;
+      g.resid_in = g.out_f32 = ws.h_b;
+      g.weight = out.w0;
+      g.cols = out.cols0;
+      g.x = ws.attn;
+      g.row_scale = out.scale0;
+      err = block_gemm(s, b.stream, g, b.rows);
+      if (err == cudaSuccess && l.ff_pad != 0) {
+        g.weight = out.w1;
+        g.cols = out.cols1;
+        g.x = ws.ff;
+        g.row_scale = out.scale1;
+        err = block_gemm(s, b.stream, g, b.rows);
+      }
+      n += l.ff_pad != 0 ? 6 : 5;
+    }
+    if (err == cudaSuccess && s->capture_stream != nullptr && b.one_session && b.capture_row < s->capture_rows) {
+      const uint32_t rows = std::min(b.rows, s->capture_rows - b.capture_row);
+      err = cudaMemcpy2DAsync(s->capture_stream + (index * s->capture_rows + b.capture_row) * plan.width,
+                              plan.width * sizeof(float), ws.h_b, plan.width_pad * sizeof(float),
+                              plan.width * sizeof(float), rows, cudaMemcpyDeviceToHost, b.stream);
+    }
+  }
+  if (launches != nullptr) *launches += n;
+  return err;
+}
+
+cudaError_t enqueue_parallel_block_head(Session *s, cudaStream_t stream, uint32_t count, const uint32_t *row_index,
+                                        uint64_t *launches) {
+  const ParallelPlan &plan = *s->parallel;
+  const BlockWorkspace &ws = s->weights->block_ws;
+  cudaError_t err = launch_stream_norm(stream, ws.h_b, nullptr, plan.final_norm, s->rms_eps, plan.width, plan.width_pad,
+                                       ws.x_bf16, plan.f32, count, row_index, s->use_pdl);
+  if (err == cudaSuccess && plan.f32) {
+    ParallelProjectionParams p{};
+    p.w0 = plan.head;
+    p.rows0 = plan.vocab;
+    p.cols0 = plan.width_pad;
+    p.x0 = ws.x_bf16;
+    p.out_f32 = ws.logits;
+    p.softcap = plan.softcap;
+    p.pdl = s->use_pdl ? 1u : 0u;
+    err = launch_parallel_projection_plain(stream, kParallelHead, p, count, true);
+  } else if (err == cudaSuccess) {
+    GemmParams g{};
+    g.weight = plan.head;
+    g.rows = plan.vocab;
+    g.cols = plan.width_pad;
+    g.x = ws.x_bf16;
+    g.epilogue = kEpilogueStore;
+    g.softcap = plan.softcap;
+    g.out_f32 = ws.logits;
+    err = block_gemm(s, stream, g, count);
+  }
+  if (launches != nullptr) *launches += 2;
+  return err;
+}
+
+}  // namespace nb

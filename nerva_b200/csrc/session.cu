@@ -112,7 +112,8 @@ static uint64_t push_optional(uint64_t &cursor, uint64_t len, const void *ptr) {
 
 // hf_decode_sequence/weights.cu:487-591 (full-attention layers) and
 // session_api_lifecycle.inc.cu:124-146 (arena order).
-ArenaLayout compute_arena_layout(const ModelDims &d, const NervaCudaHfDecodeChainLayer *layers) {
+ArenaLayout compute_arena_layout(const ModelDims &d, const NervaCudaHfDecodeChainLayer *layers,
+                                 const NervaB200ParallelModel *parallel) {
   ArenaLayout out;
   const uint64_t hidden = d.hidden, ah = d.attention_hidden(), kvh = d.kv_hidden();
   const uint64_t inter = d.intermediate;
@@ -121,6 +122,33 @@ ArenaLayout compute_arena_layout(const ModelDims &d, const NervaCudaHfDecodeChai
   out.input = push(c, hidden);
   out.scratch = push(c, hidden);
   out.layers.resize(d.layers);
+  if (parallel != nullptr) {
+    if (parallel->loop_times != 0) out.loop_vectors = push(c, static_cast<uint64_t>(parallel->loop_times) * hidden);
+    for (uint32_t i = 0; i < d.layers; ++i) {
+      const NervaB200ParallelLayer &layer = parallel->layers[i];
+      LayerLayout &l = out.layers[i];
+      const uint64_t q = static_cast<uint64_t>(layer.heads) * layer.qk_dim, k = static_cast<uint64_t>(layer.kv_heads) * layer.qk_dim;
+      const uint64_t v = static_cast<uint64_t>(layer.kv_heads) * layer.v_dim, a = static_cast<uint64_t>(layer.heads) * layer.v_dim;
+      l.rms_attn = push(c, hidden);
+      l.w_q = push(c, q * hidden);
+      l.w_k = push(c, k * hidden);
+      l.w_v = push(c, v * hidden);
+      l.w_o = push(c, hidden * a);
+      if (layer.intermediate != 0) {
+        l.w_gate = push(c, layer.intermediate * hidden);
+        l.w_up = push(c, layer.intermediate * hidden);
+        l.w_down = push(c, hidden * layer.intermediate);
+      }
+      if (layer.layer_scale != 0) {
+        l.ls_attn = push(c, hidden);
+        if (layer.intermediate != 0) l.ls_mlp = push(c, hidden);
+      }
+    }
+    out.final_norm = push(c, hidden);
+    out.lm_head = push(c, static_cast<uint64_t>(d.vocab) * hidden);
+    out.elements = c;
+    return out;
+  }
   for (uint32_t i = 0; i < d.layers; ++i) {
     const NervaCudaHfDecodeChainLayer &layer = layers[i];
     LayerLayout &l = out.layers[i];
@@ -262,6 +290,24 @@ bool plan_weights(Session *s, StaticArena &arena, void *base, SharedWeights *w) 
   for (int32_t ordinal : s->dense_ordinal) dense_layers += ordinal >= 0 ? 1u : 0u;
   uint16_t *arena_ptr = nullptr, *qkv = nullptr, *gu = nullptr;
   bool ok = carve(arena, base, s->layout.elements, &arena_ptr);
+  if (s->parallel) {
+    if (ok && w != nullptr) w->arena = arena_ptr;
+    ParallelPlan &plan = *s->parallel;
+    const uint64_t width = plan.width_pad;
+    ok = ok && carve(arena, base, std::max<uint64_t>(plan.loop_times, 1u) * width, &plan.loop_vectors);
+    for (ParallelLayerPlan &l : plan.layers) {
+      ok = ok && carve(arena, base, (l.qkv_pad + 2ull * l.ff_pad) * width, &l.w_in);
+      ok = ok && carve(arena, base, width * l.attn_pad, &l.w_o);
+      ok = ok && carve(arena, base, width * std::max(l.ff_pad, 8u), &l.w_down);
+      ok = ok && carve(arena, base, width, &l.norm);
+      ok = ok && carve(arena, base, width, &l.ls_attn);
+      ok = ok && carve(arena, base, width, &l.ls_mlp);
+      ok = ok && carve(arena, base, static_cast<uint64_t>(l.shape.rotary_pairs) + 1u, &l.frequency);
+    }
+    ok = ok && carve(arena, base, width, &plan.final_norm);
+    ok = ok && carve(arena, base, plan.vocab * width, &plan.head);
+    return ok;
+  }
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.layers) * qkv_rows * d.hidden, &qkv);
   ok = ok && carve(arena, base, std::max<uint64_t>(dense_layers, 1u) * 2u * d.intermediate * d.hidden, &gu);
   if (ok && w != nullptr) {
@@ -280,13 +326,32 @@ bool plan_state(Session *s, StaticArena &arena, void *base) {
   // latent attention caches one row of (rank + rope) values per token in the K array; the V array is not used
   s->kv_layer_elems = static_cast<uint64_t>(s->kv_pages) * NERVA_KV_CACHE_BLOCK_TOKENS * d.kv_row();
   s->max_splits = attention_default_splits(s->max_context, 1, d.kv_heads, s->sm_count);
-  const uint64_t max_x = std::max<uint64_t>(std::max<uint64_t>(d.hidden, d.intermediate), ah);
-  bool ok = carve(arena, base, d.layers * s->kv_layer_elems, &s->kv_keys);
-  ok = ok && carve(arena, base, d.mla() ? uint64_t{16} : d.layers * s->kv_layer_elems, &s->kv_values);
+  uint64_t max_x = std::max<uint64_t>(std::max<uint64_t>(d.hidden, d.intermediate), ah);
+  uint64_t hidden = d.hidden, qkv = std::max<uint64_t>(ah + 2 * kvh, d.qkv_rows()), attn = ah, ff = d.intermediate;
+  uint64_t keys = d.layers * s->kv_layer_elems, values = d.mla() ? uint64_t{16} : d.layers * s->kv_layer_elems;
+  uint64_t partial_dim = std::max(d.head_dim, d.mla_rank);
+  if (s->parallel) {
+    // 16-bit elements throughout; an fp32 session takes two per value
+    ParallelPlan &plan = *s->parallel;
+    place_parallel_cache(&plan, s->kv_pages);
+    const uint64_t words = plan.element_bytes() / 2u;
+    keys = plan.key_elems * words;
+    values = plan.value_elems * words;
+    hidden = plan.width_pad;
+    qkv = plan.max_qkv_pad;
+    attn = plan.max_attn_pad * words;
+    ff = std::max<uint64_t>(plan.max_ff_pad, 8u) * words;
+    max_x = plan.width_pad * words;
+    partial_dim = plan.max_v_pad;
+    s->kv_layer_elems = 0;
+    s->max_splits = kWindowMaxSplits;
+  }
+  bool ok = carve(arena, base, keys, &s->kv_keys);
+  ok = ok && carve(arena, base, values, &s->kv_values);
   ok = ok && carve(arena, base, static_cast<uint64_t>(s->kv_pages), &s->page_table);
-  ok = ok && carve(arena, base, static_cast<uint64_t>(d.hidden), &s->h_a);
-  ok = ok && carve(arena, base, static_cast<uint64_t>(d.hidden), &s->h_b);
-  ok = ok && carve(arena, base, std::max<uint64_t>(ah + 2 * kvh, d.qkv_rows()), &s->qkv);
+  ok = ok && carve(arena, base, hidden, &s->h_a);
+  ok = ok && carve(arena, base, hidden, &s->h_b);
+  ok = ok && carve(arena, base, qkv, &s->qkv);
   ok = ok && carve(arena, base, std::max<uint64_t>(static_cast<uint64_t>(d.heads) * d.mla_rank, 4u), &s->mla_ql);
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.hidden), &s->o_out);
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.hidden), &s->down);
@@ -295,16 +360,15 @@ bool plan_state(Session *s, StaticArena &arena, void *base) {
   const uint64_t split_slots = std::max<uint32_t>(s->max_splits, d.mla() ? 64u : 16u);
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.heads), &s->attn_tickets);
   s->x_elems = static_cast<uint32_t>(max_x);
-  ok = ok && carve(arena, base, static_cast<uint64_t>(d.heads) * split_slots * std::max(d.head_dim, d.mla_rank),
-                   &s->partial_acc);
+  ok = ok && carve(arena, base, static_cast<uint64_t>(d.heads) * split_slots * partial_dim, &s->partial_acc);
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.heads) * split_slots, &s->partial_m);
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.heads) * split_slots, &s->partial_l);
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.layers), &s->step_layers);
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.layers) * 4u + 1u, &s->step_jobs);
   ok = ok && carve(arena, base, uint64_t{4}, &s->barrier_counter);
   ok = ok && carve(arena, base, static_cast<uint64_t>(kPhaseCount), &s->phase_cycles);
-  ok = ok && carve(arena, base, ah, &s->attn_bf16);
-  ok = ok && carve(arena, base, static_cast<uint64_t>(d.intermediate), &s->ff_bf16);
+  ok = ok && carve(arena, base, attn, &s->attn_bf16);
+  ok = ok && carve(arena, base, ff, &s->ff_bf16);
   ok = ok && carve(arena, base, max_x, &s->x_scratch);
   ok = ok && carve(arena, base, static_cast<uint64_t>(s->sm_count), &s->best_value);
   ok = ok && carve(arena, base, static_cast<uint64_t>(s->sm_count), &s->best_index);
@@ -424,7 +488,7 @@ cudaError_t setup_step_kernel(Session *s) {
                                    max_rows_per_block(2u * d.intermediate, 2, s->sm_count)),
                           std::max(max_rows_per_block(d.hidden, 1, s->sm_count),
                                    max_rows_per_block(d.vocab, 1, s->sm_count)));
-  s->step_kernel_ok = !s->has_moe && !d.mla() && step_kernel_supported(d.hidden, d.heads, d.kv_heads, d.head_dim,
+  s->step_kernel_ok = !s->has_moe && !d.mla() && !s->parallel && step_kernel_supported(d.hidden, d.heads, d.kv_heads, d.head_dim,
                                                            d.intermediate, s->x_elems, s->row_elems);
   if (!s->step_kernel_ok) return cudaSuccess;
   cudaError_t err = configure_step_kernel();
@@ -598,11 +662,16 @@ cudaError_t enqueue_step(Session *s, uint32_t splits, uint32_t sample, uint64_t 
   profile_mark(s, prof, kBucketEmbed);
   cudaError_t err = cudaSuccess;
   if (!head_only) {
-    err = launch_embed(s->stream, st, arena_at(s, s->layout.embeddings), d.hidden, s->h_b);
+    if (s->parallel)
+      err = launch_embed(s->stream, st, arena_at(s, s->layout.embeddings), d.hidden, s->h_b, s->parallel->embedding_scale,
+                         s->parallel->width_pad);
+    else
+      err = launch_embed(s->stream, st, arena_at(s, s->layout.embeddings), d.hidden, s->h_b);
     n += 1;
   }
   profile_mark(s, prof, kBucketEmbed);
-  for (uint32_t l = 0; !head_only && err == cudaSuccess && l < d.layers; ++l) {
+  if (s->parallel && !head_only && err == cudaSuccess) err = enqueue_parallel_layers(s, splits, &n, prof, profile_mark);
+  for (uint32_t l = 0; !s->parallel && !head_only && err == cudaSuccess && l < d.layers; ++l) {
     const LayerLayout &L = s->layout.layers[l];
     ProjectionParams p{};
     p.error_word = s->device_error;
@@ -855,7 +924,10 @@ cudaError_t enqueue_step(Session *s, uint32_t splits, uint32_t sample, uint64_t 
     profile_mark(s, prof, kBucketDown);
   }
   uint32_t partials = 0;
-  if (err == cudaSuccess && sample != 0) {
+  if (s->parallel && err == cudaSuccess && sample != 0) {
+    err = enqueue_parallel_head(s, &partials, &n);
+    profile_mark(s, prof, kBucketLmHead);
+  } else if (err == cudaSuccess && sample != 0) {
     ProjectionParams p{};
     p.error_word = s->device_error;
     p.pdl = s->use_pdl ? 1u : 0u;
@@ -1008,6 +1080,7 @@ bool peer_failure_seen(Session *s, uint32_t step) {
 
 uint32_t splits_for(Session *s, uint32_t target_context) {
   if (s->engine == 1) return step_kernel_splits(target_context);
+  if (s->parallel) return parallel_attention_splits(*s->parallel, target_context);
   if (s->dims.mla()) return mla_attention_splits(target_context);
   if (s->fused_attention) return fused_attention_splits(target_context);
   uint32_t want = attention_default_splits(target_context, 1, s->dims.kv_heads, s->sm_count);
@@ -1042,6 +1115,7 @@ void fill_header(const Session *s, NervaCudaHfDecodeSequenceResult *out, uint32_
 }
 
 uint64_t resident_kv_bytes(const Session *s) {
+  if (s->parallel) return (s->parallel->key_elems + s->parallel->value_elems) * s->parallel->element_bytes();
   return (s->dims.mla() ? 1ull : 2ull) * s->dims.layers * s->kv_layer_elems * sizeof(uint16_t);
 }
 uint64_t device_footprint(const Session *s) {
@@ -1406,8 +1480,12 @@ cudaError_t allocate_state(Session *s, int32_t *stage) {
   // KV pages come out of the pool in FIFO order, which makes the initial
   // logical->physical table the identity, as the reference initialises it
   // (hf_decode_sequence/kernels.cu:732-739).
-  StaticArena page_space(2ull * s->dims.layers * s->kv_layer_elems * 2u + 64u);
-  const uint64_t page_bytes = NERVA_KV_CACHE_BLOCK_TOKENS * s->dims.kv_row() * 2u;
+  // A page of a parallel-block session is 16 tokens of every layer run, K and V together.
+  const uint64_t page_bytes = s->parallel ? (s->parallel->key_elems + s->parallel->value_elems) / s->kv_pages *
+                                                s->parallel->element_bytes()
+                                          : NERVA_KV_CACHE_BLOCK_TOKENS * s->dims.kv_row() * 2u;
+  StaticArena page_space(s->parallel ? page_bytes * s->kv_pages + 64u
+                                     : 2ull * s->dims.layers * s->kv_layer_elems * 2u + 64u);
   if (!s->kv_pool.preallocate(page_space, s->kv_pages, NERVA_KV_CACHE_BLOCK_TOKENS, page_bytes, 16))
     return cudaErrorMemoryAllocation;
   std::vector<uint32_t> table(s->kv_pages);
@@ -1423,8 +1501,15 @@ cudaError_t allocate_state(Session *s, int32_t *stage) {
   if (err == cudaSuccess)
     err = cudaMemsetAsync(s->attn_tickets, 0, s->dims.heads * sizeof(uint32_t), s->stream);
   if (err == cudaSuccess) err = cudaMemsetAsync(s->moe_ticket, 0, 4 * sizeof(uint32_t), s->stream);
-  s->fused_attention = !s->dims.mla() && fused_attention_supported(s->dims.heads, s->dims.kv_heads, s->dims.head_dim);
-  if (!s->dims.mla() && attention_rows_supported(s->dims.heads, s->dims.kv_heads, s->dims.head_dim)) {
+  if (s->parallel && err == cudaSuccess) {
+    // the padding behind a layer's activations multiplies zero weights, so it only has to be finite
+    const uint64_t bytes = s->parallel->element_bytes();
+    err = cudaMemsetAsync(s->attn_bf16, 0, s->parallel->max_attn_pad * bytes, s->stream);
+    if (err == cudaSuccess)
+      err = cudaMemsetAsync(s->ff_bf16, 0, std::max(s->parallel->max_ff_pad, 8u) * bytes, s->stream);
+  }
+  s->fused_attention = !s->dims.mla() && !s->parallel && fused_attention_supported(s->dims.heads, s->dims.kv_heads, s->dims.head_dim);
+  if (!s->dims.mla() && !s->parallel && attention_rows_supported(s->dims.heads, s->dims.kv_heads, s->dims.head_dim)) {
     const uint64_t rows = static_cast<uint64_t>(s->dims.layers) * s->kv_pages * NERVA_KV_CACHE_BLOCK_TOKENS;
     s->kv_maps = encode_bf16_map_2d(&s->kv_map_k, s->kv_keys, s->dims.kv_hidden(), rows, 64, NERVA_KV_CACHE_BLOCK_TOKENS) &&
                  encode_bf16_map_2d(&s->kv_map_v, s->kv_values, s->dims.kv_hidden(), rows, 64, NERVA_KV_CACHE_BLOCK_TOKENS);
@@ -1442,7 +1527,7 @@ cudaError_t allocate_state(Session *s, int32_t *stage) {
 }  // namespace
 
 static int create_session(const NervaCudaHfDecodeSequenceSessionCreateRequest *request,
-                          const NervaB200ShardInfo *shard,
+                          const NervaB200ShardInfo *shard, const NervaB200ParallelModel *parallel,
                           NervaCudaHfDecodeSequenceSessionCreateResult *out,
                           NervaCudaHfDecodeSequenceSession **session_out) {
   if (out == nullptr) return -1;
@@ -1557,7 +1642,19 @@ static int create_session(const NervaCudaHfDecodeSequenceSessionCreateRequest *r
     out->failure_stage = kStageInvalidRequest;
     return -1;
   }
-  ArenaLayout layout = compute_arena_layout(d, request->layers);
+  std::shared_ptr<ParallelPlan> plan;
+  if (parallel != nullptr) {
+    bool ok = declared_plan && mla_layers == 0 && parallel->layers != nullptr && parallel->layer_count == request->layer_count;
+    for (uint32_t i = 0; ok && i < request->layer_count; ++i)
+      ok = request->layers[i].attention_kind == NERVA_ATTENTION_KIND_FULL &&
+           request->layers[i].mlp_kind == NERVA_MLP_KIND_DENSE && parallel->layers[i].heads <= request->heads;
+    if (ok) plan = make_parallel_plan(*parallel, d.hidden, d.vocab, request->rms_eps);
+    if (!plan) {
+      out->failure_stage = kStageInvalidRequest;
+      return -1;
+    }
+  }
+  ArenaLayout layout = compute_arena_layout(d, request->layers, parallel);
   const uint64_t resident_weight_bytes = layout.elements * 2u - static_cast<uint64_t>(d.hidden) * 4u;
   out->resident_weight_bytes = resident_weight_bytes;
   if (declared_plan && (request->planned_weight_bytes != resident_weight_bytes ||
@@ -1602,6 +1699,7 @@ static int create_session(const NervaCudaHfDecodeSequenceSessionCreateRequest *r
   s->rope_theta = request->rope_theta;
   s->detailed_profile = request->detailed_profile;
   s->layout = layout;
+  s->parallel = plan;
   s->resident_weight_bytes = resident_weight_bytes;
   s->planned_weight_blocks = request->planned_weight_blocks;
   s->planned_gpu_resident_blocks = request->planned_gpu_resident_blocks;
@@ -1637,6 +1735,8 @@ static int create_session(const NervaCudaHfDecodeSequenceSessionCreateRequest *r
   if (err == cudaSuccess) err = configure_fused_attention_kernel();
   if (err == cudaSuccess) err = configure_moe_kernels();
   if (err == cudaSuccess) err = configure_mla_kernels();
+  if (err == cudaSuccess && s->parallel) err = configure_parallel_projection();
+  if (err == cudaSuccess && s->parallel) err = configure_window_attention();
   if (err != cudaSuccess) return create_fail(s, out, err, kStageSetDevice);
   if (d.mla() && !mla_session_supported(d.heads, d.mla_rank, d.mla_nope, d.mla_rope, d.head_dim)) {
     set_last_error("latent attention shape not supported: needs at most 16 heads, latent rank 128, 256 or 512, "
@@ -1684,7 +1784,8 @@ static int create_session(const NervaCudaHfDecodeSequenceSessionCreateRequest *r
   // packed replicas
   const uint64_t ah = d.attention_hidden(), kvh = d.kv_hidden();
   const uint64_t qkv_rows = d.qkv_rows();
-  for (uint32_t l = 0; err == cudaSuccess && l < d.layers; ++l) {
+  if (s->parallel) err = pack_parallel_weights(s);
+  for (uint32_t l = 0; err == cudaSuccess && !s->parallel && l < d.layers; ++l) {
     const LayerLayout &L = s->layout.layers[l];
     uint16_t *packed = s->weights->qkv_packed + l * qkv_rows * d.hidden;
     if (d.mla()) {
@@ -1727,7 +1828,21 @@ extern "C" int nerva_cuda_hf_decode_sequence_session_create(
     const NervaCudaHfDecodeSequenceSessionCreateRequest *request,
     NervaCudaHfDecodeSequenceSessionCreateResult *out,
     NervaCudaHfDecodeSequenceSession **session_out) {
-  return create_session(request, nullptr, out, session_out);
+  return create_session(request, nullptr, nullptr, out, session_out);
+}
+
+extern "C" int nerva_b200_session_create_parallel(
+    const NervaCudaHfDecodeSequenceSessionCreateRequest *request, const NervaB200ParallelModel *model,
+    NervaCudaHfDecodeSequenceSessionCreateResult *out, NervaCudaHfDecodeSequenceSession **session_out) {
+  if (model == nullptr) {
+    if (out != nullptr) {
+      memset(out, 0, sizeof(*out));
+      out->status = -1;
+      out->failure_stage = kStageInvalidRequest;
+    }
+    return -1;
+  }
+  return create_session(request, nullptr, model, out, session_out);
 }
 
 extern "C" int nerva_b200_session_create_sharded(
@@ -1741,7 +1856,7 @@ extern "C" int nerva_b200_session_create_sharded(
     }
     return -1;
   }
-  return create_session(request, shard, out, session_out);
+  return create_session(request, shard, nullptr, out, session_out);
 }
 
 // The 64-byte inter-process handle of this rank's exchange buffer.
@@ -1880,7 +1995,7 @@ extern "C" int nerva_cuda_hf_decode_sequence_session_start(
     // last position (session_decode_prefill.inc.cu:1879-2245 is the reference's counterpart).
     if (err == cudaSuccess) err = cudaEventRecord(s->ev_start, s->stream);
     uint64_t launches = 0;
-    if (err == cudaSuccess) err = enqueue_chunked_prefill(s, s->prompt_count, s->sample_kind, &launches);
+    if (err == cudaSuccess) err = enqueue_chunked_prefill(s, 0, s->prompt_count, WantedLogits{}, &launches);
     const uint32_t last = s->prompt_count - 1u;
     if (err == cudaSuccess)  // the head samples at the cursor: the last prompt position
       err = cudaMemcpyAsync(s->device_cursor, &last, sizeof(uint32_t), cudaMemcpyHostToDevice, s->stream);
@@ -2064,7 +2179,7 @@ extern "C" int nerva_cuda_hf_decode_sequence_session_run(
     // The prompt goes through the chunked prefill, exactly as session_start runs it, so that
     // run == start + advance bit for bit; the decode steps follow.
     uint64_t launches = 0, head_launches = 0;
-    if (err == cudaSuccess) err = enqueue_chunked_prefill(s, s->prompt_count, s->sample_kind, &launches);
+    if (err == cudaSuccess) err = enqueue_chunked_prefill(s, 0, s->prompt_count, WantedLogits{}, &launches);
     const uint32_t last = s->prompt_count - 1u;
     if (err == cudaSuccess)
       err = cudaMemcpyAsync(s->device_cursor, &last, sizeof(uint32_t), cudaMemcpyHostToDevice, s->stream);
@@ -2153,9 +2268,8 @@ extern "C" int nerva_cuda_hf_decode_sequence_batch_advance_one(
       return false;
     // dense full-attention models whose heads span the hidden size (session_common.inc.cu:1078-1090),
     // on the per-kernel engine of one GPU
-    if (s->dims.hidden < 128 || s->dims.heads * s->dims.head_dim != s->dims.hidden || s->has_moe ||
-        s->tp_world > 1 || s->engine != 0)
-      return false;
+    if (s->has_moe || s->tp_world > 1 || s->engine != 0) return false;
+    if (!s->parallel && (s->dims.hidden < 128 || s->dims.heads * s->dims.head_dim != s->dims.hidden)) return false;
     return s->prompt_count + s->observed == s->cursor + 1u;
   };
   auto same_model = [](const Session *a, const Session *b) {
@@ -2341,6 +2455,7 @@ extern "C" int nerva_cuda_hf_decode_sequence_session_fork_shared_weights(
   s->layout = parent->layout;
   s->layer_meta = parent->layer_meta;
   s->has_moe = parent->has_moe;
+  s->parallel = parent->parallel;
   s->dense_ordinal = parent->dense_ordinal;
   s->resident_weight_bytes = parent->resident_weight_bytes;
   s->planned_weight_blocks = parent->planned_weight_blocks;
@@ -2396,6 +2511,87 @@ extern "C" int nerva_cuda_hf_decode_sequence_session_fork_shared_weights(
   out->sync_calls = 2;
   out->status = 0;
   *session_out = s;
+  return 0;
+}
+
+// Given tokens after what the session has run.  The prompt array holds them at their positions (the
+// kernels take a position's token from it when the position is below the prompt count), so the
+// generation path needs nothing new: start is the same work from position 0.
+extern "C" int nerva_b200_session_append(Session *s, const uint32_t *tokens, uint32_t count, uint32_t reset,
+                                         const uint32_t *want, uint32_t want_count, float *logits) {
+  if (s == nullptr || tokens == nullptr || count == 0 || (want_count != 0 && (want == nullptr || logits == nullptr)) ||
+      s->tp_world > 1)
+    return -1;
+  const bool fresh = reset != 0 || !s->started;
+  const uint32_t begin = fresh ? 0u : s->cursor;
+  set_last_error("");
+  if (begin >= s->max_context || count > s->max_context - begin) {
+    set_last_error("the tokens do not fit the session's context");
+    return -1;
+  }
+  for (uint32_t i = 0; i < count; ++i) {
+    if (tokens[i] >= s->dims.embed_vocab) {
+      set_last_error("token id out of range");
+      return -1;
+    }
+  }
+  for (uint32_t i = 0; i < want_count; ++i) {
+    if (want[i] >= count) return -1;
+  }
+  const uint32_t end = begin + count;
+  NervaCudaHfDecodeSequenceResult counters{};
+  cudaError_t err;
+  if (fresh) {
+    s->has_eos = 0;
+    err = reset_request_state(s, tokens, count, &counters);
+  } else {
+    err = cudaMemcpyAsync(s->device_prompt + begin, tokens, static_cast<uint64_t>(count) * sizeof(uint32_t),
+                          cudaMemcpyHostToDevice, s->stream);
+    if (err == cudaSuccess)  // pageable source: staged before the call returns
+      err = cudaMemcpyAsync(s->device_cursor + 1, &end, sizeof(uint32_t), cudaMemcpyHostToDevice, s->stream);
+  }
+  s->started = false;
+  s->prompt_count = end;
+  if (s->weights->block_ws.block != nullptr && s->engine == 0 && count > 1) {
+    const WantedLogits wanted{want, want_count, logits};
+    if (err == cudaSuccess) err = enqueue_chunked_prefill(s, begin, end, wanted, nullptr);
+    const uint32_t last = end - 1u;
+    if (err == cudaSuccess)
+      err = cudaMemcpyAsync(s->device_cursor, &last, sizeof(uint32_t), cudaMemcpyHostToDevice, s->stream);
+    if (err == cudaSuccess) err = enqueue_step(s, splits_for(s, end), s->sample_kind, nullptr, nullptr, true);
+  } else {
+    for (uint32_t i = 0; err == cudaSuccess && i < count; ++i) {
+      bool sampled = i + 1u == count;
+      for (uint32_t k = 0; k < want_count; ++k) sampled = sampled || want[k] == i;
+      GraphEntry *graph = nullptr;
+      err = ensure_graph(s, splits_for(s, begin + i + 1u), sampled ? s->sample_kind : 0u, &graph, nullptr);
+      if (err == cudaSuccess) err = replay(s, graph);
+      for (uint32_t k = 0; err == cudaSuccess && k < want_count; ++k) {
+        if (want[k] == i)
+          err = cudaMemcpyAsync(logits + static_cast<uint64_t>(k) * s->dims.vocab, s->logits,
+                                static_cast<uint64_t>(s->dims.vocab) * sizeof(float), cudaMemcpyDeviceToHost, s->stream);
+      }
+    }
+  }
+  if (err == cudaSuccess)
+    err = cudaMemcpyAsync(s->host_error, s->device_error, sizeof(uint32_t), cudaMemcpyDeviceToHost, s->stream);
+  const cudaError_t sync = cudaStreamSynchronize(s->stream);
+  if (err == cudaSuccess) err = sync;
+  if (err != cudaSuccess) return fail(&counters, err);
+  if (device_error_set(s, &counters)) return -1;
+  s->seed_token = tokens[count - 1u];
+  s->observed = 0;
+  s->cursor = end;
+  s->started = true;
+  s->finished = false;
+  s->logits_valid = true;
+  return 0;
+}
+
+extern "C" int nerva_b200_session_capture_stream(Session *s, float *stream, uint32_t capacity_rows) {
+  if (s == nullptr || !s->parallel || (stream != nullptr && capacity_rows == 0)) return -1;
+  s->capture_stream = stream;
+  s->capture_rows = capacity_rows;
   return 0;
 }
 
@@ -2505,7 +2701,7 @@ extern "C" int nerva_b200_session_get_kv_block_table(Session *s, uint32_t *table
 extern "C" int nerva_b200_session_read_kv_row(Session *s, uint32_t layer, uint32_t token,
                                               uint32_t which, uint16_t *row, uint32_t capacity) {
   if (s == nullptr || row == nullptr || layer >= s->dims.layers || token >= s->max_context ||
-      which > 1 || capacity < s->dims.kv_row() || (which == 1 && s->dims.mla()))
+      which > 1 || s->parallel || capacity < s->dims.kv_row() || (which == 1 && s->dims.mla()))
     return -1;
   if (cudaStreamSynchronize(s->stream) != cudaSuccess) return -1;
   uint32_t physical = 0;

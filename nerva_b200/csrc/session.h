@@ -48,12 +48,15 @@ struct LayerLayout {
   // (expert_up_offset = moe_intermediate * hidden inside a stride of twice that); DeepSeek layers
   // hold all gate matrices, then all up matrices (weights_pack.inc.cu:303-312).
   uint64_t expert_stride = 0, expert_up_offset = 0;
+  // parallel-block layers (rms_attn is the layer's one norm): per-channel scales of the two sublayers
+  uint64_t ls_attn = kMissingOffset, ls_mlp = kMissingOffset;
   // expert parallel: the experts whose matrices this arena holds (all of them otherwise)
   uint32_t expert_base = 0, expert_local = 0;
 };
 
 struct ArenaLayout {
   uint64_t embeddings = 0, input = 0, scratch = 0, final_norm = 0, lm_head = 0;
+  uint64_t loop_vectors = kMissingOffset;  // [loop_times][hidden]
   uint64_t elements = 0;
   std::vector<LayerLayout> layers;
 };
@@ -82,7 +85,57 @@ struct ModelDims {
 
 bool valid_layer(const NervaCudaHfDecodeChainLayer &layer, bool require_sources);
 bool layer_supported(const NervaCudaHfDecodeChainLayer &layer);
-ArenaLayout compute_arena_layout(const ModelDims &dims, const NervaCudaHfDecodeChainLayer *layers);
+ArenaLayout compute_arena_layout(const ModelDims &dims, const NervaCudaHfDecodeChainLayer *layers,
+                                 const NervaB200ParallelModel *parallel = nullptr);
+
+// ---- parallel-block decoders (parallel_step.cu) ----
+// One layer: its attention shape and the padded copies of its weights the kernels read (every
+// dimension a projection sums over, and every output of the residual stream, rounded up to 64 with
+// zeros, so that neither TMA nor the norm prologue sees an odd size).
+struct ParallelLayerPlan {
+  WindowAttentionShape shape{};
+  uint32_t intermediate = 0, ff_pad = 0;      // 0: no feed-forward
+  uint32_t qkv_rows = 0, qkv_pad = 0;         // [Q; K; V] rows, rounded up
+  uint32_t attn_width = 0, attn_pad = 0;      // heads * v_dim
+  bool layer_scale = false;
+  std::vector<float> frequencies;
+  uint16_t *w_in = nullptr;    // [qkv_pad + 2 ff_pad][width_pad]: Q, K, V, then gate/up rows interleaved
+  uint16_t *w_o = nullptr;     // [width_pad][attn_pad]
+  uint16_t *w_down = nullptr;  // [width_pad][ff_pad]
+  uint16_t *norm = nullptr, *ls_attn = nullptr, *ls_mlp = nullptr;  // [width_pad]
+  float *frequency = nullptr;
+};
+// One execution of a layer: a looped layer runs several times, each with its own part of the cache.
+struct ParallelRun {
+  uint32_t layer = 0;
+  int32_t step = -1;  // row of the loop vectors added to the stream before this run, -1: none
+  uint64_t key_offset = 0, value_offset = 0;  // elements from the start of a session's K / V array
+};
+struct ParallelPlan {
+  bool f32 = false;
+  uint32_t width = 0, width_pad = 0, vocab = 0, loop_times = 0;
+  float embedding_scale = 1.0f, softcap = 0.0f;
+  std::vector<ParallelLayerPlan> layers;
+  std::vector<ParallelRun> runs;
+  uint64_t key_elems = 0, value_elems = 0;    // per session, all runs
+  uint32_t max_heads = 0, max_qkv_pad = 0, max_attn_pad = 0, max_ff_pad = 0, max_v_pad = 0;
+  uint16_t *loop_vectors = nullptr;           // [loop_times][width_pad]
+  uint16_t *final_norm = nullptr, *head = nullptr;  // [width_pad], [vocab][width_pad]
+  uint32_t element_bytes() const { return f32 ? 4u : 2u; }
+};
+// Null (with the reason in last_error) when the description is inconsistent or beyond the kernels.
+std::shared_ptr<ParallelPlan> make_parallel_plan(const NervaB200ParallelModel &model, uint32_t width, uint32_t vocab,
+                                                 float eps);
+// Cache offsets of the runs for a session of `pages` pages.
+void place_parallel_cache(ParallelPlan *plan, uint32_t pages);
+struct StepProfile;
+typedef void (*ProfileMark)(NervaCudaHfDecodeSequenceSession *, StepProfile *, uint32_t bucket);
+cudaError_t pack_parallel_weights(NervaCudaHfDecodeSequenceSession *s);
+// All layer runs of one decode step (s->h_b in and out), and its head; enqueue only.
+cudaError_t enqueue_parallel_layers(NervaCudaHfDecodeSequenceSession *s, uint32_t splits, uint64_t *launches,
+                                    StepProfile *prof, ProfileMark mark);
+cudaError_t enqueue_parallel_head(NervaCudaHfDecodeSequenceSession *s, uint32_t *partials, uint64_t *launches);
+uint32_t parallel_attention_splits(const ParallelPlan &plan, uint32_t target_context);
 uint64_t hash_tokens(const uint32_t *tokens, uint32_t count);
 uint64_t hash_weight_descriptors(const NervaCudaHfDecodeSequenceWeightBlock *blocks, uint32_t count);
 void set_last_error(const std::string &text);
@@ -119,6 +172,7 @@ struct BlockWorkspace {
   bool paged_rows = false;      // the rows' attention runs on the paged tensor-pipe kernel (attention.cu)
   BlockTokenRow *token_rows = nullptr;
   BlockSampleRow *sample_rows_dev = nullptr;  // [sample_rows] device copies of the sampler's row descriptors
+  uint32_t *head_rows = nullptr;  // [sample_rows] rows of the block whose logits are wanted
 };
 constexpr uint32_t kBlockArgmaxChunks = 64;
 constexpr uint32_t kBlockMaxRows = 256;       // one MMA N
@@ -177,11 +231,29 @@ cudaError_t allocate_block_workspace(NervaCudaHfDecodeSequenceSession *s);
 // synchronised.  Enqueues only; the caller copies the token slots back and synchronises.
 cudaError_t enqueue_block_decode(NervaCudaHfDecodeSequenceSession *const *sessions, uint32_t count,
                                  cudaStream_t stream, uint64_t *launches);
-// Prompt positions [0, prompt_count) of one session through every layer in chunks of up to
+// Logits wanted from a prefill: places[i] counts from the first position of the call, values go to
+// logits[i][vocab] (host).
+struct WantedLogits {
+  const uint32_t *places = nullptr;
+  uint32_t count = 0;
+  float *logits = nullptr;
+};
+// Prompt positions [begin, prompt_count) of one session through every layer in chunks of up to
 // kBlockMaxRows tokens, writing the same paged bf16 K/V the decode step reads, then the final
 // norm, lm_head and the sampler for the last position.  Leaves the cursor at prompt_count.
-cudaError_t enqueue_chunked_prefill(NervaCudaHfDecodeSequenceSession *s, uint32_t prompt_count, uint32_t sample_kind,
-                                    uint64_t *launches);
+cudaError_t enqueue_chunked_prefill(NervaCudaHfDecodeSequenceSession *s, uint32_t begin, uint32_t prompt_count,
+                                    const WantedLogits &wanted, uint64_t *launches);
+// The layer runs of a parallel-block model over the block's rows (ws.h_b in and out) and the head of
+// `count` rows (row_index: device array of block rows, null: the first `count`) into ws.logits.
+struct ParallelBlock {
+  cudaStream_t stream;
+  uint32_t rows, longest;
+  bool one_session;            // consecutive positions of one session
+  uint32_t capture_row;        // row of the capture buffer the first row of the block goes to
+};
+cudaError_t enqueue_parallel_block_layers(NervaCudaHfDecodeSequenceSession *s, const ParallelBlock &b, uint64_t *launches);
+cudaError_t enqueue_parallel_block_head(NervaCudaHfDecodeSequenceSession *s, cudaStream_t stream, uint32_t count,
+                                        const uint32_t *row_index, uint64_t *launches);
 
 }  // namespace nb
 
@@ -205,6 +277,9 @@ struct NervaCudaHfDecodeSequenceSession {
   uint64_t planned_weight_descriptor_hash = 0;
 
   std::shared_ptr<nb::SharedWeights> weights;
+  std::shared_ptr<nb::ParallelPlan> parallel;  // parallel-block models only
+  float *capture_stream = nullptr;             // host buffer of nerva_b200_session_capture_stream
+  uint32_t capture_rows = 0;
   nb::StaticArena weight_arena, state_arena;
   nb::KvPagePool kv_pool;
 

@@ -120,8 +120,9 @@ __device__ __forceinline__ void norm_single_load(NormValueRegs &r, const float *
     r.v[k] = i < vecs ? __ldcg(reinterpret_cast<const float4 *>(a) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
 }
+// mean_count: elements the mean is taken over, when the vector is padded with zeros up to cols (0: cols).
 __device__ __forceinline__ void norm_single_finish(uint16_t *x, const NormValueRegs &loaded, const NormWeightRegs &regs,
-                                                   float eps, uint32_t cols, float *scratch) {
+                                                   float eps, uint32_t cols, float *scratch, uint32_t mean_count = 0) {
   const uint32_t vecs = cols / 4u;
   const float4 *r = loaded.v;
   float sumsq = 0.0f;
@@ -134,7 +135,7 @@ __device__ __forceinline__ void norm_single_finish(uint16_t *x, const NormValueR
     }
   }
   const float total = block_sum(sumsq, scratch);
-  const float scale = rsqrtf(total / static_cast<float>(cols) + eps);
+  const float scale = rsqrtf(total / static_cast<float>(mean_count != 0 ? mean_count : cols) + eps);
 #pragma unroll
   for (uint32_t k = 0; k < kNormRegIters; ++k) {
     const uint32_t i = threadIdx.x + k * blockDim.x;

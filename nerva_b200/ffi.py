@@ -16,7 +16,7 @@ LIB_PATH = os.environ.get("NERVA_B200_LIB") or os.path.join(_HERE, "_lib", "libn
 
 _SCALARS = {
     "uint8_t": C.c_uint8, "uint16_t": C.c_uint16, "uint32_t": C.c_uint32, "uint64_t": C.c_uint64,
-    "int32_t": C.c_int32, "int64_t": C.c_int64, "float": C.c_float, "char": C.c_char,
+    "int32_t": C.c_int32, "int64_t": C.c_int64, "float": C.c_float, "double": C.c_double, "char": C.c_char,
 }
 
 structs: dict[str, type] = {}
@@ -131,6 +131,10 @@ def _bind(L: C.CDLL, reference_abi_only: bool) -> C.CDLL:
         "nerva_b200_session_read_timeline": [vp, vp, C.c_uint32],
         "nerva_b200_session_create_sharded": [P(CreateRequest), P(structs["NervaB200ShardInfo"]), P(CreateResult),
                                               P(vp)],
+        "nerva_b200_session_create_parallel": [P(CreateRequest), P(structs["NervaB200ParallelModel"]),
+                                               P(CreateResult), P(vp)],
+        "nerva_b200_session_append": [vp, vp, C.c_uint32, C.c_uint32, vp, C.c_uint32, vp],
+        "nerva_b200_session_capture_stream": [vp, vp, C.c_uint32],
         "nerva_b200_session_comm_handle": [vp, vp, C.c_uint32],
         "nerva_b200_session_attach_peers": [vp, vp, C.c_uint32],
         "nerva_b200_session_attach_loopback": [vp],

@@ -14,6 +14,7 @@ from dataclasses import dataclass, field
 import numpy as np
 
 from . import ffi
+from .safetensors_file import FileTensor
 
 CUDA_ERROR_NO_DEVICE = 100
 CUDA_ERROR_NOT_SUPPORTED = 801
@@ -147,15 +148,19 @@ def write_weight_file(checkpoint, path: str, header_bytes: int = 0) -> None:
 
 def weight_blocks(checkpoint, staged_every: int = 2, source_file: str | None = None, header_bytes: int = 0):
     """Descriptor table in upload order with contiguous offsets over the resident weight bytes.
-    Blocks come from the host tensors, or (source_file) from byte ranges of a file laid out by
+    Blocks come from the host tensors, from the file ranges a checkpoint names itself (FileTensor), or (source_file) from byte ranges of a file laid out by
     write_weight_file, which the library reads through its pinned staging buffer
     (hf_decode_sequence/weights.cu:797-850).  Returns (array, objects to keep alive)."""
-    tensors = _upload_order(checkpoint)
+    tensors = checkpoint.upload_order() if hasattr(checkpoint, "upload_order") else _upload_order(checkpoint)
     arr = (ffi.WeightBlock * len(tensors))()
     path_bytes = source_file.encode() if source_file is not None else None
     offset = 0
     for i, t in enumerate(tensors):
-        if path_bytes is None:
+        if isinstance(t, FileTensor):
+            arr[i].source_file = t.path
+            arr[i].source_file_len = len(t.path)
+            arr[i].file_offset_begin = t.offset
+        elif path_bytes is None:
             arr[i].host_source = _ptr(t)
         else:
             arr[i].source_file = path_bytes
@@ -176,23 +181,31 @@ class CudaHfDecodeSequenceSession:
     """Owns one native session handle (create ... destroy)."""
 
     def __init__(self, checkpoint, max_context_tokens: int, use_descriptors: bool = False, dtype: int = DTYPE_BF16,
-                 engine: int = 0, library=None, weight_file: str | None = None, weight_file_header: int = 0):
+                 engine: int = 0, library=None, weight_file: str | None = None, weight_file_header: int = 0,
+                 compute: str = "bfloat16"):
         """library: a handle from ffi.load_abi_library for another implementation of the same C ABI
         (default: this package's libnerva_b200.so).  weight_file: upload through descriptors that
-        name byte ranges of this file (see write_weight_file) instead of host pointers."""
+        name byte ranges of this file (see write_weight_file) instead of host pointers.
+        compute: "bfloat16", or "float32" for models that also run in true fp32 (parallel_model)."""
         cfg = checkpoint.config
         self._lib = library if library is not None else ffi.lib()
         self._own_library = library is None
         self.config = cfg
         self._keep = [checkpoint]
-        layers = chain_layers(checkpoint)
+        parallel = checkpoint.native_model(compute) if hasattr(checkpoint, "native_model") else None
+        if compute != "bfloat16" and parallel is None:
+            raise ValueError(f"{cfg.name} runs in bfloat16 only")
+        layers = chain_layers(checkpoint) if parallel is None else (ffi.ChainLayer * cfg.layers)()
         req = ffi.CreateRequest(
             dtype=dtype, hidden=cfg.hidden, heads=cfg.heads, kv_heads=cfg.kv_heads, head_dim=cfg.head_dim,
             intermediate=cfg.intermediate, vocab_size=cfg.vocab, layer_count=cfg.layers,
             max_context_tokens=max_context_tokens, rms_eps=cfg.rms_eps, rope_theta=cfg.rope_theta,
-            embeddings=_ptr(checkpoint.embeddings), layers=C.cast(layers, C.c_void_p),
-            final_norm_weight=_ptr(checkpoint.final_norm), lm_head=_ptr(checkpoint.lm_head))
-        if use_descriptors or weight_file is not None or getattr(cfg, "kv_lora_rank", 0):
+            layers=C.cast(layers, C.c_void_p))
+        if parallel is None:
+            req.embeddings = _ptr(checkpoint.embeddings)
+            req.final_norm_weight = _ptr(checkpoint.final_norm)
+            req.lm_head = _ptr(checkpoint.lm_head)
+        if use_descriptors or weight_file is not None or getattr(cfg, "kv_lora_rank", 0) or parallel is not None:
             blocks = weight_blocks(checkpoint, source_file=weight_file, header_bytes=weight_file_header)
             self._keep.append(blocks)
             req.planned_weight_blocks = len(blocks)
@@ -208,7 +221,10 @@ class CudaHfDecodeSequenceSession:
         self._handle = C.c_void_p()
         self.create_result = ffi.CreateResult()
         self.shard = getattr(checkpoint, "shard", None)
-        if self.shard is not None:
+        if parallel is not None:
+            rc = self._lib.nerva_b200_session_create_parallel(C.byref(req), C.byref(parallel),
+                                                              C.byref(self.create_result), C.byref(self._handle))
+        elif self.shard is not None:
             # a tensor- or expert-parallel rank: `checkpoint` holds this rank's slices (nerva_b200.synth.shard_checkpoint,
             # expert_shard_checkpoint)
             info = ffi.structs["NervaB200ShardInfo"](rank=self.shard.rank, world=self.shard.world,
@@ -285,6 +301,30 @@ class CudaHfDecodeSequenceSession:
         rc = self._lib.nerva_cuda_hf_decode_sequence_session_run(C.byref(req), C.byref(out))
         return Summary(_status(rc, out.status, out.cuda_error, out.device_count),
                        tokens[:out.observed_tokens].tolist(), out, self._last_error())
+
+    def append(self, tokens, want=(), reset: bool = False) -> np.ndarray:
+        """Runs given tokens after the positions this session has already run (reset: from position 0)
+        and returns the logits at the places `want` among them, [len(want), vocab].  The last position is
+        sampled as after start, so a CudaHfDecodeSequenceLoop can go on from here."""
+        ids = np.ascontiguousarray(tokens, dtype=np.uint32)
+        places = np.ascontiguousarray(want, dtype=np.uint32)
+        logits = np.empty((places.size, self.config.vocab), dtype=np.float32)
+        if ffi.lib().nerva_b200_session_append(self._handle, _ptr(ids), ids.size, int(reset), _ptr(places), places.size,
+                                               _ptr(logits)) != 0:
+            raise RuntimeError("append failed: " + (ffi.last_error() or "invalid arguments"))
+        return logits
+
+    def append_with_stream(self, tokens, reset: bool = False) -> np.ndarray:
+        """append of at least two tokens; returns the residual stream after every layer run, [runs, tokens, hidden]
+        (parallel-block models)."""
+        stream = np.zeros((self.config.layer_runs, len(tokens), self.config.hidden), dtype=np.float32)
+        if ffi.lib().nerva_b200_session_capture_stream(self._handle, _ptr(stream), len(tokens)) != 0:
+            raise RuntimeError("no stream capture for this model")
+        try:
+            self.append(tokens, reset=reset)
+        finally:
+            ffi.lib().nerva_b200_session_capture_stream(self._handle, None, 0)
+        return stream
 
     def read_logits(self) -> np.ndarray:
         logits = np.empty(self.config.vocab, dtype=np.float32)
