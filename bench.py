@@ -754,6 +754,108 @@ def run_deepseek_workload(args, rank: int = 0, world: int = 1) -> None:
     session.destroy()
 
 
+# Layer shapes of the vuvolix workload: (hidden, heads, kv_heads, head size, intermediate, vocab, layer runs).
+# The dense model beside each has the same shapes and as many layers as the design has layer runs.
+VUVOLIX_SIZES = {
+    "0.6b": (1024, 16, 8, 128, 3072, 151936, 28),
+    "1.7b": (2048, 16, 8, 128, 6144, 151936, 28),
+    "8b": (4096, 32, 8, 128, 12288, 151936, 36),
+}
+
+
+def vuvolix_config(size: str, window: int):
+    """Two thirds of the layer runs come from distinct layers, one third from a second pass over the middle ones."""
+    from nerva_b200 import parallel_model as pm
+    hidden, heads, kv_heads, dim, inter, vocab, runs = VUVOLIX_SIZES[size]
+    looped = runs // 3
+    layers = runs - looped
+    spec = pm.ParallelLayer(heads=heads, kv_heads=kv_heads, qk_dim=dim, v_dim=dim, intermediate=inter, window=window,
+                            score_scale=dim ** -0.5, rotary_dims=dim // 2, rotary_base=1e6,
+                            scaling={"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0})
+    start = (layers - looped) // 2
+    return pm.ParallelConfig(name=f"vuvolix-{size}", hidden=hidden, vocab=vocab, rms_eps=1e-6, layer_specs=(spec,) * layers,
+                             embedding_scale=hidden ** 0.5, logit_softcap=30.0, loop_start=start, loop_stop=start + looped,
+                             loop_times=2)
+
+
+def run_vuvolix_workload(args) -> None:
+    """Prefill and decode of the Vuvolix design (parallel blocks, windowed attention, a looped range of layers)
+    beside the dense model of equal layer shapes: per size one JSON line with both models' prefill tok/s at
+    several prompt lengths, batch-1 decode tok/s after the longest prompt, and the packed step of 16 forks.
+    Device time (CUDA events inside the library) for prefill and decode; wall clock around the calls for the
+    packed step.  Every timed decode step streams more weight bytes than the L2 holds."""
+    from nerva_b200 import build, ops, parallel_model, synth
+    from nerva_b200.session import CudaHfDecodeSequenceLoop, CudaHfDecodeSequenceSession, SmokeStatus
+    build.build()
+    prompts = [args.prompt_tokens] if args.prompt_tokens else [256, 512, 2048]
+    window = args.context or 1024
+    peaks = measured_peaks()
+    for size in [args.shape] if args.shape else list(VUVOLIX_SIZES):
+        hidden, heads, kv_heads, dim, inter, vocab, runs = VUVOLIX_SIZES[size]
+        cfg = vuvolix_config(size, window)
+        dense = synth.DecoderConfig(f"dense-{size}", layers=runs, hidden=hidden, heads=heads, kv_heads=kv_heads, head_dim=dim,
+                                    intermediate=inter, vocab=vocab)
+        line = {"workload": "vuvolix beside the dense model of equal layer shapes", "size": size, "steps": args.steps,
+                "config": {"hidden": hidden, "heads": heads, "kv_heads": kv_heads, "head_size": dim, "intermediate": inter,
+                           "vocab": vocab, "layer_runs": runs, "window": window, "layers": cfg.layers,
+                           "loop": [cfg.loop_start, cfg.loop_stop, cfg.loop_times], "weights": "random-init bf16 (synthetic)",
+                           "l2": "every step streams more weight bytes than the L2 holds"}}
+        for name, model, nbytes in (("vuvolix", cfg, cfg.streamed_bytes_per_token()),
+                                    ("dense", dense, dense.projection_bytes_per_token())):
+            if name == "vuvolix":
+                ck = parallel_model.random_checkpoint(cfg, fill=ops.synth_normal_bf16)
+            else:
+                ck = synth.dense_checkpoint(dense, fill=ops.synth_normal_bf16)
+            context = max(prompts) + max(args.warmup, 3) + args.steps + 48 + MAX_EXTRA_CLOCK_STEPS
+            session = CudaHfDecodeSequenceSession(ck, context, use_descriptors=True)
+            del ck
+            if session.status != SmokeStatus.OK:
+                raise RuntimeError(f"{name}: {session.error}")
+            sampler = ClockSampler(int(os.environ.get("NERVA_GPU_INDEX", "0")))
+            sampler.start()
+            sampler.mark()
+            prefill = {}
+            for n in prompts:
+                ids = synth.prompt_ids(dense, count=n)
+                times = []
+                for i in range(6):
+                    start, loop = CudaHfDecodeSequenceLoop.start(session, ids)
+                    if start.status != SmokeStatus.OK:
+                        raise RuntimeError(f"{name}: {start.error}")
+                    if i >= 3:
+                        times.append(start.device_elapsed_ns * 1e-9)
+                prefill[n] = n / (sum(times) / len(times))
+            loop.advance(max(args.warmup, 3))
+            timed = loop.advance(args.steps)
+            if timed.status != SmokeStatus.OK:
+                raise RuntimeError(f"{name}: {timed.error}")
+            seconds = timed.device_elapsed_ns * 1e-9
+            extra = extra_clock_steps(seconds, args.steps)
+            if extra:
+                loop.advance(extra)
+            clocks = sampler.stop()
+            profile = session.profile_steps(4)
+            forks = [session] + [session.fork_shared_weights() for _ in range(15)]
+            packed = None  # the packed step takes dense models only where the heads span the hidden size
+            if CudaHfDecodeSequenceSession.batch_advance_one(forks, 16, 16).block_tokens == 16:
+                CudaHfDecodeSequenceSession.batch_advance_one(forks, 16, 16)
+                t0 = time.perf_counter()
+                for _ in range(16):
+                    out = CudaHfDecodeSequenceSession.batch_advance_one(forks, 16, 16)
+                    if out.status != SmokeStatus.OK or out.block_tokens != 16:
+                        raise RuntimeError(f"{name}: packed step: {out.error}")
+                packed = 16 * 16 / (time.perf_counter() - t0)
+            line[name] = {"prefill_tok_s": prefill, "decode_tok_s": args.steps / seconds,
+                          "decode_frac_of_measured_hbm": nbytes * args.steps / seconds / 1e9 / peaks["hbm_gbs"],
+                          "streamed_bytes_per_token": nbytes, "packed_16_tok_s": packed, "clocks": clocks,
+                          "decode_us_by_bucket": {k: v["ns"] / 4e3 for k, v in profile.items()},
+                          "launches_per_step": int(timed.graph_nodes)}
+            for f in forks:
+                f.destroy()
+        line["peak_source"] = peaks["source"]
+        print(json.dumps(line), flush=True)
+
+
 def run_operator_workloads(kind: str, only_shape: str = "", only_tokens: int = 0, only_batch: int = 0,
                            only_context: int = 0) -> None:
     """Per-operator sweeps (isolated projection shapes, long-context attention) through the per-op C ABI (host buffers in,
@@ -874,13 +976,13 @@ def main() -> None:
     ap.add_argument("--layers", type=int, default=0,
                     help="cut the model to this many layers (profiler captures only; not a bench line)")
     ap.add_argument("--prompt-tokens", type=int, default=0, help="override the prompt length")
-    ap.add_argument("--workload", default="decode", choices=["decode", "linear", "attention", "reference-gpu", "batch", "deepseek"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "linear", "attention", "reference-gpu", "batch", "deepseek", "vuvolix"],
                     help="decode: the bench line; linear / attention: per-operator sweeps of the isolated "
                          "projection shapes and of long-context attention (one JSON line per case)")
-    ap.add_argument("--shape", default="", help="linear sweep: only this projection (qkv, o, gate_up, down, lm_head)")
+    ap.add_argument("--shape", default="", help="vuvolix: only this size (0.6b, 1.7b, 8b); linear sweep: only this projection (qkv, o, gate_up, down, lm_head)")
     ap.add_argument("--tokens", type=int, default=0, help="linear sweep: only this block size")
     ap.add_argument("--batch", type=int, default=0, help="attention sweep: only this batch size")
-    ap.add_argument("--context", type=int, default=0, help="attention sweep: only this context length")
+    ap.add_argument("--context", type=int, default=0, help="attention sweep: only this context length; vuvolix: the window")
     ap.add_argument("--shard-of", type=int, default=0, choices=[0, 2, 4, 8],
                     help="attention sweep on one GPU: measure one rank's shard of an N-way split by KV head")
     ap.add_argument("--timeline", action="store_true",
@@ -905,6 +1007,10 @@ def main() -> None:
     if args.workload in ("linear", "attention"):
         if rank == 0:
             run_operator_workloads(args.workload, args.shape, args.tokens, args.batch, args.context)
+        return
+    if args.workload == "vuvolix":
+        if rank == 0:
+            run_vuvolix_workload(args)
         return
     cfg = workload(args.config, args.layers, args.prompt_tokens)
     if args.workload == "reference-gpu":

@@ -254,17 +254,17 @@ def test_packed_batches_of_unequal_requests(built_lib, full, dtype):
         assert f.status == SmokeStatus.OK
         history = tokens[i:i + n]
         f.append(history, reset=True)
+        first = CudaHfDecodeSequenceLoop(f).advance(1)  # the token the last given position sampled
+        assert first.status == SmokeStatus.OK
         forks.append(f)
-        histories.append(list(history))
+        histories.append(list(history) + first.tokens)
     for step in range(6):
         out = CudaHfDecodeSequenceSession.batch_advance_one(forks, target_block_tokens=len(forks))
         assert out.status == SmokeStatus.OK and out.block_tokens == len(forks), out.error
         for f, history, token in zip(forks, histories, out.tokens):
-            if step:
-                # the packed step ran the previous token; its logits chose this one
-                want = O.forward(cfg, w, history)[-1]
-                assert M.distance(f.read_logits(), want) < 3 * M.TOLERANCE[dtype]
-                assert want.max() - want[token] < 0.1 * want.std()
+            want = O.forward(cfg, w, history)[-1]
+            assert M.distance(f.read_logits(), want) < 3 * M.TOLERANCE[dtype]
+            assert want.max() - want[token] < 0.3 * want.std()
             history.append(token)
 
 
