@@ -331,9 +331,10 @@ cudaError_t launch_moe_experts(cudaStream_t stream, const MoeExpertParams &p, ui
 // the residual stream.  All vectors are padded to multiples of 64 with zeros, matrices have zero
 // columns (and rows) there.
 enum ParallelProjectionKind : uint32_t {
-  kParallelIn = 0,    // x = norm(h + step); matrix 0 -> out_f32 (fp32), matrix 1 (gate/up rows interleaved) -> out_act
+  kParallelIn = 0,    // x = norm(h + step); matrix 0 -> out_f32 (fp32); the plain form also does kParallelGate
   kParallelOut = 1,   // h_out = (h + step) + scale0 * (matrix 0 . x0) + scale1 * (matrix 1 . x1)
   kParallelHead = 2,  // x = norm(h); matrix 0 -> soft-capped out_f32 and per-block arg-max partials
+  kParallelGate = 3,  // x = norm(h + step); matrix 1 (gate/up rows interleaved, cols0 columns) -> out_act
 };
 struct ParallelProjectionParams {
   const uint16_t *w0, *w1;       // [rows][cols] bf16
@@ -355,6 +356,12 @@ struct ParallelProjectionParams {
   uint32_t pdl;
 };
 // bf16 activations, weights through the TMA ring (row_stream.cuh).  Shapes it cannot hold go to the plain form.
+// The launches of a layer, in stream order with programmatic dependent launch, are kParallelIn, attention,
+// kParallelGate, kParallelOut.  The gate/up stream does not depend on the attention and runs beside it:
+//   * kParallelIn lets its successor start only after its own wait, so once the attention's blocks run, the
+//     stream h of the previous layer is complete;
+//   * kParallelGate therefore reads h without waiting, and waits for the attention only before it ends, so
+//     that its own completion covers both.
 bool parallel_stream_eligible(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count);
 uint32_t parallel_stream_blocks(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count);
 cudaError_t launch_parallel_projection(cudaStream_t stream, uint32_t kind, const ParallelProjectionParams &p,
@@ -405,7 +412,7 @@ struct WindowAttentionParams {
   const struct FusedAttentionRow *rows;
   uint32_t row_count;
 };
-constexpr uint32_t kWindowMaxSplits = 16;
+constexpr uint32_t kWindowMaxSplits = 32;  // a lane per span in the merge
 bool window_attention_supported(const WindowAttentionShape &s, bool f32);
 uint32_t window_attention_splits(uint32_t target_context, uint32_t window);
 cudaError_t configure_window_attention();

@@ -5,12 +5,15 @@
 // The streaming form puts two weight matrices into one launch on the row-stream core
 // (row_stream.cuh): its ring runs across a job list, so the second matrix's bytes follow the first's
 // without a gap.
-//   kParallelIn    [Q; K; V] and the interleaved gate/up matrix behind one norm prologue
+//   kParallelIn    [Q; K; V] behind the norm prologue
+//   kParallelGate  the interleaved gate/up matrix behind the same prologue
 //   kParallelOut   O and down, dealt to the blocks by the same row ranges, so the block that owns a
 //                  row of the stream has both sums and writes h + scale0 * O + scale1 * down once
 //   kParallelHead  the head behind the final norm, logits soft-capped before the arg-max
-// A layer is three launches with the attention in between, and the residual stream is read and
-// written once.
+// In a parallel block the feed-forward does not wait for the attention: kParallelGate streams its
+// matrix while the attention of the same layer runs beside it on the same SMs.  For that the two
+// kernels around the attention take two ring slots per warp instead of three, which leaves shared
+// memory for the attention's blocks (see the launch order in kernels.cuh).
 #include "kernels.cuh"
 #include "row_stream.cuh"
 #include "step_device.cuh"
@@ -19,12 +22,16 @@ namespace nb {
 namespace {
 
 constexpr uint32_t kNoIndex = 0xffffffffu;
-constexpr uint32_t kPrewaitSlots = kStreamSlots - 1;  // ring slots filled ahead of a norm prologue's loads
+// Ring slots per warp: two where an attention block shares the SM.
+constexpr uint32_t slots_of(uint32_t kind) { return kind == kParallelIn || kind == kParallelGate ? 2u : kStreamSlots; }
+constexpr uint32_t ring_bytes(uint32_t kind) { return kStreamWarps * slots_of(kind) * kChunkBytes; }
 
 __device__ __forceinline__ bool candidate_better(float v, uint32_t i, float best_v, uint32_t best_i) {
   return v > best_v || (v == best_v && i < best_i);
 }
 __device__ __forceinline__ float soft_cap(float y, float cap) { return cap > 0.0f ? cap * tanhf(y / cap) : y; }
+
+constexpr uint32_t kPlainL2PrefetchBytes = 16384;  // per warp, behind the plain vector copies
 
 struct ParallelShared {
   StreamShared first, second;  // the ring's barriers are first's; each job has its own edge records
@@ -38,29 +45,33 @@ __host__ __device__ inline uint32_t round128(uint32_t v) { return (v + 127u) & ~
 
 template <uint32_t KIND>
 __global__ void __launch_bounds__(kStreamThreads, 1) parallel_stream_kernel(ParallelProjectionParams p) {
+  constexpr uint32_t SLOTS = slots_of(KIND);
+  constexpr uint32_t kRing = ring_bytes(KIND);
   extern __shared__ __align__(128) uint8_t smem[];
   uint8_t *ring = smem;
-  uint16_t *x0 = reinterpret_cast<uint16_t *>(smem + kRingBytes);
-  uint16_t *x1 = reinterpret_cast<uint16_t *>(smem + kRingBytes + round128(p.cols0 * 2u));
-  const uint32_t x_bytes = round128(p.cols0 * 2u) + (KIND == kParallelOut && p.rows1 != 0 ? round128(p.cols1 * 2u) : 0u);
-  ParallelShared &sh = *reinterpret_cast<ParallelShared *>(smem + kRingBytes + x_bytes);
-  float *total0 = reinterpret_cast<float *>(smem + kRingBytes + x_bytes + round128(sizeof(ParallelShared)));
-  const bool second = KIND != kParallelHead && p.rows1 != 0;
-  const uint32_t unit1 = KIND == kParallelIn ? 2u : 1u;
+  uint16_t *x0 = reinterpret_cast<uint16_t *>(smem + kRing);
+  uint16_t *x1 = reinterpret_cast<uint16_t *>(smem + kRing + round128(p.cols0 * 2u));
+  const bool second = KIND == kParallelOut && p.rows1 != 0;
+  const uint32_t x_bytes = round128(p.cols0 * 2u) + (second ? round128(p.cols1 * 2u) : 0u);
+  ParallelShared &sh = *reinterpret_cast<ParallelShared *>(smem + kRing + x_bytes);
+  float *total0 = reinterpret_cast<float *>(smem + kRing + x_bytes + round128(sizeof(ParallelShared)));
+  constexpr uint32_t unit = KIND == kParallelGate ? 2u : 1u;
+  const uint32_t rows_all = KIND == kParallelGate ? p.rows1 : p.rows0;
 
-  pdl_trigger();
+  if (KIND != kParallelIn) pdl_trigger();
   if (threadIdx.x == 0) {
-    sh.jobs[0] = JobDesc{p.w0, p.rows0, p.cols0, 1, 0};
-    sh.jobs[1] = JobDesc{p.w1, p.rows1, KIND == kParallelIn ? p.cols0 : p.cols1, unit1, 0};
+    sh.jobs[0] = JobDesc{KIND == kParallelGate ? p.w1 : p.w0, rows_all, p.cols0, unit, 0};
+    sh.jobs[1] = JobDesc{p.w1, p.rows1, p.cols1, 1, 0};
   }
   __syncthreads();
   RowStream rs;
-  stream_init(rs, ring, sh.first, sh.jobs, second ? 2u : 1u);
-  stream_fill(rs, KIND == kParallelOut ? kStreamSlots : kPrewaitSlots);
+  stream_init<SLOTS>(rs, ring, sh.first, sh.jobs, second ? 2u : 1u);
+  // ahead of a norm prologue one slot is held back: the activation loads would queue behind a whole ring
+  stream_fill<SLOTS>(rs, KIND == kParallelOut ? SLOTS : SLOTS - 1u);
 
   uint32_t begin0, end0, begin1 = 0, end1 = 0;
-  block_row_range(p.rows0, 1, blockIdx.x, gridDim.x, &begin0, &end0);
-  if (second) block_row_range(p.rows1, unit1, blockIdx.x, gridDim.x, &begin1, &end1);
+  block_row_range(rows_all, unit, blockIdx.x, gridDim.x, &begin0, &end0);
+  if (second) block_row_range(p.rows1, 1, blockIdx.x, gridDim.x, &begin1, &end1);
   const uint32_t rows0 = end0 - begin0, rows1 = end1 - begin1;
   float *total1 = total0 + rows0;
   for (uint32_t r = threadIdx.x; r < rows0 + rows1; r += blockDim.x) total0[r] = 0.0f;
@@ -75,14 +86,16 @@ __global__ void __launch_bounds__(kStreamThreads, 1) parallel_stream_kernel(Para
       const uint4 *src1 = reinterpret_cast<const uint4 *>(p.x1);
       for (uint32_t i = threadIdx.x; i < p.cols1 / 8u; i += blockDim.x) reinterpret_cast<uint4 *>(x1)[i] = __ldcg(src1 + i);
     }
+    stream_prefetch_l2(rs, kPlainL2PrefetchBytes);
   } else {
     NormWeightRegs weights, step;
     norm_weights_preload(weights, p.norm, p.cols0);
     if (p.step != nullptr) norm_weights_preload(step, p.step, p.cols0);
-    pdl_wait();
+    if (KIND != kParallelGate) pdl_wait();
+    if (KIND == kParallelIn) pdl_trigger();  // whoever runs after this knows that h is complete
     NormValueRegs values;
     norm_single_load(values, p.h, p.cols0);
-    stream_fill(rs);  // the ring slot held back, now behind the activation loads
+    stream_fill<SLOTS>(rs);  // the ring slot held back, now behind the activation loads
     if (p.step != nullptr) {
 #pragma unroll
       for (uint32_t k = 0; k < kNormRegIters; ++k) {
@@ -96,19 +109,21 @@ __global__ void __launch_bounds__(kStreamThreads, 1) parallel_stream_kernel(Para
   }
   __syncthreads();
 
-  stream_consume(rs, sh.first, 0, x0, total0, p.error_word);
-  if (second) stream_consume(rs, sh.second, 1, KIND == kParallelOut ? x1 : x0, total1, p.error_word);
+  stream_consume<false, SLOTS>(rs, sh.first, 0, x0, total0, p.error_word);
+  if (second) stream_consume<false, SLOTS>(rs, sh.second, 1, x1, total1, p.error_word);
   __syncthreads();
 
   if (KIND == kParallelIn) {
     for (uint32_t r = threadIdx.x; r < rows0; r += blockDim.x)
       p.out_f32[begin0 + r] = stream_row_total(sh.first, total0, r);
+  } else if (KIND == kParallelGate) {
     uint16_t *act = reinterpret_cast<uint16_t *>(p.out_act);
-    for (uint32_t i = threadIdx.x; i < rows1 / 2u; i += blockDim.x) {
-      const float gate = stream_row_total(sh.second, total1, 2u * i);
-      const float up = stream_row_total(sh.second, total1, 2u * i + 1u);
-      act[begin1 / 2u + i] = f32_to_bf16_bits(silu(gate) * up);
+    for (uint32_t i = threadIdx.x; i < rows0 / 2u; i += blockDim.x) {
+      const float gate = stream_row_total(sh.first, total0, 2u * i);
+      const float up = stream_row_total(sh.first, total0, 2u * i + 1u);
+      act[begin0 / 2u + i] = f32_to_bf16_bits(silu(gate) * up);
     }
+    pdl_wait();  // the attention beside this launch: the next launch waits for this one only
   } else if (KIND == kParallelOut) {
     for (uint32_t r = threadIdx.x; r < rows0; r += blockDim.x) {
       const uint32_t row = begin0 + r;
@@ -160,25 +175,26 @@ __global__ void __launch_bounds__(kStreamThreads, 1) parallel_stream_kernel(Para
       p.best_index[blockIdx.x] = bi;
     }
   }
-  stream_drain(rs);
+  stream_drain<SLOTS>(rs);
 }
 
 uint32_t stream_blocks(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count) {
   // one block per SM; fewer when the matrices are too small to give every warp of every block 4 KiB
-  uint64_t bytes = static_cast<uint64_t>(p.rows0) * p.cols0 * 2u;
-  if (kind != kParallelHead)
-    bytes += static_cast<uint64_t>(p.rows1) * (kind == kParallelIn ? p.cols0 : p.cols1) * 2u;
+  const uint32_t rows = kind == kParallelGate ? p.rows1 : p.rows0;
+  uint64_t bytes = static_cast<uint64_t>(rows) * p.cols0 * 2u;
+  if (kind == kParallelOut) bytes += static_cast<uint64_t>(p.rows1) * p.cols1 * 2u;
   uint64_t blocks = bytes / (static_cast<uint64_t>(kStreamWarps) * 4096u);
-  if (blocks > p.rows0) blocks = p.rows0;
+  const uint32_t units = kind == kParallelGate ? rows / 2u : rows;
+  if (blocks > units) blocks = units;
   if (blocks > sm_count) blocks = sm_count;
   return blocks == 0 ? 1u : static_cast<uint32_t>(blocks);
 }
 
 uint32_t stream_smem_bytes(uint32_t kind, const ParallelProjectionParams &p, uint32_t blocks) {
-  const bool second = kind != kParallelHead && p.rows1 != 0;
-  uint32_t rows = max_rows_per_block(p.rows0, 1, blocks);
-  if (second) rows += max_rows_per_block(p.rows1, kind == kParallelIn ? 2u : 1u, blocks);
-  return kRingBytes + round128(p.cols0 * 2u) + (kind == kParallelOut && second ? round128(p.cols1 * 2u) : 0u) +
+  const bool second = kind == kParallelOut && p.rows1 != 0;
+  uint32_t rows = kind == kParallelGate ? max_rows_per_block(p.rows1, 2, blocks) : max_rows_per_block(p.rows0, 1, blocks);
+  if (second) rows += max_rows_per_block(p.rows1, 1, blocks);
+  return ring_bytes(kind) + round128(p.cols0 * 2u) + (second ? round128(p.cols1 * 2u) : 0u) +
          round128(sizeof(ParallelShared)) + round128(rows * 4u + 16u);
 }
 
@@ -305,14 +321,18 @@ cudaError_t configure_parallel_projection() {
   if (err == cudaSuccess)
     err = cudaFuncSetAttribute(parallel_stream_kernel<kParallelOut>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
   if (err == cudaSuccess)
+    err = cudaFuncSetAttribute(parallel_stream_kernel<kParallelGate>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
+  if (err == cudaSuccess)
     err = cudaFuncSetAttribute(parallel_stream_kernel<kParallelHead>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
   return err;
 }
 
 bool parallel_stream_eligible(uint32_t kind, const ParallelProjectionParams &p, uint32_t sm_count) {
   auto aligned = [](const void *q) { return reinterpret_cast<uintptr_t>(q) % 16u == 0; };
-  if (p.rows0 == 0 || p.cols0 == 0 || p.cols0 % 8u != 0 || !aligned(p.w0)) return false;
-  if (p.rows1 != 0 && (!aligned(p.w1) || p.cols1 % 8u != 0 || (kind == kParallelIn && p.rows1 % 2u != 0))) return false;
+  if (p.cols0 == 0 || p.cols0 % 8u != 0) return false;
+  if (kind == kParallelGate ? p.rows1 == 0 || p.rows1 % 2u != 0 || !aligned(p.w1) : p.rows0 == 0 || !aligned(p.w0))
+    return false;
+  if (kind == kParallelOut && p.rows1 != 0 && (!aligned(p.w1) || p.cols1 % 8u != 0)) return false;
   if (kind == kParallelOut) {
     if (!aligned(p.x0) || (p.rows1 != 0 && (!aligned(p.x1) || p.rows1 != p.rows0))) return false;
   } else if (p.cols0 / 4u > kNormRegIters * kStreamThreads || !aligned(p.h) ||
@@ -330,16 +350,17 @@ cudaError_t launch_parallel_projection(cudaStream_t stream, uint32_t kind, const
                                        uint32_t sm_count) {
   if (!parallel_stream_eligible(kind, p, sm_count)) return cudaErrorInvalidValue;
   const uint32_t blocks = stream_blocks(kind, p, sm_count);
-  void (*kernel)(ParallelProjectionParams) = kind == kParallelIn    ? parallel_stream_kernel<kParallelIn>
-                                             : kind == kParallelOut ? parallel_stream_kernel<kParallelOut>
-                                                                    : parallel_stream_kernel<kParallelHead>;
+  void (*kernel)(ParallelProjectionParams) = kind == kParallelIn     ? parallel_stream_kernel<kParallelIn>
+                                             : kind == kParallelOut  ? parallel_stream_kernel<kParallelOut>
+                                             : kind == kParallelGate ? parallel_stream_kernel<kParallelGate>
+                                                                     : parallel_stream_kernel<kParallelHead>;
   return launch_with_pdl(kernel, dim3(blocks), dim3(kStreamThreads), stream_smem_bytes(kind, p, blocks), stream,
                          p.pdl != 0, p);
 }
 
 cudaError_t launch_parallel_projection_plain(cudaStream_t stream, uint32_t kind, const ParallelProjectionParams &p,
                                              uint32_t tokens, bool f32) {
-  if (tokens == 0 || p.rows0 == 0 || p.cols0 % 64u != 0 || p.cols1 % 64u != 0) return cudaErrorInvalidValue;
+  if (tokens == 0 || kind > kParallelHead || p.rows0 == 0 || p.cols0 % 64u != 0 || p.cols1 % 64u != 0) return cudaErrorInvalidValue;
   const uint32_t units = p.rows0 + (kind == kParallelIn ? p.rows1 / 2u : 0u);
   const dim3 grid((units + kPlainWarps - 1u) / kPlainWarps, (tokens + kPlainTokens - 1u) / kPlainTokens);
   void (*kernel)(ParallelProjectionParams, uint32_t);

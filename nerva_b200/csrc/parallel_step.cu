@@ -5,8 +5,8 @@
 // (block_step.cu).  Token fetch, embedding, sampler, token ring, graphs, page table and forks are the
 // session's own.
 //
-// Decode step, per layer run: norm + [Q; K; V | gate/up] -> attention -> [O | down] + residual: three
-// launches.  Block step: norm, one projection for all five input matrices, q/k preparation + cache
+// Decode step, per layer run: norm + [Q; K; V] -> attention, with norm + gate/up streaming beside it ->
+// [O | down] + residual: four launches.  Block step: norm, one projection for all five input matrices, q/k preparation + cache
 // append, attention, O and down with the residual add in their epilogues.
 #include <math.h>
 
@@ -286,7 +286,9 @@ cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launc
     out.step = step;
     out.x0 = s->attn_bf16;
     out.x1 = s->ff_bf16;
+    const bool gate = l.ff_pad != 0;
     const bool streamed = !plan.f32 && parallel_stream_eligible(kParallelIn, in, s->sm_count) &&
+                          (!gate || parallel_stream_eligible(kParallelGate, in, s->sm_count)) &&
                           parallel_stream_eligible(kParallelOut, first_matrix(out), s->sm_count) &&
                           (out.rows1 == 0 || parallel_stream_eligible(kParallelOut, second_matrix(out), s->sm_count));
     if (streamed) {
@@ -323,6 +325,12 @@ cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launc
     n += 1;
     mark(s, prof, kBucketAttention);
     if (err != cudaSuccess) break;
+    if (streamed && gate) {
+      err = launch_parallel_projection(s->stream, kParallelGate, in, s->sm_count);
+      n += 1;
+      mark(s, prof, kBucketGateUp);
+      if (err != cudaSuccess) break;
+    }
 
     if (!streamed) {
       err = launch_parallel_projection_plain(s->stream, kParallelOut, out, 1, plan.f32);

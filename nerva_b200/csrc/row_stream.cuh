@@ -152,11 +152,13 @@ struct RowStream {
   uint64_t policy;  // L2 evict-first: weights are read once per step
 };
 
+// SLOTS (at most kStreamSlots): ring slots per warp; a kernel that shares its SM with another takes fewer.
+template <uint32_t SLOTS = kStreamSlots>
 __device__ inline void stream_init(RowStream &rs, uint8_t *ring_base, StreamShared &sh,
                                    const JobDesc *jobs, uint32_t job_count) {
   const uint32_t warp = threadIdx.x >> 5;
-  rs.ring = ring_base + warp * kStreamSlots * kChunkBytes;
-  rs.bars = sh.bars + warp * kStreamSlots;
+  rs.ring = ring_base + warp * SLOTS * kChunkBytes;
+  rs.bars = sh.bars + warp * SLOTS;
   rs.jobs = jobs;
   rs.job_count = job_count;
   rs.issued = rs.consumed = 0;
@@ -169,14 +171,15 @@ __device__ inline void stream_init(RowStream &rs, uint8_t *ring_base, StreamShar
     rs.issue_cursor = cursor_at_start(rs.issue);
   }
   if ((threadIdx.x & 31u) == 0) {
-    for (uint32_t s = 0; s < kStreamSlots; ++s) mbar_init(&rs.bars[s], 1);
+    for (uint32_t s = 0; s < SLOTS; ++s) mbar_init(&rs.bars[s], 1);
     mbar_init_fence();
   }
   __syncwarp();
 }
 
 // Issues chunks, crossing into later jobs, while ring slots are free (at most `depth` in flight).
-__device__ __forceinline__ void stream_fill(RowStream &rs, uint32_t depth = kStreamSlots) {
+template <uint32_t SLOTS = kStreamSlots>
+__device__ __forceinline__ void stream_fill(RowStream &rs, uint32_t depth = SLOTS) {
   if (rs.dead) return;
   while (rs.issue_job < rs.job_count && rs.issued - rs.consumed < depth) {
     if (rs.issue_cursor.pos >= rs.issue.end) {
@@ -189,7 +192,7 @@ __device__ __forceinline__ void stream_fill(RowStream &rs, uint32_t depth = kStr
     }
     uint32_t pos, row_end;
     const uint32_t len = cursor_next(rs.issue, rs.issue_cursor, &pos, &row_end);
-    const uint32_t slot = rs.issued % kStreamSlots;
+    const uint32_t slot = rs.issued % SLOTS;
     if ((threadIdx.x & 31u) == 0) {
       mbar_arrive_expect_tx(&rs.bars[slot], len);
       tma_load_1d_hint(rs.ring + slot * kChunkBytes, rs.issue.base + pos, len, &rs.bars[slot], rs.policy);
@@ -284,7 +287,7 @@ __device__ __forceinline__ float2 dot_piece_x2(const uint8_t *wp, const float4 *
 // before the block's previous synchronisation) receives the total of every row
 // that lies wholly inside this warp's range; partial rows go to sh.edge.
 // XF32: `x` points at fp32 activations instead of bf16 ones.
-template <bool XF32 = false>
+template <bool XF32 = false, uint32_t SLOTS = kStreamSlots>
 __device__ __forceinline__ void stream_consume(RowStream &rs, StreamShared &sh, uint32_t index,
                                                const void *x, float *row_total,
                                                uint32_t *error_word) {
@@ -301,9 +304,9 @@ __device__ __forceinline__ void stream_consume(RowStream &rs, StreamShared &sh, 
   while (cur.pos < job.end) {
     uint32_t pos, row_end, row;
     const uint32_t len = cursor_next(job, cur, &pos, &row_end, &row);
-    stream_fill(rs);
-    const uint32_t slot = rs.consumed % kStreamSlots;
-    const uint32_t parity = (rs.consumed / kStreamSlots) & 1u;
+    stream_fill<SLOTS>(rs);
+    const uint32_t slot = rs.consumed % SLOTS;
+    const uint32_t parity = (rs.consumed / SLOTS) & 1u;
     if (!rs.dead && !mbar_wait_bounded(&rs.bars[slot], parity)) {
       rs.dead = true;
       rs.drain_from = rs.consumed;
@@ -398,7 +401,7 @@ __device__ __forceinline__ void stream_consume(RowStream &rs, StreamShared &sh, 
     rs.consumed += 1;
   }
   // keep the ring full while the block goes on to its next phase
-  stream_fill(rs);
+  stream_fill<SLOTS>(rs);
 }
 
 // After the block has synchronised behind stream_consume: row r's total with
@@ -416,10 +419,11 @@ __device__ __forceinline__ float stream_row_total(const StreamShared &sh, const 
 
 // After a timeout: give copies still in flight one more bounded chance to land
 // before the block's shared memory is released.
+template <uint32_t SLOTS = kStreamSlots>
 __device__ inline void stream_drain(RowStream &rs) {
   if (!rs.dead) return;
   for (uint32_t c = rs.drain_from; c < rs.drain_to; ++c) {
-    mbar_wait_bounded(&rs.bars[c % kStreamSlots], (c / kStreamSlots) & 1u);
+    mbar_wait_bounded(&rs.bars[c % SLOTS], (c / SLOTS) & 1u);
   }
 }
 

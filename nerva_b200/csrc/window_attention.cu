@@ -25,7 +25,6 @@ namespace {
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr uint32_t kPageTokens = NERVA_KV_CACHE_BLOCK_TOKENS;
 constexpr uint32_t kTile = 32;             // tokens of one score tile: one per lane
-constexpr uint32_t kWarps = 8;
 constexpr uint32_t kHeadsPerBlock = 8;
 constexpr uint32_t kMaxSmem = 227u * 1024u;
 
@@ -73,18 +72,26 @@ __device__ __forceinline__ float dot_piece(const uint16_t *k, const float *q, fl
   return fmaf(bf16x2_hi(w.w), b.w, acc);
 }
 
-// One warp: the head in v[0 .. qk_dim) (shared memory) is rotated and normalised in place.
-__device__ __forceinline__ void rotate_and_norm(float *v, const WindowAttentionShape &s, uint32_t position) {
+// (sin, cos) of pair i at a position, with the magnitude of a scaled rotation.
+__device__ __forceinline__ float2 rotation(const WindowAttentionShape &s, uint32_t position, uint32_t i) {
+  float2 t;
+  sincosf(static_cast<float>(position) * s.frequency[i], &t.x, &t.y);
+  t.x *= s.rotary_magnitude;
+  t.y *= s.rotary_magnitude;
+  return t;
+}
+
+// One warp: the head in v[0 .. qk_dim) (shared memory) is rotated (turn(i): rotation of pair i) and
+// normalised in place.
+template <class Turn>
+__device__ __forceinline__ void rotate_and_norm(float *v, const WindowAttentionShape &s, Turn turn) {
   const uint32_t lane = threadIdx.x & 31u;
   __syncwarp();
   for (uint32_t i = lane; i < s.rotary_pairs; i += 32u) {
-    float sn, cs;
-    sincosf(static_cast<float>(position) * s.frequency[i], &sn, &cs);
-    sn *= s.rotary_magnitude;
-    cs *= s.rotary_magnitude;
+    const float2 t = turn(i);
     const float a = v[i], b = v[i + s.rotary_pairs];
-    v[i] = a * cs - b * sn;
-    v[i + s.rotary_pairs] = b * cs + a * sn;
+    v[i] = a * t.y - b * t.x;
+    v[i + s.rotary_pairs] = b * t.y + a * t.x;
   }
   __syncwarp();
   if (s.qk_norm == 0) return;
@@ -117,7 +124,7 @@ __global__ void __launch_bounds__(32) window_publish_kernel(WindowAttentionParam
   float *row = p.qkv + static_cast<uint64_t>(blockIdx.y) * p.qkv_stride;
   float *src = row + (query ? 0u : s.heads * s.qk_dim) + h * s.qk_dim;
   for (uint32_t i = lane; i < s.qk_dim; i += 32u) head[i] = __ldcg(src + i);
-  rotate_and_norm(head, s, r.position);
+  rotate_and_norm(head, s, [&](uint32_t i) { return rotation(s, r.position, i); });
   if (query) {
     for (uint32_t i = lane; i < s.qk_dim; i += 32u) src[i] = head[i];
     return;
@@ -147,17 +154,24 @@ struct DecodeLayout {
   }
 };
 
-// Score tiles per chunk: two, or one where two stages of two tiles do not fit shared memory.
+// Score tiles per chunk of the row form: two, or one where two stages of two tiles do not fit shared memory.
 template <class T>
-__host__ __device__ inline uint32_t chunk_tiles(const WindowAttentionShape &s) {
-  return DecodeLayout<T>(s, 2u * kTile).total <= kMaxSmem - 1024u ? 2u : 1u;
+inline uint32_t chunk_tiles(const WindowAttentionShape &s, bool rows) {
+  if (!rows) return 1u;
+  return DecodeLayout<T>(s, 2u * kTile).total <= kMaxSmem - 2048u ? 2u : 1u;
 }
 
 // PAIRS: value pairs (2 lane + 64 j, +1) a lane accumulates; v_pad <= 64 PAIRS.
+// A warp has at most two work items: heads x tiles <= 2 warps.  The lone step runs small blocks (4 warps,
+// one tile per chunk) that fit beside a weight-streaming block on the same SM.
+template <bool ROWS>
+constexpr uint32_t decode_warps() { return ROWS ? 8u : 4u; }
 template <class T, uint32_t PAIRS, bool ROWS>
-__global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAttentionParams p, uint32_t tiles) {
+__global__ void __launch_bounds__(decode_warps<ROWS>() * 32) window_attention_kernel(WindowAttentionParams p, uint32_t tiles) {
+  constexpr uint32_t kWarps = decode_warps<ROWS>();
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ uint32_t ticket;
+  __shared__ float2 turn[ROWS ? 1 : 128];  // sin and cos of the lone step's rotation
   const WindowAttentionShape &s = p.s;
   const uint32_t chunk_tokens = tiles * kTile;
   const DecodeLayout<T> layout(s, chunk_tokens);
@@ -208,9 +222,8 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   const uint32_t lo = s.window != 0 && position + 1u > s.window ? position + 1u - s.window : 0u;
   const uint32_t first_chunk = lo / chunk_tokens;
   const uint32_t chunks = (hist + chunk_tokens - 1u) / chunk_tokens - first_chunk;  // lo <= hist: never negative
-  const uint32_t per_span = (chunks + S - 1u) / S;
-  const uint32_t chunk_begin = first_chunk + (span * per_span < chunks ? span * per_span : chunks);
-  const uint32_t chunk_end = first_chunk + ((span + 1u) * per_span < chunks ? (span + 1u) * per_span : chunks);
+  const uint32_t chunk_begin = first_chunk + chunks * span / S;
+  const uint32_t chunk_end = first_chunk + chunks * (span + 1u) / S;
   const bool owns_current = !ROWS && span + 1u == S;
 
   const uint32_t k_pieces = s.qk_pad * static_cast<uint32_t>(sizeof(T)) / 16u;
@@ -250,23 +263,27 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   // cached rows were written by earlier steps: requested before the wait for this step's projection
   if (chunk_begin < chunk_end) issue(chunk_begin, 0);
   if (chunk_begin + 1u < chunk_end) issue(chunk_begin + 1u, 1);
-  if (!ROWS) pdl_wait();
+  if (!ROWS) {
+    for (uint32_t i = threadIdx.x; i < s.rotary_pairs; i += blockDim.x) turn[i] = rotation(s, position, i);
+    __syncthreads();
+    pdl_wait();
+  }
 
   const float *qkv = p.qkv + static_cast<uint64_t>(row) * p.qkv_stride;
   const float qscale = s.scale * kLog2e;
-  if (warp < hb) {
-    float *q = q_sh + warp * s.qk_pad;
-    const float *src = qkv + (head0 + warp) * s.qk_dim;
+  for (uint32_t w = warp; w < hb; w += kWarps) {
+    float *q = q_sh + w * s.qk_pad;
+    const float *src = qkv + (head0 + w) * s.qk_dim;
     for (uint32_t i = lane; i < s.qk_pad; i += 32u) q[i] = i < s.qk_dim ? __ldcg(src + i) : 0.0f;
-    if (!ROWS) rotate_and_norm(q, s, position);
+    if (!ROWS) rotate_and_norm(q, s, [&](uint32_t i) { return turn[i]; });
     __syncwarp();
     for (uint32_t i = lane; i < s.qk_dim; i += 32u) q[i] *= qscale;
   }
-  if (owns_current && warp == kWarps - 1u) {  // after its query, when the block has eight
+  if (owns_current && warp == kWarps - 1u) {  // the warp with the fewest queries
     const float *k_src = qkv + s.heads * s.qk_dim + kvh * s.qk_dim;
     const float *v_src = qkv + (s.heads + s.kv_heads) * s.qk_dim + kvh * s.v_dim;
     for (uint32_t i = lane; i < s.qk_pad; i += 32u) k_new[i] = i < s.qk_dim ? __ldcg(k_src + i) : 0.0f;
-    rotate_and_norm(k_new, s, position);
+    rotate_and_norm(k_new, s, [&](uint32_t i) { return turn[i]; });
     __syncwarp();
     uint32_t page = table[position / kPageTokens];
     if (page >= page_count) {
@@ -340,7 +357,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
           for (uint32_t i = 0; i < 2u * PAIRS; ++i) acc[u][i] *= corr;
           p_sh[item * kTile + lane] = pr;
           __syncwarp();
-#pragma unroll 4
+#pragma unroll 8
           for (uint32_t t = t0; t < t1; ++t) {
             const float pt = p_sh[item * kTile + t];
             const T *v_row = reinterpret_cast<const T *>(v_stage + (tile * kTile + t) * layout.v_row);
@@ -363,7 +380,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   }
   __syncthreads();  // q, k_new, v_new are visible also when no chunk ran; the stages are idle
 
-  // every item's state through the stage memory, then warp w finishes head w
+  // every item's state through the stage memory, then a warp finishes each head
   float *handoff = reinterpret_cast<float *>(smem);  // [item][32 lanes][2 PAIRS + 2]
   constexpr uint32_t kRec = 2u * PAIRS + 2u;
 #pragma unroll
@@ -379,8 +396,8 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   }
   __syncthreads();
   const uint64_t out_row = static_cast<uint64_t>(row) * p.out_stride;
-  if (warp < hb) {
-    const uint32_t h = head0 + warp;
+  for (uint32_t w = warp; w < hb; w += kWarps) {
+    const uint32_t h = head0 + w;
     float m = -INFINITY, l = 0.0f, a[2u * PAIRS];
 #pragma unroll
     for (uint32_t i = 0; i < 2u * PAIRS; ++i) a[i] = 0.0f;
@@ -393,11 +410,11 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
       m = m2;
     };
     for (uint32_t tile = 0; tile < tiles; ++tile) {
-      const float *src = handoff + ((tile * hb + warp) * 32u + lane) * kRec;
+      const float *src = handoff + ((tile * hb + w) * 32u + lane) * kRec;
       if (src[2u * PAIRS + 1u] > 0.0f) fold(src[2u * PAIRS], src[2u * PAIRS + 1u], src);
     }
     if (owns_current) {
-      const float *q = q_sh + warp * s.qk_pad;
+      const float *q = q_sh + w * s.qk_pad;
       float dot = 0.0f;
       for (uint32_t i = lane; i < s.qk_pad; i += 32u) dot = fmaf(q[i], k_new[i], dot);
       dot = warp_sum(dot);
@@ -443,8 +460,8 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   }
   __syncthreads();
   if (ticket != S - 1u) return;
-  if (warp < hb) {
-    const uint32_t h = head0 + warp;
+  for (uint32_t hw = warp; hw < hb; hw += kWarps) {
+    const uint32_t h = head0 + hw;
     const uint64_t slot0 = (static_cast<uint64_t>(row) * s.heads + h) * S;
     float ms = -INFINITY, ls = 0.0f;
     if (lane < S) {
@@ -711,15 +728,16 @@ uint32_t decode_smem(const WindowAttentionShape &s, uint32_t tiles) {
 
 template <class T>
 cudaError_t launch_decode(cudaStream_t stream, const WindowAttentionParams &p) {
-  const uint32_t tiles = chunk_tiles<T>(p.s);
+  const uint32_t tiles = chunk_tiles<T>(p.s, p.rows != nullptr);
   const uint32_t bytes = decode_smem<T>(p.s, tiles);
-  if (bytes == 0 || bytes > kMaxSmem - 1024u) return cudaErrorNotSupported;
+  if (bytes == 0 || bytes > kMaxSmem - 2048u) return cudaErrorNotSupported;
   const uint32_t group = p.s.heads / p.s.kv_heads;
   const uint32_t subs = (group + kHeadsPerBlock - 1u) / kHeadsPerBlock;
   const bool rows = p.rows != nullptr;
   const dim3 grid(p.s.kv_heads * subs * p.splits, rows ? p.row_count : 1u);
   return launch_with_pdl(rows ? decode_kernel<T, true>(p.s.v_pad) : decode_kernel<T, false>(p.s.v_pad), grid,
-                         dim3(kWarps * 32), bytes, stream, p.pdl != 0, p, tiles);
+                         dim3((rows ? decode_warps<true>() : decode_warps<false>()) * 32u), bytes, stream, p.pdl != 0, p,
+                         tiles);
 }
 
 }  // namespace
@@ -728,18 +746,23 @@ bool window_attention_supported(const WindowAttentionShape &s, bool f32) {
   if (s.heads == 0 || s.kv_heads == 0 || s.heads % s.kv_heads != 0 || s.qk_dim == 0 || s.v_dim == 0 || s.qk_pad > 256u ||
       s.v_pad > 256u || s.qk_pad % 16u != 0 || s.v_pad % 16u != 0 || 2u * s.rotary_pairs > s.qk_dim)
     return false;
-  const uint32_t bytes = f32 ? decode_smem<float>(s, chunk_tiles<float>(s)) : decode_smem<uint16_t>(s, chunk_tiles<uint16_t>(s));
-  return bytes != 0 && bytes <= kMaxSmem - 1024u && (f32 || PrefillLayout(s).total <= kMaxSmem - 1024u);
+  const uint32_t bytes = f32 ? decode_smem<float>(s, chunk_tiles<float>(s, true))
+                             : decode_smem<uint16_t>(s, chunk_tiles<uint16_t>(s, true));
+  const uint32_t lone = f32 ? decode_smem<float>(s, 1) : decode_smem<uint16_t>(s, 1);
+  return bytes != 0 && lone != 0 && bytes <= kMaxSmem - 2048u && lone <= kMaxSmem - 2048u && (f32 || PrefillLayout(s).total <= kMaxSmem - 2048u);
 }
 
-// Spans for a step whose context is at most target_context: one 64-token chunk per block up to
-// kWindowMaxSplits, in powers of two so that a growing context re-captures the step rarely.
+// Spans for a step whose context is at most target_context: one 32-token tile per block up to
+// kWindowMaxSplits, in powers of two so that a growing context re-captures the step rarely, but never
+// more than a full window (which may begin and end inside a tile) needs.
 uint32_t window_attention_splits(uint32_t target_context, uint32_t window) {
-  uint32_t keys = target_context;
-  if (window != 0 && window + 64u < keys) keys = window + 64u;  // a window may start inside a chunk
-  const uint32_t chunks = (keys + 63u) / 64u;
+  const uint32_t tiles = (target_context + kTile - 1u) / kTile;
   uint32_t s = 1;
-  while (s < chunks && s < kWindowMaxSplits) s <<= 1;
+  while (s < tiles && s < kWindowMaxSplits) s <<= 1;
+  if (window != 0) {
+    const uint32_t most = (window + 2u * kTile - 2u) / kTile;
+    if (s > most) s = most;
+  }
   return s;
 }
 
@@ -747,7 +770,7 @@ cudaError_t configure_window_attention() {
   cudaError_t err = cudaSuccess;
   auto set = [&](const void *kernel) {
     if (err == cudaSuccess)
-      err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kMaxSmem - 1024u));
+      err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kMaxSmem - 2048u));
   };
   for (uint32_t v : {64u, 128u, 256u}) {
     set(reinterpret_cast<const void *>(decode_kernel<uint16_t, false>(v)));
