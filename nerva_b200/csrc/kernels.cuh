@@ -412,9 +412,10 @@ struct WindowAttentionParams {
   const struct FusedAttentionRow *rows;
   uint32_t row_count;
 };
-constexpr uint32_t kWindowMaxSplits = 32;  // a lane per span in the merge
+constexpr uint32_t kWindowMaxSplits = 16;
 bool window_attention_supported(const WindowAttentionShape &s, bool f32);
-uint32_t window_attention_splits(uint32_t target_context, uint32_t window);
+uint32_t window_attention_splits(uint32_t target_context, uint32_t window);  // the lone step
+uint32_t window_rows_splits(const WindowAttentionShape &s, uint32_t rows, uint32_t longest_context, uint32_t sm_count);
 cudaError_t configure_window_attention();
 // q/k rotation and norm, K/V rows into the cache, for the rows of a block step.
 cudaError_t launch_window_publish(cudaStream_t stream, const WindowAttentionParams &p);

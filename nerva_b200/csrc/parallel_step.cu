@@ -429,9 +429,7 @@ cudaError_t enqueue_parallel_block_layers(Session *s, const ParallelBlock &b, ui
       if (b.one_session && b.rows >= kPrefillTileMinRows && !plan.f32) {
         err = launch_window_prefill(b.stream, a);
       } else {
-        // rows x KV heads fill the machine already: as few spans as keep about four blocks per SM
-        const uint32_t machine = 4u * s->sm_count / (b.rows * l.shape.kv_heads);
-        a.splits = std::min(window_attention_splits(b.longest, l.shape.window), std::max(machine, 1u));
+        a.splits = window_rows_splits(l.shape, b.rows, b.longest, s->sm_count);
         err = launch_window_attention(b.stream, a);
       }
     }

@@ -4,10 +4,13 @@
 // alike here), then an optional weightless RMS norm of q and k, softmax over the keys in the window.
 //
 //   window_attention_kernel   one query token per row.  The lone decode step (ROWS = false) prepares
-//                             q, appends the new K/V row and attends in one launch; block rows
-//                             (ROWS = true) find both done by window_publish_kernel.  Grid (KV head x
-//                             group of 8 query heads x span, row); the spans divide the window, not
-//                             the context.  fp32 arithmetic on the CUDA cores, K/V in shared memory.
+//                             q, appends the new K/V row and attends in one launch; block rows of an
+//                             fp32 session (ROWS = true) find both done by window_publish_kernel.
+//                             Grid (KV head x group of 8 query heads x span, row); the spans divide
+//                             the window, not the context.  fp32 arithmetic on the CUDA cores, K/V in
+//                             shared memory.
+//   window_rows_kernel        the block rows of a bf16 session (packed decode step, short portions) on
+//                             the tensor pipe, same grid.
 //   window_prefill_kernel     64 (position, head) rows of one KV head against 64-token tiles on the
 //                             tensor pipe (mma.sync, bf16), flash-attention style: scores and softmax
 //                             stay in registers.  Queries and probabilities are split into a bf16
@@ -108,23 +111,32 @@ __device__ __forceinline__ uint64_t cache_row(uint32_t page, uint32_t token, uin
   return ((static_cast<uint64_t>(page) * kPageTokens + token % kPageTokens) * kv_heads + kvh) * width;
 }
 
-// Grid (heads + kv_heads, rows), one warp each: a query head is prepared in place, a KV head's K and
-// V go to the cache.
+// Grid ((heads + kv_heads) / 8, rows), a warp per head: a query head is prepared in place, a KV head's K
+// and V go to the cache.
+constexpr uint32_t kPublishWarps = 8;
 template <class T>
-__global__ void __launch_bounds__(32) window_publish_kernel(WindowAttentionParams p) {
-  __shared__ float head[256];
+__global__ void __launch_bounds__(kPublishWarps * 32) window_publish_kernel(WindowAttentionParams p) {
+  __shared__ float heads[kPublishWarps][256];
+  __shared__ float2 turn[128];
   pdl_trigger();
-  pdl_wait();
   const WindowAttentionShape &s = p.s;
   const FusedAttentionRow &r = p.rows[blockIdx.y];
-  if (r.position >= r.max_context) return;
-  const uint32_t lane = threadIdx.x;
-  const bool query = blockIdx.x < s.heads;
-  const uint32_t h = query ? blockIdx.x : blockIdx.x - s.heads;
+  if (r.position >= r.max_context) {
+    pdl_wait();
+    return;
+  }
+  for (uint32_t i = threadIdx.x; i < s.rotary_pairs; i += blockDim.x) turn[i] = rotation(s, r.position, i);
+  __syncthreads();
+  pdl_wait();
+  const uint32_t lane = threadIdx.x & 31u, unit = blockIdx.x * kPublishWarps + (threadIdx.x >> 5);
+  if (unit >= s.heads + s.kv_heads) return;
+  float *head = heads[threadIdx.x >> 5];
+  const bool query = unit < s.heads;
+  const uint32_t h = query ? unit : unit - s.heads;
   float *row = p.qkv + static_cast<uint64_t>(blockIdx.y) * p.qkv_stride;
   float *src = row + (query ? 0u : s.heads * s.qk_dim) + h * s.qk_dim;
   for (uint32_t i = lane; i < s.qk_dim; i += 32u) head[i] = __ldcg(src + i);
-  rotate_and_norm(head, s, [&](uint32_t i) { return rotation(s, r.position, i); });
+  rotate_and_norm(head, s, [&](uint32_t i) { return turn[i]; });
   if (query) {
     for (uint32_t i = lane; i < s.qk_dim; i += 32u) src[i] = head[i];
     return;
@@ -159,6 +171,60 @@ template <class T>
 inline uint32_t chunk_tiles(const WindowAttentionShape &s, bool rows) {
   if (!rows) return 1u;
   return DecodeLayout<T>(s, 2u * kTile).total <= kMaxSmem - 2048u ? 2u : 1u;
+}
+
+// After every thread's partials of its block are stored: the block that draws the last ticket of its
+// heads merges their spans (one acquire-release atomic between the block's barriers orders the
+// partials).  Called by the whole block.
+template <class T, uint32_t PAIRS>
+__device__ __forceinline__ void merge_spans(const WindowAttentionParams &p, uint32_t row, uint32_t head0, uint32_t hb,
+                                            uint32_t *ticket) {
+  const WindowAttentionShape &s = p.s;
+  const uint32_t lane = threadIdx.x & 31u, warps = blockDim.x >> 5, S = p.splits;
+  uint32_t *counter = p.tickets + static_cast<uint64_t>(row) * s.heads + head0;
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    uint32_t drawn;
+    asm volatile("atom.acq_rel.gpu.global.add.u32 %0, [%1], 1;" : "=r"(drawn) : "l"(counter) : "memory");
+    *ticket = drawn;
+  }
+  __syncthreads();
+  if (*ticket != S - 1u) return;
+  for (uint32_t hw = threadIdx.x >> 5; hw < hb; hw += warps) {
+    const uint32_t h = head0 + hw;
+    const uint64_t slot0 = (static_cast<uint64_t>(row) * s.heads + h) * S;
+    float ms = -INFINITY, ls = 0.0f;
+    if (lane < S) {
+      ms = __ldcg(p.partial_m + slot0 + lane);
+      ls = __ldcg(p.partial_l + slot0 + lane);
+    }
+    const float m = warp_max(ls > 0.0f ? ms : -INFINITY);
+    float w = ls > 0.0f ? exp2f(ms - m) : 0.0f;
+    w /= warp_sum(ls * w);
+    float a[2u * PAIRS];
+#pragma unroll
+    for (uint32_t i = 0; i < 2u * PAIRS; ++i) a[i] = 0.0f;
+#pragma unroll 8
+    for (uint32_t i = 0; i < S; ++i) {
+      const float wi = __shfl_sync(0xffffffffu, w, i);
+#pragma unroll
+      for (uint32_t j = 0; j < PAIRS; ++j) {
+        const uint32_t d = 2u * lane + 64u * j;
+        if (d < s.v_pad) {
+          const float2 v = __ldcg(reinterpret_cast<const float2 *>(p.partial_acc + (slot0 + i) * s.v_pad + d));
+          a[2u * j] = fmaf(v.x, wi, a[2u * j]);
+          a[2u * j + 1u] = fmaf(v.y, wi, a[2u * j + 1u]);
+        }
+      }
+    }
+    T *out = reinterpret_cast<T *>(p.out) + static_cast<uint64_t>(row) * p.out_stride + h * s.v_dim;
+#pragma unroll
+    for (uint32_t i = 0; i < 2u * PAIRS; ++i) {
+      const uint32_t d = 2u * lane + 64u * (i / 2u) + (i & 1u);
+      if (d < s.v_dim) to_cache(out + d, a[i]);
+    }
+  }
+  if (threadIdx.x == 0) *counter = 0;  // ready for the next launch
 }
 
 // PAIRS: value pairs (2 lane + 64 j, +1) a lane accumulates; v_pad <= 64 PAIRS.
@@ -449,79 +515,260 @@ __global__ void __launch_bounds__(decode_warps<ROWS>() * 32) window_attention_ke
     }
   }
   if (S == 1u) return;
-  // the block that draws the last ticket of its heads merges their spans (one acquire-release atomic
-  // between the block's barriers orders the partials)
-  uint32_t *counter = p.tickets + static_cast<uint64_t>(row) * s.heads + head0;
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    uint32_t drawn;
-    asm volatile("atom.acq_rel.gpu.global.add.u32 %0, [%1], 1;" : "=r"(drawn) : "l"(counter) : "memory");
-    ticket = drawn;
+  merge_spans<T, PAIRS>(p, row, head0, hb, &ticket);
+}
+
+// ------------------------------------------------------- block rows on the tensor pipe ----
+// One query token per row, bf16 cache.  A block serves up to eight query heads of one KV head over one
+// span of pages; each of its four warps walks its own pages through a private ring of cp.async stages
+// (no block barrier in the loop).  The sixteen rows of the MMA hold the heads twice: rows 0..7 the bf16
+// roundings of the queries (and of the probabilities), rows 8..15 what the rounding lost; the accumulator
+// fragment puts rows r and r + 8 into one thread, which adds them.
+constexpr uint32_t kRowWarps = 4;
+constexpr uint32_t kRowStages = 3;
+
+struct RowLayout {
+  uint32_t k_row, v_row, stage, ring, total;
+  __host__ __device__ explicit RowLayout(const WindowAttentionShape &s) {
+    k_row = s.qk_pad * 2u + 16u;  // an odd number of 16-byte pieces: ldmatrix without bank conflicts
+    v_row = s.v_pad * 2u + 16u;
+    stage = kPageTokens * (k_row + v_row);
+    ring = kRowStages * stage;
+    total = kRowWarps * ring + 16u * k_row;  // rings | q: 8 rows high parts, 8 rows low parts
   }
-  __syncthreads();
-  if (ticket != S - 1u) return;
-  for (uint32_t hw = warp; hw < hb; hw += kWarps) {
-    const uint32_t h = head0 + hw;
-    const uint64_t slot0 = (static_cast<uint64_t>(row) * s.heads + h) * S;
-    float ms = -INFINITY, ls = 0.0f;
-    if (lane < S) {
-      ms = __ldcg(p.partial_m + slot0 + lane);
-      ls = __ldcg(p.partial_l + slot0 + lane);
-    }
-    const float m = warp_max(ls > 0.0f ? ms : -INFINITY);
-    float w = ls > 0.0f ? exp2f(ms - m) : 0.0f;
-    w /= warp_sum(ls * w);
-    float a[2u * PAIRS];
+};
+
+template <uint32_t PAIRS>
+__global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAttentionParams p) {
+  constexpr uint32_t NT = 8u * PAIRS;  // value n-tiles of 8 dims: v_pad <= 64 PAIRS
+  extern __shared__ __align__(128) uint8_t smem[];
+  __shared__ uint32_t ticket;
+  const WindowAttentionShape &s = p.s;
+  const RowLayout L(s);
+  uint8_t *q_sh = smem + kRowWarps * L.ring;
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t row = blockIdx.y;
+  const FusedAttentionRow &r = p.rows[row];
+  if (r.position >= r.max_context) return;
+  const uint16_t *keys = r.key_pages + p.key_offset, *values = r.value_pages + p.value_offset;
+  const uint32_t lane = threadIdx.x & 31u, warp = threadIdx.x >> 5;
+  const uint32_t group = s.heads / s.kv_heads;
+  const uint32_t subs = (group + kHeadsPerBlock - 1u) / kHeadsPerBlock;
+  const uint32_t S = p.splits;
+  const uint32_t unit = blockIdx.x / S, span = blockIdx.x - unit * S;
+  const uint32_t kvh = unit / subs, sub = unit - kvh * subs;
+  const uint32_t head0 = kvh * group + sub * kHeadsPerBlock;
+  const uint32_t left_heads = group - sub * kHeadsPerBlock;
+  const uint32_t hb = left_heads < kHeadsPerBlock ? left_heads : kHeadsPerBlock;
+  const uint32_t hist = r.position + 1u;
+  const uint32_t lo = s.window != 0 && hist > s.window ? hist - s.window : 0u;
+  const uint32_t first_page = lo / kPageTokens;
+  const uint32_t pages = (hist + kPageTokens - 1u) / kPageTokens - first_page;
+  const uint32_t page_begin = first_page + pages * span / S, page_end = first_page + pages * (span + 1u) / S;
+  const uint32_t first = page_begin + warp;
+  const uint32_t my_pages = first < page_end ? (page_end - first + kRowWarps - 1u) / kRowWarps : 0u;
+
+  uint8_t *ring = smem + warp * L.ring;
+  const uint32_t k_pieces = s.qk_pad / 8u, v_pieces = s.v_pad / 8u, row_pieces = k_pieces + v_pieces;
+  auto issue = [&](uint32_t i) {  // one commit group per page, also when there is none left
+    if (i < my_pages) {
+      const uint32_t logical = first + i * kRowWarps;
+      uint32_t page = r.page_table[logical];
+      if (page >= r.page_count) {
+        report_error(r.error_word, kErrPageOutOfRange);
+        page = 0;
+      }
+      uint8_t *k_stage = ring + (i % kRowStages) * L.stage;
+      uint8_t *v_stage = k_stage + kPageTokens * L.k_row;
+      const uint32_t token0 = logical * kPageTokens;
+      // a lane takes one 16-byte piece of the K or V row of all sixteen tokens
+      for (uint32_t piece = lane; piece < row_pieces; piece += 32u) {
+        const bool is_k = piece < k_pieces;
+        const uint16_t *src = is_k ? keys + cache_row(page, 0, s.kv_heads, kvh, s.qk_pad) + piece * 8u
+                                   : values + cache_row(page, 0, s.kv_heads, kvh, s.v_pad) + (piece - k_pieces) * 8u;
+        const uint32_t src_step = s.kv_heads * (is_k ? s.qk_pad : s.v_pad);
+        uint8_t *dst = is_k ? k_stage + piece * 16u : v_stage + (piece - k_pieces) * 16u;
+        const uint32_t dst_step = is_k ? L.k_row : L.v_row;
+        if (token0 >= lo && token0 + kPageTokens <= hist) {
 #pragma unroll
-    for (uint32_t i = 0; i < 2u * PAIRS; ++i) a[i] = 0.0f;
-#pragma unroll 4
-    for (uint32_t i = 0; i < S; ++i) {
-      const float wi = __shfl_sync(0xffffffffu, w, i);
+          for (uint32_t t = 0; t < kPageTokens; ++t) cp_async_16(dst + t * dst_step, src + t * src_step);
+        } else {  // tokens outside the window are filled with zeros
 #pragma unroll
-      for (uint32_t j = 0; j < PAIRS; ++j) {
-        const uint32_t d = 2u * lane + 64u * j;
-        if (d < s.v_pad) {
-          const float2 v = __ldcg(reinterpret_cast<const float2 *>(p.partial_acc + (slot0 + i) * s.v_pad + d));
-          a[2u * j] = fmaf(v.x, wi, a[2u * j]);
-          a[2u * j + 1u] = fmaf(v.y, wi, a[2u * j + 1u]);
+          for (uint32_t t = 0; t < kPageTokens; ++t)
+            cp_async_zfill<16>(dst + t * dst_step, src + t * src_step, token0 + t >= lo && token0 + t < hist);
         }
       }
     }
+    cp_async_commit();
+  };
+  issue(0);
+  issue(1);
+
+  const float qscale = s.scale * kLog2e;
+  const float *q_in = p.qkv + static_cast<uint64_t>(row) * p.qkv_stride + head0 * s.qk_dim;
+  const uint32_t q_pairs = s.qk_pad / 2u;
+  for (uint32_t i = threadIdx.x; i < kHeadsPerBlock * q_pairs; i += blockDim.x) {
+    const uint32_t h = i / q_pairs, d = 2u * (i - h * q_pairs);
+    const float a = h < hb && d < s.qk_dim ? __ldcg(q_in + h * s.qk_dim + d) * qscale : 0.0f;
+    const float b = h < hb && d + 1u < s.qk_dim ? __ldcg(q_in + h * s.qk_dim + d + 1u) * qscale : 0.0f;
+    *reinterpret_cast<uint32_t *>(q_sh + h * L.k_row + d * 2u) = pack_bf16_hi(a, b);
+    *reinterpret_cast<uint32_t *>(q_sh + (h + 8u) * L.k_row + d * 2u) = pack_bf16_lo(a, b);
+  }
+  __syncthreads();
+
+  const uint32_t t4 = lane & 3u, g = lane >> 2;
+  const uint32_t q_addr = smem_addr(q_sh) + ((lane & 7u) + 8u * ((lane >> 3) & 1u)) * L.k_row + (lane >> 4) * 16u;
+  const uint32_t k_off = ((lane & 7u) + 8u * (lane >> 4)) * L.k_row + ((lane >> 3) & 1u) * 16u;
+  const uint32_t v_off = ((lane & 7u) + 8u * ((lane >> 3) & 1u)) * L.v_row + (lane >> 4) * 16u;
+  float m_run = -INFINITY, l_run = 0.0f;
+  float o[NT][4];
 #pragma unroll
-    for (uint32_t i = 0; i < 2u * PAIRS; ++i) {
-      const uint32_t d = 2u * lane + 64u * (i / 2u) + (i & 1u);
-      if (d < s.v_dim) to_cache(reinterpret_cast<T *>(p.out) + out_row + h * s.v_dim + d, a[i]);
+  for (uint32_t n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
+  for (uint32_t i = 0; i < my_pages; ++i) {
+    issue(i + 2u);
+    cp_async_wait<2>();
+    __syncwarp();
+    const uint32_t k_base = smem_addr(ring + (i % kRowStages) * L.stage);
+    const uint32_t v_base = k_base + kPageTokens * L.k_row;
+    const uint32_t token0 = (first + i * kRowWarps) * kPageTokens;
+    float sc[2][4];
+#pragma unroll
+    for (uint32_t n = 0; n < 2u; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.0f;
+#pragma unroll 4
+    for (uint32_t ks = 0; ks < s.qk_pad / 16u; ++ks) {
+      uint32_t qa[4], kb[4];
+      ldmatrix_x4(qa, q_addr + ks * 32u);
+      ldmatrix_x4(kb, k_base + k_off + ks * 32u);
+      mma_bf16(sc[0], qa, kb[0], kb[1]);
+      mma_bf16(sc[1], qa, kb[2], kb[3]);
+    }
+    // head g's scores of tokens 2t, 2t + 1 and 8 + 2t, 9 + 2t
+    float v[4] = {sc[0][0] + sc[0][2], sc[0][1] + sc[0][3], sc[1][0] + sc[1][2], sc[1][1] + sc[1][3]};
+#pragma unroll
+    for (uint32_t j = 0; j < 4u; ++j) {
+      const uint32_t token = token0 + 8u * (j >> 1) + 2u * t4 + (j & 1u);
+      if (token < lo || token >= hist) v[j] = -INFINITY;
+    }
+    float m_page = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
+    m_page = fmaxf(m_page, __shfl_xor_sync(0xffffffffu, m_page, 1));
+    m_page = fmaxf(m_page, __shfl_xor_sync(0xffffffffu, m_page, 2));
+    const float m_new = fmaxf(m_run, m_page);  // every page of the span has a visible token: finite
+    const float corr = exp2f(m_run - m_new);
+    m_run = m_new;
+#pragma unroll
+    for (uint32_t j = 0; j < 4u; ++j) v[j] = exp2f(v[j] - m_new);
+    l_run = l_run * corr + ((v[0] + v[1]) + (v[2] + v[3]));  // this thread's share; the quad is summed at the end
+#pragma unroll
+    for (uint32_t n = 0; n < NT; ++n) {
+      o[n][0] *= corr;
+      o[n][1] *= corr;
+      o[n][2] *= corr;
+      o[n][3] *= corr;
+    }
+    const uint32_t pa[4] = {pack_bf16_hi(v[0], v[1]), pack_bf16_lo(v[0], v[1]), pack_bf16_hi(v[2], v[3]),
+                            pack_bf16_lo(v[2], v[3])};
+#pragma unroll
+    for (uint32_t np = 0; np < NT / 2u; ++np) {
+      if (np * 16u < s.v_pad) {
+        uint32_t vb[4];
+        ldmatrix_x4_trans(vb, v_base + v_off + np * 32u);
+        mma_bf16(o[2u * np], pa, vb[0], vb[1]);
+        mma_bf16(o[2u * np + 1u], pa, vb[2], vb[3]);
+      }
+    }
+    __syncwarp();  // the stage is free for the copy the next iteration issues
+  }
+  cp_async_wait<0>();
+  l_run += __shfl_xor_sync(0xffffffffu, l_run, 1);
+  l_run += __shfl_xor_sync(0xffffffffu, l_run, 2);
+  __syncthreads();
+  // the warps' states through the ring memory: [warp][head][v_pad | m | l]
+  float *merge = reinterpret_cast<float *>(smem);
+  const uint32_t rec = s.v_pad + 2u;
+  if (g < hb) {
+    float *dst = merge + (warp * kHeadsPerBlock + g) * rec;
+#pragma unroll
+    for (uint32_t n = 0; n < NT; ++n) {
+      if (n * 8u < s.v_pad) {
+        dst[n * 8u + 2u * t4] = o[n][0] + o[n][2];
+        dst[n * 8u + 2u * t4 + 1u] = o[n][1] + o[n][3];
+      }
+    }
+    if (t4 == 0) {
+      dst[s.v_pad] = m_run;
+      dst[s.v_pad + 1u] = l_run;
     }
   }
-  if (threadIdx.x == 0) *counter = 0;  // ready for the next launch
+  __syncthreads();
+  for (uint32_t idx = threadIdx.x; idx < hb * s.v_pad; idx += blockDim.x) {
+    const uint32_t h = idx / s.v_pad, d = idx - h * s.v_pad;
+    float m = -INFINITY, a = 0.0f, l = 0.0f;
+    for (uint32_t w = 0; w < kRowWarps; ++w) m = fmaxf(m, merge[(w * kHeadsPerBlock + h) * rec + s.v_pad]);
+    for (uint32_t w = 0; w < kRowWarps; ++w) {
+      const float *src = merge + (w * kHeadsPerBlock + h) * rec;
+      if (src[s.v_pad + 1u] > 0.0f) {
+        const float c = exp2f(src[s.v_pad] - m);
+        a = fmaf(src[d], c, a);
+        l = fmaf(src[s.v_pad + 1u], c, l);
+      }
+    }
+    if (S == 1u) {
+      if (d < s.v_dim)
+        reinterpret_cast<uint16_t *>(p.out)[static_cast<uint64_t>(row) * p.out_stride + (head0 + h) * s.v_dim + d] =
+            f32_to_bf16_bits(a / l);
+    } else {
+      const uint64_t slot = (static_cast<uint64_t>(row) * s.heads + head0 + h) * S + span;
+      p.partial_acc[slot * s.v_pad + d] = a;
+      if (d == 0) {
+        p.partial_m[slot] = m;
+        p.partial_l[slot] = l;
+      }
+    }
+  }
+  if (S != 1u) merge_spans<uint16_t, PAIRS>(p, row, head0, hb, &ticket);
+}
+
+uint32_t rows_smem(const WindowAttentionShape &s) {
+  const RowLayout L(s);
+  const uint32_t merge = kRowWarps * kHeadsPerBlock * (s.v_pad + 2u) * 4u;
+  return merge <= kRowWarps * L.ring ? L.total : 0u;
 }
 
 // ------------------------------------------------------------------ prefill tile ----
 constexpr uint32_t kTileRows = 64;    // (position, head) rows of a block: 16 per warp
 constexpr uint32_t kKeyTile = 64;
-constexpr uint32_t kPrefillThreads = 128;
+constexpr uint32_t kPrefillThreads = 128;  // per key group
+
+// GROUPS sets of four warps share the block's queries and take every GROUPS-th key tile each; their
+// softmax states are merged at the end.  A chunk of 256 positions gives fewer blocks than SMs at eight KV
+// heads, so one set of warps would leave the SM idle while its loads and shuffles are in flight.
 
 struct PrefillLayout {
   uint32_t q_row, k_row, v_row, stage, total;  // bytes; rows are an odd number of 16-byte pieces apart
-  __host__ __device__ explicit PrefillLayout(const WindowAttentionShape &s) {
+  __host__ __device__ PrefillLayout(const WindowAttentionShape &s, uint32_t groups) {
     q_row = k_row = s.qk_pad * 2u + 16u;
     v_row = s.v_pad * 2u + 16u;
     stage = kKeyTile * (k_row + v_row);
-    total = 2u * kTileRows * q_row + 2u * stage;  // q high and low parts | two K/V stages
+    total = 2u * kTileRows * q_row + groups * 2u * stage;  // q high and low parts | two K/V stages per group
   }
 };
 
 // NT: value n-tiles of 8 dims held in registers (v_pad <= 8 NT).
-template <uint32_t NT>
-__global__ void __launch_bounds__(kPrefillThreads) window_prefill_kernel(WindowAttentionParams p) {
+template <uint32_t NT, uint32_t GROUPS>
+__global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kernel(WindowAttentionParams p) {
   extern __shared__ __align__(128) uint8_t smem[];
   const WindowAttentionShape &s = p.s;
-  const PrefillLayout L(s);
+  const PrefillLayout L(s, GROUPS);
+  const uint32_t key_group = GROUPS == 1u ? 0u : threadIdx.x / kPrefillThreads;
+  auto group_sync = [&]() {
+    asm volatile("bar.sync %0, %1;" ::"r"(1u + key_group), "n"(kPrefillThreads) : "memory");
+  };
   uint8_t *q_hi = smem, *q_lo = smem + kTileRows * L.q_row;
-  uint8_t *stages = smem + 2u * kTileRows * L.q_row;
+  uint8_t *stages = smem + 2u * kTileRows * L.q_row + key_group * 2u * L.stage;
   pdl_trigger();
   pdl_wait();
-  const uint32_t tid = threadIdx.x, lane = tid & 31u, warp = tid >> 5;
+  const uint32_t tid = threadIdx.x % kPrefillThreads, lane = tid & 31u, warp = tid >> 5;
   const uint32_t group = s.heads / s.kv_heads;
   const uint32_t kvh = blockIdx.y;
   const uint32_t total_rows = p.row_count * group;
@@ -535,10 +782,10 @@ __global__ void __launch_bounds__(kPrefillThreads) window_prefill_kernel(WindowA
 
   const uint32_t kv_lo = s.window != 0 && pos_first + 1u > s.window ? pos_first + 1u - s.window : 0u;
   const uint32_t kv_end = pos_last + 1u;
-  const uint32_t tile_begin = kv_lo / kKeyTile, tile_end = (kv_end + kKeyTile - 1u) / kKeyTile;
+  const uint32_t tile_begin = kv_lo / kKeyTile + key_group, tile_end = (kv_end + kKeyTile - 1u) / kKeyTile;
   const uint32_t k_pieces = s.qk_pad / 8u, v_pieces = s.v_pad / 8u, row_pieces = k_pieces + v_pieces;
   auto issue = [&](uint32_t tile) {
-    uint8_t *k_stage = stages + ((tile - tile_begin) & 1u) * L.stage;
+    uint8_t *k_stage = stages + ((tile - tile_begin) / GROUPS & 1u) * L.stage;
     uint8_t *v_stage = k_stage + kKeyTile * L.k_row;
     const uint32_t first = tile * kKeyTile;
     uint32_t my_page = 0;
@@ -564,13 +811,13 @@ __global__ void __launch_bounds__(kPrefillThreads) window_prefill_kernel(WindowA
     }
     cp_async_commit();
   };
-  issue(tile_begin);
-  if (tile_begin + 1u < tile_end) issue(tile_begin + 1u);
+  if (tile_begin < tile_end) issue(tile_begin);
+  if (tile_begin + GROUPS < tile_end) issue(tile_begin + GROUPS);
 
   // queries, scaled so that the softmax runs on exp2, as a bf16 rounding and its remainder
   const float qscale = s.scale * kLog2e;
   const uint32_t q_pairs = s.qk_pad / 2u;
-  for (uint32_t i = tid; i < kTileRows * q_pairs; i += kPrefillThreads) {
+  for (uint32_t i = threadIdx.x; i < kTileRows * q_pairs; i += GROUPS * kPrefillThreads) {
     const uint32_t row = i / q_pairs, d = 2u * (i - row * q_pairs);
     const uint32_t f = f0 + row;
     float a = 0.0f, b = 0.0f;
@@ -605,14 +852,15 @@ __global__ void __launch_bounds__(kPrefillThreads) window_prefill_kernel(WindowA
   const uint32_t q_hi_addr = smem_addr(q_hi) + q_row * L.q_row + q_piece * 16u;
   const uint32_t q_lo_addr = smem_addr(q_lo) + q_row * L.q_row + q_piece * 16u;
 
-  for (uint32_t tile = tile_begin; tile < tile_end; ++tile) {
-    if (tile + 1u < tile_end) {
+  __syncthreads();  // the queries are in place
+  for (uint32_t tile = tile_begin; tile < tile_end; tile += GROUPS) {
+    if (tile + GROUPS < tile_end) {
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
-    __syncthreads();
-    const uint32_t k_base = smem_addr(stages + ((tile - tile_begin) & 1u) * L.stage);
+    group_sync();
+    const uint32_t k_base = smem_addr(stages + ((tile - tile_begin) / GROUPS & 1u) * L.stage);
     const uint32_t v_base = k_base + kKeyTile * L.k_row;
     const uint32_t first = tile * kKeyTile;
     float sc[8][4];
@@ -688,13 +936,54 @@ __global__ void __launch_bounds__(kPrefillThreads) window_prefill_kernel(WindowA
         }
       }
     }
-    __syncthreads();
-    if (tile + 2u < tile_end) issue(tile + 2u);
+    group_sync();
+    if (tile + 2u * GROUPS < tile_end) issue(tile + 2u * GROUPS);
   }
 #pragma unroll
   for (uint32_t i = 0; i < 2u; ++i) {
     l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 1);
     l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 2);
+  }
+  if (GROUPS == 2u) {
+    // the second group's state goes through the stages (idle now): [thread][4 NT + 4], one column per thread
+    float *hand = reinterpret_cast<float *>(smem + 2u * kTileRows * L.q_row) + tid;
+    __syncthreads();
+    if (key_group == 1u) {
+#pragma unroll
+      for (uint32_t n = 0; n < NT; ++n) {
+        if (n * 8u < s.v_pad) {
+#pragma unroll
+          for (uint32_t j = 0; j < 4u; ++j) hand[(4u + n * 4u + j) * kPrefillThreads] = o[n][j];
+        }
+      }
+#pragma unroll
+      for (uint32_t i = 0; i < 2u; ++i) {
+        hand[i * kPrefillThreads] = m_run[i];
+        hand[(2u + i) * kPrefillThreads] = l_run[i];
+      }
+    }
+    __syncthreads();
+    if (key_group == 1u) return;
+    float c0[2], c1[2];
+#pragma unroll
+    for (uint32_t i = 0; i < 2u; ++i) {
+      const float m1 = hand[i * kPrefillThreads], l1 = hand[(2u + i) * kPrefillThreads];
+      const float m = fmaxf(m_run[i], m1);  // one of the groups has seen the row's own key: finite
+      c0[i] = exp2f(m_run[i] - m);
+      c1[i] = exp2f(m1 - m);
+      l_run[i] = l_run[i] * c0[i] + l1 * c1[i];
+    }
+#pragma unroll
+    for (uint32_t n = 0; n < NT; ++n) {
+      if (n * 8u < s.v_pad) {
+#pragma unroll
+        for (uint32_t j = 0; j < 4u; ++j)
+          o[n][j] = o[n][j] * c0[j >> 1] + hand[(4u + n * 4u + j) * kPrefillThreads] * c1[j >> 1];
+      }
+    }
+  }
+#pragma unroll
+  for (uint32_t i = 0; i < 2u; ++i) {
     if (!live[i]) continue;
     const uint32_t f = f0 + warp * 16u + g + 8u * i;
     uint16_t *dst = reinterpret_cast<uint16_t *>(p.out) + static_cast<uint64_t>(f / group) * p.out_stride +
@@ -707,6 +996,13 @@ __global__ void __launch_bounds__(kPrefillThreads) window_prefill_kernel(WindowA
       if (d + 1u < s.v_dim) dst[d + 1u] = f32_to_bf16_bits(o[n][2u * i + 1u] * inv);
     }
   }
+}
+
+// Two key groups where their stages fit and the hand-over fits the stages.
+uint32_t prefill_groups(const WindowAttentionShape &s) {
+  const PrefillLayout L(s, 2);
+  const uint32_t hand = (4u + s.v_pad / 8u * 4u) * kPrefillThreads * 4u;
+  return s.v_pad <= 128u && L.total <= kMaxSmem - 2048u && hand <= 4u * L.stage ? 2u : 1u;
 }
 
 template <class T, bool ROWS>
@@ -728,6 +1024,7 @@ uint32_t decode_smem(const WindowAttentionShape &s, uint32_t tiles) {
 
 template <class T>
 cudaError_t launch_decode(cudaStream_t stream, const WindowAttentionParams &p) {
+  constexpr bool kHasRows = sizeof(T) == 4u;  // bf16 rows run on the tensor pipe
   const uint32_t tiles = chunk_tiles<T>(p.s, p.rows != nullptr);
   const uint32_t bytes = decode_smem<T>(p.s, tiles);
   if (bytes == 0 || bytes > kMaxSmem - 2048u) return cudaErrorNotSupported;
@@ -735,7 +1032,7 @@ cudaError_t launch_decode(cudaStream_t stream, const WindowAttentionParams &p) {
   const uint32_t subs = (group + kHeadsPerBlock - 1u) / kHeadsPerBlock;
   const bool rows = p.rows != nullptr;
   const dim3 grid(p.s.kv_heads * subs * p.splits, rows ? p.row_count : 1u);
-  return launch_with_pdl(rows ? decode_kernel<T, true>(p.s.v_pad) : decode_kernel<T, false>(p.s.v_pad), grid,
+  return launch_with_pdl(rows && kHasRows ? decode_kernel<float, true>(p.s.v_pad) : decode_kernel<T, false>(p.s.v_pad), grid,
                          dim3((rows ? decode_warps<true>() : decode_warps<false>()) * 32u), bytes, stream, p.pdl != 0, p,
                          tiles);
 }
@@ -746,10 +1043,9 @@ bool window_attention_supported(const WindowAttentionShape &s, bool f32) {
   if (s.heads == 0 || s.kv_heads == 0 || s.heads % s.kv_heads != 0 || s.qk_dim == 0 || s.v_dim == 0 || s.qk_pad > 256u ||
       s.v_pad > 256u || s.qk_pad % 16u != 0 || s.v_pad % 16u != 0 || 2u * s.rotary_pairs > s.qk_dim)
     return false;
-  const uint32_t bytes = f32 ? decode_smem<float>(s, chunk_tiles<float>(s, true))
-                             : decode_smem<uint16_t>(s, chunk_tiles<uint16_t>(s, true));
+  const uint32_t bytes = f32 ? decode_smem<float>(s, chunk_tiles<float>(s, true)) : rows_smem(s);
   const uint32_t lone = f32 ? decode_smem<float>(s, 1) : decode_smem<uint16_t>(s, 1);
-  return bytes != 0 && lone != 0 && bytes <= kMaxSmem - 2048u && lone <= kMaxSmem - 2048u && (f32 || PrefillLayout(s).total <= kMaxSmem - 2048u);
+  return bytes != 0 && lone != 0 && bytes <= kMaxSmem - 2048u && lone <= kMaxSmem - 2048u && (f32 || PrefillLayout(s, prefill_groups(s)).total <= kMaxSmem - 2048u);
 }
 
 // Spans for a step whose context is at most target_context: one 32-token tile per block up to
@@ -766,6 +1062,17 @@ uint32_t window_attention_splits(uint32_t target_context, uint32_t window) {
   return s;
 }
 
+// Spans of a block of rows: two blocks per SM are resident, so the count that minimises waves x pages per
+// span, as for the paged kernel of the dense models.
+uint32_t window_rows_splits(const WindowAttentionShape &s, uint32_t rows, uint32_t longest_context, uint32_t sm_count) {
+  const uint32_t group = s.heads / s.kv_heads;
+  uint32_t keys = longest_context;
+  if (s.window != 0 && s.window + kPageTokens < keys) keys = s.window + kPageTokens;
+  const uint32_t splits =
+      attention_default_splits(keys, rows, s.kv_heads * ((group + kHeadsPerBlock - 1u) / kHeadsPerBlock), sm_count);
+  return splits > kWindowMaxSplits ? kWindowMaxSplits : splits;
+}
+
 cudaError_t configure_window_attention() {
   cudaError_t err = cudaSuccess;
   auto set = [&](const void *kernel) {
@@ -774,27 +1081,38 @@ cudaError_t configure_window_attention() {
   };
   for (uint32_t v : {64u, 128u, 256u}) {
     set(reinterpret_cast<const void *>(decode_kernel<uint16_t, false>(v)));
-    set(reinterpret_cast<const void *>(decode_kernel<uint16_t, true>(v)));
     set(reinterpret_cast<const void *>(decode_kernel<float, false>(v)));
     set(reinterpret_cast<const void *>(decode_kernel<float, true>(v)));
   }
-  set(reinterpret_cast<const void *>(window_prefill_kernel<8>));
-  set(reinterpret_cast<const void *>(window_prefill_kernel<16>));
-  set(reinterpret_cast<const void *>(window_prefill_kernel<32>));
+  set(reinterpret_cast<const void *>(window_rows_kernel<1>));
+  set(reinterpret_cast<const void *>(window_rows_kernel<2>));
+  set(reinterpret_cast<const void *>(window_rows_kernel<4>));
+  set(reinterpret_cast<const void *>(window_prefill_kernel<8, 1>));
+  set(reinterpret_cast<const void *>(window_prefill_kernel<16, 1>));
+  set(reinterpret_cast<const void *>(window_prefill_kernel<32, 1>));
+  set(reinterpret_cast<const void *>(window_prefill_kernel<8, 2>));
+  set(reinterpret_cast<const void *>(window_prefill_kernel<16, 2>));
   return err;
 }
 
 cudaError_t launch_window_publish(cudaStream_t stream, const WindowAttentionParams &p) {
   if (p.rows == nullptr || p.row_count == 0 || p.row_count > 65535u) return cudaErrorInvalidValue;
-  const dim3 grid(p.s.heads + p.s.kv_heads, p.row_count);
-  if (p.f32 != 0)
-    return launch_with_pdl(window_publish_kernel<float>, grid, dim3(32), 0, stream, p.pdl != 0, p);
-  return launch_with_pdl(window_publish_kernel<uint16_t>, grid, dim3(32), 0, stream, p.pdl != 0, p);
+  const dim3 grid((p.s.heads + p.s.kv_heads + kPublishWarps - 1u) / kPublishWarps, p.row_count);
+  return launch_with_pdl(p.f32 != 0 ? window_publish_kernel<float> : window_publish_kernel<uint16_t>, grid,
+                         dim3(kPublishWarps * 32), 0, stream, p.pdl != 0, p);
 }
 
 cudaError_t launch_window_attention(cudaStream_t stream, const WindowAttentionParams &p) {
   if (p.splits == 0 || p.splits > kWindowMaxSplits || (p.rows != nullptr && (p.row_count == 0 || p.row_count > 65535u)))
     return cudaErrorInvalidValue;
+  if (p.rows != nullptr && p.f32 == 0) {
+    const uint32_t subs = (p.s.heads / p.s.kv_heads + kHeadsPerBlock - 1u) / kHeadsPerBlock;
+    void (*kernel)(WindowAttentionParams) = p.s.v_pad <= 64u    ? window_rows_kernel<1>
+                                            : p.s.v_pad <= 128u ? window_rows_kernel<2>
+                                                                : window_rows_kernel<4>;
+    return launch_with_pdl(kernel, dim3(p.s.kv_heads * subs * p.splits, p.row_count), dim3(kRowWarps * 32),
+                           rows_smem(p.s), stream, p.pdl != 0, p);
+  }
   return p.f32 != 0 ? launch_decode<float>(stream, p) : launch_decode<uint16_t>(stream, p);
 }
 
@@ -802,11 +1120,14 @@ cudaError_t launch_window_prefill(cudaStream_t stream, const WindowAttentionPara
   if (p.rows == nullptr || p.row_count == 0 || p.f32 != 0) return cudaErrorInvalidValue;
   const uint32_t rows = p.row_count * (p.s.heads / p.s.kv_heads);
   const dim3 grid((rows + kTileRows - 1u) / kTileRows, p.s.kv_heads);
-  const uint32_t bytes = PrefillLayout(p.s).total;
-  void (*kernel)(WindowAttentionParams) = p.s.v_pad <= 64u    ? window_prefill_kernel<8>
-                                          : p.s.v_pad <= 128u ? window_prefill_kernel<16>
-                                                              : window_prefill_kernel<32>;
-  return launch_with_pdl(kernel, grid, dim3(kPrefillThreads), bytes, stream, p.pdl != 0, p);
+  const uint32_t groups = prefill_groups(p.s);
+  const uint32_t bytes = PrefillLayout(p.s, groups).total;
+  void (*kernel)(WindowAttentionParams);
+  if (groups == 2u)
+    kernel = p.s.v_pad <= 64u ? window_prefill_kernel<8, 2> : window_prefill_kernel<16, 2>;
+  else
+    kernel = p.s.v_pad <= 64u ? window_prefill_kernel<8, 1> : (p.s.v_pad <= 128u ? window_prefill_kernel<16, 1> : window_prefill_kernel<32, 1>);
+  return launch_with_pdl(kernel, grid, dim3(groups * kPrefillThreads), bytes, stream, p.pdl != 0, p);
 }
 
 }  // namespace nb
