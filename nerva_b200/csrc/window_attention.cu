@@ -28,6 +28,7 @@ namespace {
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr uint32_t kPageTokens = NERVA_KV_CACHE_BLOCK_TOKENS;
 constexpr uint32_t kTile = 32;             // tokens of one score tile: one per lane
+constexpr uint32_t kWarps = 8;             // of a window_attention_kernel block
 constexpr uint32_t kHeadsPerBlock = 8;
 constexpr uint32_t kMaxSmem = 227u * 1024u;
 
@@ -166,10 +167,9 @@ struct DecodeLayout {
   }
 };
 
-// Score tiles per chunk of the row form: two, or one where two stages of two tiles do not fit shared memory.
+// Score tiles per chunk: two, or one where two stages of two tiles do not fit shared memory.
 template <class T>
-inline uint32_t chunk_tiles(const WindowAttentionShape &s, bool rows) {
-  if (!rows) return 1u;
+uint32_t chunk_tiles(const WindowAttentionShape &s) {
   return DecodeLayout<T>(s, 2u * kTile).total <= kMaxSmem - 2048u ? 2u : 1u;
 }
 
@@ -193,27 +193,43 @@ __device__ __forceinline__ void merge_spans(const WindowAttentionParams &p, uint
   for (uint32_t hw = threadIdx.x >> 5; hw < hb; hw += warps) {
     const uint32_t h = head0 + hw;
     const uint64_t slot0 = (static_cast<uint64_t>(row) * s.heads + h) * S;
+    // every load of a batch of spans is issued before anything is computed from it; the first batch
+    // travels together with the spans' maxima and sums
+    constexpr uint32_t kBatch = PAIRS <= 2u ? 16u : 8u;
+    float2 v[kBatch][PAIRS];
+    auto load = [&](uint32_t first) {
+#pragma unroll
+      for (uint32_t u = 0; u < kBatch; ++u) {
+#pragma unroll
+        for (uint32_t j = 0; j < PAIRS; ++j) {
+          const uint32_t d = 2u * lane + 64u * j;
+          v[u][j] = first + u < S && d < s.v_pad
+                        ? __ldcg(reinterpret_cast<const float2 *>(p.partial_acc + (slot0 + first + u) * s.v_pad + d))
+                        : make_float2(0.0f, 0.0f);
+        }
+      }
+    };
     float ms = -INFINITY, ls = 0.0f;
     if (lane < S) {
       ms = __ldcg(p.partial_m + slot0 + lane);
       ls = __ldcg(p.partial_l + slot0 + lane);
     }
+    load(0);
     const float m = warp_max(ls > 0.0f ? ms : -INFINITY);
     float w = ls > 0.0f ? exp2f(ms - m) : 0.0f;
     w /= warp_sum(ls * w);
     float a[2u * PAIRS];
 #pragma unroll
     for (uint32_t i = 0; i < 2u * PAIRS; ++i) a[i] = 0.0f;
-#pragma unroll 8
-    for (uint32_t i = 0; i < S; ++i) {
-      const float wi = __shfl_sync(0xffffffffu, w, i);
+    for (uint32_t first = 0; first < S; first += kBatch) {
+      if (first != 0) load(first);
 #pragma unroll
-      for (uint32_t j = 0; j < PAIRS; ++j) {
-        const uint32_t d = 2u * lane + 64u * j;
-        if (d < s.v_pad) {
-          const float2 v = __ldcg(reinterpret_cast<const float2 *>(p.partial_acc + (slot0 + i) * s.v_pad + d));
-          a[2u * j] = fmaf(v.x, wi, a[2u * j]);
-          a[2u * j + 1u] = fmaf(v.y, wi, a[2u * j + 1u]);
+      for (uint32_t u = 0; u < kBatch; ++u) {
+        const float wi = __shfl_sync(0xffffffffu, w, (first + u) & 31u);  // zero beyond the last span
+#pragma unroll
+        for (uint32_t j = 0; j < PAIRS; ++j) {
+          a[2u * j] = fmaf(v[u][j].x, wi, a[2u * j]);
+          a[2u * j + 1u] = fmaf(v[u][j].y, wi, a[2u * j + 1u]);
         }
       }
     }
@@ -228,13 +244,10 @@ __device__ __forceinline__ void merge_spans(const WindowAttentionParams &p, uint
 }
 
 // PAIRS: value pairs (2 lane + 64 j, +1) a lane accumulates; v_pad <= 64 PAIRS.
-// A warp has at most two work items: heads x tiles <= 2 warps.  The lone step runs small blocks (4 warps,
-// one tile per chunk) that fit beside a weight-streaming block on the same SM.
-template <bool ROWS>
-constexpr uint32_t decode_warps() { return ROWS ? 8u : 4u; }
+// A warp has at most two work items: heads x tiles <= 2 kWarps.  Two stages of two 128-dim bf16 tiles take
+// 75 KB, which fits beside a weight-streaming block with two ring slots per warp on the same SM.
 template <class T, uint32_t PAIRS, bool ROWS>
-__global__ void __launch_bounds__(decode_warps<ROWS>() * 32) window_attention_kernel(WindowAttentionParams p, uint32_t tiles) {
-  constexpr uint32_t kWarps = decode_warps<ROWS>();
+__global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAttentionParams p, uint32_t tiles) {
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ uint32_t ticket;
   __shared__ float2 turn[ROWS ? 1 : 128];  // sin and cos of the lone step's rotation
@@ -1025,7 +1038,7 @@ uint32_t decode_smem(const WindowAttentionShape &s, uint32_t tiles) {
 template <class T>
 cudaError_t launch_decode(cudaStream_t stream, const WindowAttentionParams &p) {
   constexpr bool kHasRows = sizeof(T) == 4u;  // bf16 rows run on the tensor pipe
-  const uint32_t tiles = chunk_tiles<T>(p.s, p.rows != nullptr);
+  const uint32_t tiles = chunk_tiles<T>(p.s);
   const uint32_t bytes = decode_smem<T>(p.s, tiles);
   if (bytes == 0 || bytes > kMaxSmem - 2048u) return cudaErrorNotSupported;
   const uint32_t group = p.s.heads / p.s.kv_heads;
@@ -1033,7 +1046,7 @@ cudaError_t launch_decode(cudaStream_t stream, const WindowAttentionParams &p) {
   const bool rows = p.rows != nullptr;
   const dim3 grid(p.s.kv_heads * subs * p.splits, rows ? p.row_count : 1u);
   return launch_with_pdl(rows && kHasRows ? decode_kernel<float, true>(p.s.v_pad) : decode_kernel<T, false>(p.s.v_pad), grid,
-                         dim3((rows ? decode_warps<true>() : decode_warps<false>()) * 32u), bytes, stream, p.pdl != 0, p,
+                         dim3(kWarps * 32), bytes, stream, p.pdl != 0, p,
                          tiles);
 }
 
@@ -1043,20 +1056,21 @@ bool window_attention_supported(const WindowAttentionShape &s, bool f32) {
   if (s.heads == 0 || s.kv_heads == 0 || s.heads % s.kv_heads != 0 || s.qk_dim == 0 || s.v_dim == 0 || s.qk_pad > 256u ||
       s.v_pad > 256u || s.qk_pad % 16u != 0 || s.v_pad % 16u != 0 || 2u * s.rotary_pairs > s.qk_dim)
     return false;
-  const uint32_t bytes = f32 ? decode_smem<float>(s, chunk_tiles<float>(s, true)) : rows_smem(s);
-  const uint32_t lone = f32 ? decode_smem<float>(s, 1) : decode_smem<uint16_t>(s, 1);
-  return bytes != 0 && lone != 0 && bytes <= kMaxSmem - 2048u && lone <= kMaxSmem - 2048u && (f32 || PrefillLayout(s, prefill_groups(s)).total <= kMaxSmem - 2048u);
+  const uint32_t lone = f32 ? decode_smem<float>(s, chunk_tiles<float>(s)) : decode_smem<uint16_t>(s, chunk_tiles<uint16_t>(s));
+  auto fits = [](uint32_t bytes) { return bytes != 0 && bytes <= kMaxSmem - 2048u; };
+  return fits(lone) && (f32 || (fits(rows_smem(s)) && fits(PrefillLayout(s, prefill_groups(s)).total)));
 }
 
-// Spans for a step whose context is at most target_context: one 32-token tile per block up to
+// Spans for a step whose context is at most target_context: one 64-token chunk per block up to
 // kWindowMaxSplits, in powers of two so that a growing context re-captures the step rarely, but never
-// more than a full window (which may begin and end inside a tile) needs.
+// more than a full window (which may begin and end inside a chunk) needs.
 uint32_t window_attention_splits(uint32_t target_context, uint32_t window) {
-  const uint32_t tiles = (target_context + kTile - 1u) / kTile;
+  constexpr uint32_t kChunk = 2u * kTile;
+  const uint32_t chunks = target_context / kChunk + (target_context % kChunk != 0 ? 1u : 0u);
   uint32_t s = 1;
-  while (s < tiles && s < kWindowMaxSplits) s <<= 1;
+  while (s < chunks && s < kWindowMaxSplits) s <<= 1;
   if (window != 0) {
-    const uint32_t most = (window + 2u * kTile - 2u) / kTile;
+    const uint32_t most = (window - 1u) / kChunk + 2u;
     if (s > most) s = most;
   }
   return s;
