@@ -889,21 +889,43 @@ int nerva_b200_session_attach_peers(NervaCudaHfDecodeSequenceSession *session,
  * the bounded-wait path on one GPU without faulting or hanging anything. */
 int nerva_b200_session_attach_loopback(NervaCudaHfDecodeSequenceSession *session);
 
-/* ---- parallel-block decoders (no counterpart in the reference) ----
- * A decoder whose layers are described one by one: one norm in front of both sublayers,
- * x += ls1 * attention(norm(x)) + ls2 * mlp(norm(x)), sliding-window grouped-query attention with
- * a rotation of part of each head (optionally YaRN-scaled) and a weightless RMS norm of q and k
- * after it, a range of layers that runs several times with the same weights (each pass with its
- * own cache), a scaled embedding and soft-capped logits.  Every size is per layer.
+/* ---- decoders described layer by layer (no counterpart in the reference) ----
+ * Two kinds of block:
+ *   NERVA_B200_BLOCK_PARALLEL  one norm in front of both sublayers,
+ *       x += ls1 * mixer(norm(x)) + ls2 * mlp(norm(x))
+ *   NERVA_B200_BLOCK_SANDWICH  a norm in front of and a norm behind each sublayer,
+ *       x += norm1b(mixer(norm1(x))), then x += norm2b(mlp(norm2(x)))
+ * and, in sandwich blocks, two kinds of mixer per layer:
+ *   NERVA_B200_MIXER_ATTENTION    sliding-window grouped-query attention; optionally first tokens that
+ *       stay visible, a rotation of part of each head (plain or YaRN-scaled), a weightless RMS norm of
+ *       q and k after it, soft-capped scores, one output gate per head
+ *   NERVA_B200_MIXER_STATE_SPACE  a causal convolution per channel, a selective state-space recurrence
+ *       per head, and a gated RMS norm in groups in front of the output projection
+ * A range of layers may run several times with the same weights (each pass with its own cache and
+ * state), a pass may begin with a projection of the stream joined with the embedding output, the
+ * embedding may be scaled and the logits scaled and soft-capped.  Every size is per layer.
  *
  * The session is an ordinary one: start / advance / run / append / fork / batch_advance_one /
  * read_logits work on it as on any other.  The create request carries the planned weight
  * descriptors (required) and the scalars that are common to the model (hidden, vocab_size,
  * layer_count, max_context_tokens, rms_eps; heads, kv_heads, head_dim and intermediate hold the
- * largest of any layer; every chain layer is FULL / DENSE).  Descriptor order: embeddings,
- * loop vectors (when loop_times != 0), per layer {norm, w_q, w_k, w_v, w_o, w_gate, w_up, w_down
- * (the last three when intermediate != 0), attention scale, mlp scale (when intermediate != 0)},
- * final norm, head. */
+ * largest of any layer; every chain layer is FULL / DENSE).  Descriptor order: embeddings, join
+ * projection (when loop_input), loop vectors (when loop_times != 0), the layers, final norm, head.
+ *   parallel layer: norm, w_q, w_k, w_v, w_g (when head_gate), w_o, w_gate, w_up, w_down (these three when
+ *     intermediate != 0), attention scale, mlp scale (when layer_scale; the second when intermediate != 0)
+ *   sandwich layer: norm in front, the mixer (attention: w_q, w_k, w_v, w_g (when head_gate), w_o; state
+ *     space: w_in, convolution, its bias, step bias, log decay, skip, norm, w_o), norm behind, and, when
+ *     intermediate != 0: norm in front, w_gate, w_up, w_down, norm behind
+ * The rows of a state space's w_in are z [heads * v_dim], x [heads * v_dim], B [groups * state], C [groups
+ * * state], step [heads]; the convolution runs over x, B and C. */
+#define NERVA_B200_BLOCK_PARALLEL 0u
+#define NERVA_B200_BLOCK_SANDWICH 1u
+#define NERVA_B200_MIXER_ATTENTION 0u
+#define NERVA_B200_MIXER_STATE_SPACE 1u
+#define NERVA_B200_NORM_RMS 0u
+#define NERVA_B200_NORM_LAYER 1u
+#define NERVA_B200_ACTIVATION_SILU 0u
+#define NERVA_B200_ACTIVATION_GELU_TANH 1u
 typedef struct NervaB200ParallelLayer {
   uint32_t heads;
   uint32_t kv_heads;
@@ -919,7 +941,15 @@ typedef struct NervaB200ParallelLayer {
   double yarn_fast;
   double yarn_slow;
   float score_scale;
-  uint32_t layer_scale;      /* 1: per-channel scales ls1 / ls2 follow the layer's weights */
+  uint32_t layer_scale;      /* 1: per-channel scales ls1 / ls2 follow the layer's weights (parallel blocks) */
+  uint32_t keep_first;       /* positions below this stay visible behind the window */
+  float score_softcap;       /* 0, or a scaled score s becomes softcap * tanh(s / softcap) */
+  uint32_t head_gate;        /* 1: head i's output is multiplied by sigmoid(w_g row i . mixer input) */
+  uint32_t mixer;            /* NERVA_B200_MIXER_*.  A state space takes heads and v_dim from above and: */
+  uint32_t state_size;       /* at most 256 */
+  uint32_t state_groups;     /* B and C are shared by heads / state_groups heads */
+  uint32_t conv_taps;        /* at most 16, the current token included */
+  uint32_t norm_groups;      /* equal parts of heads * v_dim with a root mean square of their own */
 } NervaB200ParallelLayer;
 typedef struct NervaB200ParallelModel {
   uint32_t layer_count;
@@ -929,6 +959,12 @@ typedef struct NervaB200ParallelModel {
   uint32_t loop_times;
   float embedding_scale;
   float logit_softcap;       /* 0: none */
+  float logit_scale;         /* 0: none; in front of the soft cap */
+  uint32_t block;            /* NERVA_B200_BLOCK_* */
+  uint32_t norm;             /* NERVA_B200_NORM_*: the layers' norms and the final one (parallel blocks: RMS) */
+  uint32_t activation;       /* NERVA_B200_ACTIVATION_* of the gated feed-forward */
+  uint32_t loop_input;       /* 1: every pass begins with x <- W_join [x; embedding output] (sandwich blocks),
+                              * before its loop vector is added */
   uint32_t reserved;
   const NervaB200ParallelLayer *layers;
 } NervaB200ParallelModel;

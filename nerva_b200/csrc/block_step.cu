@@ -34,8 +34,9 @@ __device__ __forceinline__ uint32_t row_token(const BlockTokenRow &r) {
 }
 
 // h[row][:] = embedding row of the row's token, as f32, times scale; rows of `padded` values, zero beyond hidden.
+// copy (optional): receives the same.
 __global__ void block_embed_kernel(const BlockTokenRow *rows, const uint16_t *embeddings, uint32_t hidden, float *h,
-                                   float scale, uint32_t padded) {
+                                   float scale, uint32_t padded, float *copy) {
   pdl_trigger();
   const BlockTokenRow r = rows[blockIdx.x];
   uint32_t token = row_token(r);
@@ -44,8 +45,12 @@ __global__ void block_embed_kernel(const BlockTokenRow *rows, const uint16_t *em
     token = 0;
   }
   const uint16_t *src = embeddings + static_cast<uint64_t>(token) * hidden;
-  float *dst = h + static_cast<uint64_t>(blockIdx.x) * padded;
-  for (uint32_t i = threadIdx.x; i < padded; i += blockDim.x) dst[i] = i < hidden ? bf16_bits_to_f32(src[i]) * scale : 0.0f;
+  const uint64_t row = static_cast<uint64_t>(blockIdx.x) * padded;
+  for (uint32_t i = threadIdx.x; i < padded; i += blockDim.x) {
+    const float v = i < hidden ? bf16_bits_to_f32(src[i]) * scale : 0.0f;
+    h[row + i] = v;
+    if (copy != nullptr) copy[row + i] = v;
+  }
 }
 
 // x[row][:] = bf16(h[row][:] * rsqrt(mean(h^2) + eps) * w): the arithmetic, thread mapping and
@@ -196,17 +201,25 @@ bool plan_workspace(const Session *s, BlockWorkspace *ws, StaticArena &arena, vo
   if (s->parallel) {
     const ParallelPlan &plan = *s->parallel;
     const uint64_t words = plan.element_bytes() / 2u;
-    const uint64_t slots = rows * plan.max_heads * kWindowMaxSplits;
-    bool ok = carve(arena, base, rows * plan.width_pad * words, &ws->x_bf16);
+    const uint64_t slots = std::max<uint64_t>(rows * plan.max_heads * kWindowMaxSplits, 1u);
+    bool ok = carve(arena, base, rows * plan.x_width() * words, &ws->x_bf16);
     ok = ok && carve(arena, base, rows * plan.max_qkv_pad, &ws->qkv);
     ok = ok && carve(arena, base, rows * plan.max_attn_pad * words, &ws->attn);
     ok = ok && carve(arena, base, rows * plan.width_pad, &ws->h_b);
     ok = ok && carve(arena, base, rows * std::max<uint64_t>(plan.max_ff_pad, 8u) * words, &ws->ff);
     ok = ok && carve(arena, base, sample * d.vocab, &ws->logits);
-    ok = ok && carve(arena, base, slots * plan.max_v_pad, &ws->partial_acc);
+    ok = ok && carve(arena, base, slots * std::max(plan.max_v_pad, 1u), &ws->partial_acc);
     ok = ok && carve(arena, base, slots, &ws->partial_m);
     ok = ok && carve(arena, base, slots, &ws->partial_l);
-    ok = ok && carve(arena, base, rows * plan.max_heads, &ws->attn_tickets);
+    ok = ok && carve(arena, base, rows * std::max(plan.max_heads, 1u), &ws->attn_tickets);
+    if (plan.sandwich) ok = ok && carve(arena, base, rows * plan.width_pad, &ws->h_a);
+    if (plan.loop_input) ok = ok && carve(arena, base, rows * plan.width_pad, &ws->first);
+    if (plan.max_space_pad != 0) {
+      uint16_t *convolved = nullptr;
+      ok = ok && carve(arena, base, rows * plan.max_space_pad, &ws->mixed);
+      ok = ok && carve(arena, base, rows * plan.max_conv_width * words, &convolved);
+      ws->convolved = convolved;
+    }
     ok = ok && carve(arena, base, gemm_tc_workspace_bytes(ws->max_rows, s->sm_count) / sizeof(float), &ws->gemm_workspace);
     ok = ok && carve(arena, base, sample * kBlockArgmaxChunks, &ws->best_value);
     ok = ok && carve(arena, base, sample * kBlockArgmaxChunks, &ws->best_index);
@@ -293,7 +306,8 @@ cudaError_t enqueue_block_layers(const BlockPlan &b, uint64_t *launches) {
   cudaError_t err = launch_with_pdl(block_embed_kernel, dim3(b.rows), dim3(256), 0, b.stream, false, ws.token_rows,
                                     arena_at(s, s->layout.embeddings), d.hidden, ws.h_b,
                                     s->parallel ? s->parallel->embedding_scale : 1.0f,
-                                    s->parallel ? s->parallel->width_pad : d.hidden);
+                                    s->parallel ? s->parallel->width_pad : d.hidden,
+                                    s->parallel && s->parallel->loop_input ? ws.first : nullptr);
   n += 1;
   if (s->parallel) {
     if (launches != nullptr) *launches += n;
@@ -424,6 +438,7 @@ FusedAttentionRow attention_row(Session *s, const BlockWorkspace &ws, uint32_t r
   r.value_pages = s->kv_values;
   r.kv_layer_elems = s->kv_layer_elems;
   r.page_table = s->page_table;
+  r.recurrent = s->recurrent;
   r.partial_acc = ws.partial_acc + static_cast<uint64_t>(row) * d.heads * 16u * d.head_dim;
   r.partial_m = ws.partial_m + static_cast<uint64_t>(row) * d.heads * 16u;
   r.partial_l = ws.partial_l + static_cast<uint64_t>(row) * d.heads * 16u;

@@ -21,7 +21,7 @@ __device__ __forceinline__ uint32_t current_token(const StepState &st, uint32_t 
 }
 
 __global__ void embed_kernel(StepState st, const uint16_t *embeddings, uint32_t hidden,
-                             float *input, float scale, uint32_t padded) {
+                             float *input, float scale, uint32_t padded, float *copy) {
   pdl_trigger();  // the first projection may start prefetching its weights now
   const uint32_t position = *st.cursor;
   if (position >= st.max_context) {
@@ -34,8 +34,11 @@ __global__ void embed_kernel(StepState st, const uint16_t *embeddings, uint32_t 
     token = 0;
   }
   const uint16_t *row = embeddings + static_cast<uint64_t>(token) * hidden;
-  for (uint32_t i = threadIdx.x; i < padded; i += blockDim.x)
-    input[i] = i < hidden ? bf16_bits_to_f32(row[i]) * scale : 0.0f;
+  for (uint32_t i = threadIdx.x; i < padded; i += blockDim.x) {
+    const float v = i < hidden ? bf16_bits_to_f32(row[i]) * scale : 0.0f;
+    input[i] = v;
+    if (copy != nullptr) copy[i] = v;
+  }
 }
 
 // One block per head: blocks [0, heads) are query heads, [heads, heads+kv_heads)
@@ -335,8 +338,8 @@ uint32_t grid_for(uint64_t count) {
 }  // namespace
 
 cudaError_t launch_embed(cudaStream_t stream, const StepState &st, const uint16_t *embeddings,
-                         uint32_t hidden, float *input, float scale, uint32_t padded) {
-  embed_kernel<<<1, 256, 0, stream>>>(st, embeddings, hidden, input, scale, padded == 0 ? hidden : padded);
+                         uint32_t hidden, float *input, float scale, uint32_t padded, float *copy) {
+  embed_kernel<<<1, 256, 0, stream>>>(st, embeddings, hidden, input, scale, padded == 0 ? hidden : padded, copy);
   return cudaGetLastError();
 }
 

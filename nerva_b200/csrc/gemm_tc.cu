@@ -72,6 +72,9 @@ struct GemmKernelParams {
   uint32_t split_row;         // kEpilogueStoreSwiglu: first row of the gate/up pairs (a multiple of 32)
   const float *resid_in;
   const uint16_t *row_scale;  // kEpilogueStore, optional: y is multiplied by row_scale[row] before the residual add
+  const uint16_t *row_add;    // kEpilogueStore, optional: added to y
+  uint32_t activation;        // of the gate in gate/up pairs
+  float scale;                // kEpilogueStore: 0, or a factor on y
   float softcap;              // kEpilogueStore: 0, or y becomes softcap * tanh(y / softcap)
   float *out_f32;
   uint16_t *out_bf16;
@@ -235,11 +238,12 @@ __device__ __forceinline__ void row_epilogue(const GemmKernelParams &p, const fl
       const float other = __shfl_xor_sync(0xffffffffu, v[j], 1);
       const uint32_t m = m0 + j;
       if ((lane & 1u) == 0 && row + 1u < p.rows && m < p.tokens)
-        p.out_bf16[static_cast<uint64_t>(m) * width + (row - base) / 2u] = f32_to_bf16_bits(silu(v[j]) * other);
+        p.out_bf16[static_cast<uint64_t>(m) * width + (row - base) / 2u] = f32_to_bf16_bits(activate(p.activation, v[j]) * other);
     }
   } else if (row < p.rows) {
     const uint32_t width = p.epilogue == kEpilogueStoreSwiglu ? p.split_row : p.rows;
     const float scale = p.row_scale != nullptr ? bf16_bits_to_f32(p.row_scale[row]) : 1.0f;
+    const float add = p.row_add != nullptr ? bf16_bits_to_f32(p.row_add[row]) : 0.0f;
 #pragma unroll
     for (uint32_t j = 0; j < N; ++j) {
       const uint32_t m = m0 + j;
@@ -247,6 +251,8 @@ __device__ __forceinline__ void row_epilogue(const GemmKernelParams &p, const fl
         const uint64_t at = static_cast<uint64_t>(m) * width + row;
         float y = v[j];
         if (p.row_scale != nullptr) y *= scale;
+        if (p.row_add != nullptr) y += add;
+        if (p.scale != 0.0f) y *= p.scale;
         if (p.softcap > 0.0f) y = p.softcap * tanhf(y / p.softcap);
         p.out_f32[at] = p.resid_in != nullptr ? y + __ldcg(p.resid_in + at) : y;
       }
@@ -597,6 +603,9 @@ cudaError_t launch_gemm_tc(cudaStream_t stream, const GemmParams &g, uint32_t sm
   p.split_row = g.split_row;
   p.resid_in = g.resid_in;
   p.row_scale = g.row_scale;
+  p.row_add = g.row_add;
+  p.activation = g.activation;
+  p.scale = g.scale;
   p.softcap = g.softcap;
   p.out_f32 = g.out_f32;
   p.out_bf16 = g.out_bf16;

@@ -114,6 +114,9 @@ struct GemmParams {
                            // kEpilogueStoreSwiglu: out_f32[token][split_row], out_bf16[token][(rows - split_row)/2]
   uint32_t split_row;
   const uint16_t *row_scale;  // optional bf16 [rows], kEpilogueStore: y * row_scale[row] is what is stored / added
+  const uint16_t *row_add;    // optional bf16 [rows], kEpilogueStore: added to what is stored
+  uint32_t activation;     // of the gate in gate/up pairs (common.cuh Activation)
+  float scale;             // kEpilogueStore: 0, or a factor on y (in front of the soft cap)
   float softcap;           // kEpilogueStore: 0, or softcap * tanh(y / softcap) is stored
   const float *resid_in;   // optional [tokens][rows]; may be out_f32
   float *out_f32;          // [tokens][rows]
@@ -155,8 +158,9 @@ struct StepState {
 
 // input[h] = embedding[token(cursor)][h] as f32.
 // scale: multiplies every element (1: as stored); padded (0: hidden): elements of `input`, zero beyond hidden.
+// copy (optional): receives the same values.
 cudaError_t launch_embed(cudaStream_t stream, const StepState &st, const uint16_t *embeddings,
-                         uint32_t hidden, float *input, float scale = 1.0f, uint32_t padded = 0);
+                         uint32_t hidden, float *input, float scale = 1.0f, uint32_t padded = 0, float *copy = nullptr);
 
 struct QkvPrepareParams {
   float *qkv;  // [heads*d | kv_heads*d | kv_heads*d] f32, q is normalised/rotated in place
@@ -222,6 +226,7 @@ struct FusedAttentionRow {
   uint16_t *key_pages, *value_pages;  // layer 0 of the row's session; the kernel adds layer * kv_layer_elems
   uint64_t kv_layer_elems;
   const uint32_t *page_table;
+  float *recurrent;        // the row's session's recurrent state (state-space layers)
   float *partial_acc, *partial_m, *partial_l;
   uint32_t *tickets;
   uint16_t *out_bf16;
@@ -325,16 +330,27 @@ cudaError_t configure_moe_kernels();
 // Two launches: routing + gate/up of the chosen experts, then SwiGLU + down and the weighted sum.
 cudaError_t launch_moe_experts(cudaStream_t stream, const MoeExpertParams &p, uint32_t sm_count, bool pdl);
 
-// ---- parallel-block layers (parallel_projection.cu) ----
-// Several weight matrices in one launch for one token: the projections of a layer whose mixer and
-// feed-forward read the same normalised vector, and the two output projections that are summed into
-// the residual stream.  All vectors are padded to multiples of 64 with zeros, matrices have zero
-// columns (and rows) there.
+// ---- projections of decoders described layer by layer (parallel_projection.cu) ----
+// All vectors are padded to multiples of 64 with zeros, matrices have zero columns (and rows) there.
+//
+// Parallel blocks: several weight matrices in one launch for one token, the projections of a layer whose
+// mixer and feed-forward read the same normalised vector, and the two output projections that are summed
+// into the residual stream.
+//
+// Sandwich blocks: a sublayer's output is normalised over the whole vector before it joins the stream, so
+// its projection stores the plain result, and the prologue of the next projection does the rest in every
+// block: h' = h + norm(pending), x = norm(h').  Block 0 stores h'.
 enum ParallelProjectionKind : uint32_t {
   kParallelIn = 0,    // x = norm(h + step); matrix 0 -> out_f32 (fp32); the plain form also does kParallelGate
   kParallelOut = 1,   // h_out = (h + step) + scale0 * (matrix 0 . x0) + scale1 * (matrix 1 . x1)
   kParallelHead = 2,  // x = norm(h); matrix 0 -> soft-capped out_f32 and per-block arg-max partials
   kParallelGate = 3,  // x = norm(h + step); matrix 1 (gate/up rows interleaved, cols0 columns) -> out_act
+  kSandwichIn = 4,    // x = norm(h'); matrix 0 -> out_f32
+  kSandwichGate = 5,  // x = norm(h'); matrix 1 (gate/up rows interleaved, cols0 columns) -> out_act
+  kSandwichHead = 6,  // x = norm(h'); matrix 0 -> scaled, soft-capped out_f32 and per-block arg-max partials
+  kSandwichOut = 7,   // matrix 0 . x0 -> out_f32; x0 is bf16, or (groups != 0) x = grouped RMS norm of x_f32
+  kSandwichJoin = 8,  // x = [h'; first], cols0 = 2 x the padded width; matrix 0 . x + row_add -> out_f32
+  kProjectionKinds = 9,
 };
 struct ParallelProjectionParams {
   const uint16_t *w0, *w1;       // [rows][cols] bf16
@@ -349,6 +365,15 @@ struct ParallelProjectionParams {
   float *h_out;                  // kParallelOut; may be h
   float *out_f32;
   void *out_act;                 // kParallelIn: [rows1 / 2]
+  const float *pending;          // sandwich prologue: optional sublayer output that has not joined the stream yet ...
+  const uint16_t *after;         // ... and its norm's weight; h_out (needed with pending) receives h'
+  uint32_t layer_norm;           // sandwich prologue: 1: both norms take the mean off, 0: RMS norms
+  const float *first;            // kSandwichJoin: [padded width] embedding output
+  const uint16_t *row_add;       // kSandwichJoin (and the plain kParallelIn): optional bf16 [rows0] added to the result
+  const float *x_f32;            // kSandwichOut with groups != 0: [cols0]; its norm's weight is `norm`, `width` its length
+  uint32_t groups;
+  uint32_t activation;           // of gate/up pairs (common.cuh Activation)
+  float scale;                   // heads: 0, or a factor on the logits in front of the soft cap
   float softcap;
   float *best_value;             // kParallelHead [blocks]
   uint32_t *best_index;
@@ -370,13 +395,25 @@ cudaError_t configure_parallel_projection();
 // The plain form: any number of tokens, activations fp32 (f32 = true: true fp32 throughout) or bf16,
 // no norm and no pass vector in front (x0 is the activation block of kParallelIn / kParallelHead).
 // Row strides are cols0 / cols1 for x, rows0 for h, h_out and out_f32, rows1 / 2 for out_act.
+// Sandwich layers run on kParallelIn (either matrix may be absent) and kParallelHead.
 cudaError_t launch_parallel_projection_plain(cudaStream_t stream, uint32_t kind, const ParallelProjectionParams &p,
                                              uint32_t tokens, bool f32);
-// x[row] = norm(h[source] + step) for `rows` rows; source = row_index[row] when given.  step is also added
-// to h itself (then no row_index).  x is fp32 or bf16 [rows][padded].
-cudaError_t launch_stream_norm(cudaStream_t stream, float *h, const uint16_t *step, const uint16_t *norm, float eps,
-                               uint32_t width, uint32_t padded, void *x, bool f32, uint32_t rows,
-                               const uint32_t *row_index, bool pdl);
+// One launch between two projections of a block of rows: h += step, h += norm(pending), both optional, then
+// x = norm(h), or x = [h; first] (no norm), or nothing (x null).
+struct StreamNormParams {
+  float *h;                   // [..][padded]; changed in place by step and pending (then no row_index)
+  const uint16_t *step;       // optional bf16 [padded]
+  const float *pending;       // optional [rows][padded]
+  const uint16_t *after;      // bf16 [padded]: the weight of pending's norm
+  const uint16_t *norm;       // bf16 [padded]: the weight of x's norm, zero beyond width
+  const float *first;         // optional [rows][padded]: x rows are [h; first], 2 padded wide
+  uint32_t layer_norm;        // 1: both norms take the mean off, 0: RMS norms
+  float eps;
+  uint32_t width, padded;
+  void *x;                    // fp32 or bf16, one row per row, or null
+  const uint32_t *row_index;  // optional: x row i comes from h row row_index[i]
+};
+cudaError_t launch_stream_norm(cudaStream_t stream, const StreamNormParams &p, bool f32, uint32_t rows, bool pdl);
 
 // ---- sliding-window grouped-query attention (window_attention.cu) ----
 // Head sizes are arbitrary up to 256; cached rows are [kv_heads][qk_pad] and [kv_heads][v_pad] elements
@@ -384,6 +421,9 @@ cudaError_t launch_stream_norm(cudaStream_t stream, float *h, const uint16_t *st
 struct WindowAttentionShape {
   uint32_t heads, kv_heads, qk_dim, v_dim, qk_pad, v_pad;
   uint32_t window;         // keys a query sees, itself included; 0: all
+  uint32_t keep_first;     // positions below this are seen behind the window too
+  uint32_t head_gate;      // a head's output is multiplied by the sigmoid of its value behind v in the projection's row
+  float softcap;           // 0, or a scaled score s becomes softcap * tanh(s / softcap)
   uint32_t rotary_pairs;   // pairs (i, i + rotary_pairs) of a head that are rotated
   uint32_t qk_norm;        // weightless RMS norm of q and k after the rotation
   float rotary_magnitude;  // factor on cos and sin
@@ -392,7 +432,7 @@ struct WindowAttentionShape {
 };
 struct WindowAttentionParams {
   WindowAttentionShape s;
-  float *qkv;              // [rows][qkv_stride]: q | k | v of the projection; prepared queries are written back
+  float *qkv;              // [rows][qkv_stride]: q | k | v | gate of the projection; prepared queries are written back
   uint32_t qkv_stride;
   void *out;               // [rows][out_stride] bf16 or fp32
   uint32_t out_stride;
@@ -414,7 +454,7 @@ struct WindowAttentionParams {
 };
 constexpr uint32_t kWindowMaxSplits = 16;
 bool window_attention_supported(const WindowAttentionShape &s, bool f32);
-uint32_t window_attention_splits(uint32_t target_context, uint32_t window);  // the lone step
+uint32_t window_attention_splits(uint32_t target_context, uint32_t window, uint32_t keep_first);  // the lone step
 uint32_t window_rows_splits(const WindowAttentionShape &s, uint32_t rows, uint32_t longest_context, uint32_t sm_count);
 cudaError_t configure_window_attention();
 // q/k rotation and norm, K/V rows into the cache, for the rows of a block step.
@@ -423,6 +463,55 @@ cudaError_t launch_window_publish(cudaStream_t stream, const WindowAttentionPara
 cudaError_t launch_window_attention(cudaStream_t stream, const WindowAttentionParams &p);
 // Consecutive positions of one session on the tensor pipe (bf16 cache only).
 cudaError_t launch_window_prefill(cudaStream_t stream, const WindowAttentionParams &p);
+
+// ---- state-space mixer (state_space.cu) ----
+// Per channel of x, B and C a causal convolution and silu, then per head h (group h / (heads / groups)) a state
+// [state][v_dim] in fp32:  S <- exp(-exp(a_log) d) S + d B x^T,  y = S^T C + skip x,  d = softplus(step + bias).
+// What is handed on is y * silu(z); the grouped norm belongs to the output projection.
+//
+// A session's recurrent state of a layer run: the heads' states at state_offset, and at history_offset the last
+// `taps` inputs of the convolution as a ring [position % taps][channels].  A token only reads slots it does not
+// write, so the blocks of a launch need no order.  At position 0 both count as zero whatever they hold.
+struct StateSpaceShape {
+  uint32_t heads, v_dim, state, groups, taps, norm_groups;
+  float eps;               // of the grouped norm
+  __host__ __device__ uint32_t inner() const { return heads * v_dim; }
+  __host__ __device__ uint32_t channels() const { return heads * v_dim + 2u * groups * state; }  // x | B | C
+  __host__ __device__ uint32_t in_rows() const { return inner() + channels() + heads; }          // z | x | B | C | step
+  // convolved block: heads and groups padded to 16 elements
+  __host__ __device__ uint32_t v_pad() const { return (v_dim + 15u) / 16u * 16u; }
+  __host__ __device__ uint32_t state_pad() const { return (state + 15u) / 16u * 16u; }
+  __host__ __device__ uint32_t conv_width() const { return heads * v_pad() + 2u * groups * state_pad(); }
+};
+struct StateSpaceParams {
+  StateSpaceShape s;
+  const float *in;         // [rows][in_stride]: the input projection
+  uint32_t in_stride;
+  const uint16_t *conv, *conv_bias, *step_bias, *a_log, *skip;  // bf16 [channels][taps], [channels], [heads] x 3
+  float *out;              // [rows][out_stride]: y * silu(z)
+  uint32_t out_stride;
+  void *convolved;         // block of one session: scratch [rows][conv_width]
+  uint64_t state_offset, history_offset;  // floats from the start of a session's recurrent state
+  uint32_t f32;            // block of one session: convolved values in fp32
+  uint32_t pdl;
+  // one token of one session
+  const uint32_t *cursor;
+  uint32_t max_context;
+  float *recurrent;
+  // block step: the rows' positions and sessions
+  const struct FusedAttentionRow *rows;
+  uint32_t row_count;
+};
+bool state_space_supported(const StateSpaceShape &s);
+cudaError_t configure_state_space();
+// One token per row: the lone step (rows == nullptr) or rows of different sessions.
+cudaError_t launch_state_space_step(cudaStream_t stream, const StateSpaceParams &p);
+// Consecutive positions of one session: convolution, then the recurrence (two launches).
+cudaError_t launch_state_space_block(cudaStream_t stream, const StateSpaceParams &p);
+// The grouped RMS norm of `rows` rows in front of the output projection; x is fp32 or bf16 [rows][x_stride].
+cudaError_t launch_grouped_norm(cudaStream_t stream, const float *y, uint32_t y_stride, const uint16_t *weight,
+                                uint32_t width, uint32_t groups, float eps, void *x, uint32_t x_stride, bool f32,
+                                uint32_t rows, bool pdl);
 
 // ---- greedy sampling ----
 // Reduces per-block (value, index) partials, writes the token slot at the

@@ -1,9 +1,9 @@
-// Decoders made of parallel blocks: x += ls1 * attention(norm(x)) + ls2 * mlp(norm(x)), every size per
-// layer, a range of layers run several times with the same weights (NervaB200ParallelModel).  This
-// file turns the description into a plan (padded weights, layer runs, cache offsets) and enqueues the
-// layers for the session's two step functions: the decode step (session.cu) and the block step
-// (block_step.cu).  Token fetch, embedding, sampler, token ring, graphs, page table and forks are the
-// session's own.
+// Decoders described layer by layer, every size per layer, a range of layers run several times with the
+// same weights (NervaB200ParallelModel).  This file turns the description into a plan (padded weights,
+// layer runs, cache and state offsets) and enqueues the layers of parallel blocks,
+// x += ls1 * attention(norm(x)) + ls2 * mlp(norm(x)), for the session's two step functions: the decode
+// step (session.cu) and the block step (block_step.cu); sandwich blocks are in sandwich_step.cu.  Token
+// fetch, embedding, sampler, token ring, graphs, page table and forks are the session's own.
 //
 // Decode step, per layer run: norm + [Q; K; V] -> attention, with norm + gate/up streaming beside it ->
 // [O | down] + residual: four launches.  Block step: norm, one projection for all five input matrices, q/k preparation + cache
@@ -13,6 +13,7 @@
 #include <algorithm>
 #include <vector>
 
+#include "common.cuh"
 #include "session.h"
 
 namespace nb {
@@ -112,7 +113,64 @@ WindowAttentionParams layer_attention(const ParallelPlan &plan, const ParallelLa
   return p;
 }
 
-cudaError_t block_gemm(Session *s, cudaStream_t stream, GemmParams g, uint32_t tokens) {
+// Rows below which a block's attention is one query per thread block: a tile of the tensor-pipe kernel
+// would be mostly empty and walk its keys alone.
+constexpr uint32_t kPrefillTileMinRows = 8;
+
+// Checks a layer's attention and fills its part of the plan; why it is refused, or null.
+const char *plan_attention(const NervaB200ParallelLayer &in, bool f32, float eps, ParallelPlan *plan, ParallelLayerPlan *out) {
+  ParallelLayerPlan &l = *out;
+  if (in.heads == 0 || in.kv_heads == 0 || in.heads % in.kv_heads != 0 || in.qk_dim == 0 || in.v_dim == 0 ||
+      in.qk_dim > 256u || in.v_dim > 256u)
+    return "needs heads divisible by kv_heads and head sizes of 1 to 256";
+  if (in.rotary_dims % 2u != 0 || in.rotary_dims > in.qk_dim ||
+      (in.rotary_dims != 0 && !(in.rotary_base > 0.0 && in.rotary_base != 1.0)) ||
+      (in.yarn_factor != 0.0 && !(in.yarn_factor > 0.0 && in.yarn_original > 0.0 && in.yarn_fast > 0.0 && in.yarn_slow > 0.0)))
+    return "rotation";
+  if (!(in.score_softcap >= 0.0f)) return "score soft cap";
+  WindowAttentionShape &a = l.shape;
+  a.heads = in.heads;
+  a.kv_heads = in.kv_heads;
+  a.qk_dim = in.qk_dim;
+  a.v_dim = in.v_dim;
+  a.qk_pad = round_up(in.qk_dim, 16);
+  a.v_pad = round_up(in.v_dim, 16);
+  a.window = in.window;
+  a.keep_first = in.window != 0 ? in.keep_first : 0u;
+  a.head_gate = in.head_gate != 0 ? 1u : 0u;
+  a.softcap = in.score_softcap;
+  a.rotary_pairs = in.rotary_dims / 2u;
+  a.qk_norm = in.qk_norm;
+  a.scale = in.score_scale;
+  a.eps = eps;
+  rotary_table(in, &l.frequencies, &a.rotary_magnitude);
+  if (!window_attention_supported(a, f32)) return "attention shape";
+  l.qkv_rows = in.heads * in.qk_dim + in.kv_heads * (in.qk_dim + in.v_dim) + (a.head_gate != 0 ? in.heads : 0u);
+  plan->max_heads = std::max(plan->max_heads, in.heads);
+  plan->max_v_pad = std::max(plan->max_v_pad, a.v_pad);
+  return nullptr;
+}
+
+const char *plan_state_space(const NervaB200ParallelLayer &in, float eps, ParallelPlan *plan, ParallelLayerPlan *l) {
+  StateSpaceShape &space = l->space;
+  space.heads = in.heads;
+  space.v_dim = in.v_dim;
+  space.state = in.state_size;
+  space.groups = in.state_groups;
+  space.taps = in.conv_taps;
+  space.norm_groups = in.norm_groups;
+  space.eps = eps;
+  if (!state_space_supported(space))
+    return "needs heads divisible by state groups, a state of 1 to 256, 1 to 16 convolution taps and norm groups of equal size";
+  l->state_space = true;
+  l->qkv_rows = space.in_rows();
+  plan->max_conv_width = std::max(plan->max_conv_width, space.conv_width());
+  return nullptr;
+}
+
+}  // namespace
+
+cudaError_t parallel_block_gemm(NervaCudaHfDecodeSequenceSession *s, cudaStream_t stream, GemmParams g, uint32_t tokens) {
   const BlockWorkspace &ws = s->weights->block_ws;
   g.tokens = tokens;
   g.workspace = ws.gemm_workspace;
@@ -121,15 +179,31 @@ cudaError_t block_gemm(Session *s, cudaStream_t stream, GemmParams g, uint32_t t
   return launch_gemm_tc(stream, g, s->sm_count);
 }
 
-// Rows below which a block's attention is one query per thread block: a tile of the tensor-pipe kernel
-// would be mostly empty and walk its keys alone.
-constexpr uint32_t kPrefillTileMinRows = 8;
+StreamNormParams layer_stream_norm(const NervaCudaHfDecodeSequenceSession *s, float *h, const uint16_t *weight, void *x) {
+  const ParallelPlan &plan = *s->parallel;
+  StreamNormParams p{};
+  p.h = h;
+  p.norm = weight;
+  p.layer_norm = plan.layer_norm;
+  p.eps = s->rms_eps;
+  p.width = plan.width;
+  p.padded = plan.width_pad;
+  p.x = x;
+  return p;
+}
 
-}  // namespace
+cudaError_t capture_block_stream(NervaCudaHfDecodeSequenceSession *s, const ParallelBlock &b, size_t run) {
+  if (s->capture_stream == nullptr || !b.one_session || b.capture_row >= s->capture_rows) return cudaSuccess;
+  const ParallelPlan &plan = *s->parallel;
+  const uint32_t rows = std::min(b.rows, s->capture_rows - b.capture_row);
+  return cudaMemcpy2DAsync(s->capture_stream + (run * s->capture_rows + b.capture_row) * plan.width, plan.width * sizeof(float),
+                           s->weights->block_ws.h_b, plan.width_pad * sizeof(float), plan.width * sizeof(float), rows,
+                           cudaMemcpyDeviceToHost, b.stream);
+}
 
 std::shared_ptr<ParallelPlan> make_parallel_plan(const NervaB200ParallelModel &m, uint32_t width, uint32_t vocab, float eps) {
   auto refuse = [](const char *why) {
-    set_last_error(std::string("parallel-block model not supported: ") + why);
+    set_last_error(std::string("model not supported: ") + why);
     return std::shared_ptr<ParallelPlan>();
   };
   auto plan = std::make_shared<ParallelPlan>();
@@ -139,45 +213,36 @@ std::shared_ptr<ParallelPlan> make_parallel_plan(const NervaB200ParallelModel &m
   plan->width_pad = round_up(width, 64);
   plan->vocab = vocab;
   plan->embedding_scale = m.embedding_scale;
+  plan->logit_scale = m.logit_scale;
   plan->softcap = m.logit_softcap;
   plan->loop_times = m.loop_times;
+  if (m.block > NERVA_B200_BLOCK_SANDWICH || m.norm > NERVA_B200_NORM_LAYER || m.activation > NERVA_B200_ACTIVATION_GELU_TANH)
+    return refuse("block, norm or activation");
+  plan->sandwich = m.block == NERVA_B200_BLOCK_SANDWICH;
+  plan->layer_norm = m.norm == NERVA_B200_NORM_LAYER ? 1u : 0u;
+  plan->activation = m.activation == NERVA_B200_ACTIVATION_GELU_TANH ? kActivationGeluTanh : kActivationSilu;
+  plan->loop_input = m.loop_input != 0 && m.loop_times != 0;
+  if (!plan->sandwich && (plan->layer_norm != 0 || plan->loop_input))
+    return refuse("layer norms and a loop's input projection come with sandwich blocks");
   if (m.loop_times != 0 && (m.loop_start >= m.loop_stop || m.loop_stop > m.layer_count)) return refuse("loop range");
   for (uint32_t i = 0; i < m.layer_count; ++i) {
     const NervaB200ParallelLayer &in = m.layers[i];
-    if (in.heads == 0 || in.kv_heads == 0 || in.heads % in.kv_heads != 0 || in.qk_dim == 0 || in.v_dim == 0 ||
-        in.qk_dim > 256u || in.v_dim > 256u)
-      return refuse("needs heads divisible by kv_heads and head sizes of 1 to 256");
-    if (in.rotary_dims % 2u != 0 || in.rotary_dims > in.qk_dim ||
-        (in.rotary_dims != 0 && !(in.rotary_base > 0.0 && in.rotary_base != 1.0)) ||
-        (in.yarn_factor != 0.0 && !(in.yarn_factor > 0.0 && in.yarn_original > 0.0 && in.yarn_fast > 0.0 && in.yarn_slow > 0.0)))
-      return refuse("rotation");
     ParallelLayerPlan l;
-    WindowAttentionShape &a = l.shape;
-    a.heads = in.heads;
-    a.kv_heads = in.kv_heads;
-    a.qk_dim = in.qk_dim;
-    a.v_dim = in.v_dim;
-    a.qk_pad = round_up(in.qk_dim, 16);
-    a.v_pad = round_up(in.v_dim, 16);
-    a.window = in.window;
-    a.rotary_pairs = in.rotary_dims / 2u;
-    a.qk_norm = in.qk_norm;
-    a.scale = in.score_scale;
-    a.eps = eps;
-    rotary_table(in, &l.frequencies, &a.rotary_magnitude);
-    if (!window_attention_supported(a, plan->f32)) return refuse("attention shape");
+    const bool space = in.mixer == NERVA_B200_MIXER_STATE_SPACE;
+    if (in.mixer > NERVA_B200_MIXER_STATE_SPACE || (space && !plan->sandwich)) return refuse("mixer");
+    if (plan->sandwich && in.layer_scale != 0) return refuse("layer scales come with parallel blocks");
+    const char *why = space ? plan_state_space(in, eps, plan.get(), &l) : plan_attention(in, plan->f32, eps, plan.get(), &l);
+    if (why != nullptr) return refuse(why);
     l.intermediate = in.intermediate;
     l.ff_pad = round_up(in.intermediate, 64);
-    l.qkv_rows = in.heads * in.qk_dim + in.kv_heads * (in.qk_dim + in.v_dim);
     l.qkv_pad = round_up(l.qkv_rows, 64);
     l.attn_width = in.heads * in.v_dim;
     l.attn_pad = round_up(l.attn_width, 64);
     l.layer_scale = in.layer_scale != 0;
-    plan->max_heads = std::max(plan->max_heads, in.heads);
     plan->max_qkv_pad = std::max(plan->max_qkv_pad, l.qkv_pad);
     plan->max_attn_pad = std::max(plan->max_attn_pad, l.attn_pad);
     plan->max_ff_pad = std::max(plan->max_ff_pad, l.ff_pad);
-    plan->max_v_pad = std::max(plan->max_v_pad, a.v_pad);
+    if (space) plan->max_space_pad = std::max(plan->max_space_pad, l.attn_pad);
     plan->layers.push_back(l);
   }
   auto run = [&](uint32_t layer, int32_t step) {
@@ -196,8 +261,19 @@ std::shared_ptr<ParallelPlan> make_parallel_plan(const NervaB200ParallelModel &m
 
 void place_parallel_cache(ParallelPlan *plan, uint32_t pages) {
   const uint64_t tokens = static_cast<uint64_t>(pages) * NERVA_KV_CACHE_BLOCK_TOKENS;
-  plan->key_elems = plan->value_elems = 0;
+  plan->key_elems = plan->value_elems = plan->recurrent_floats = 0;
   for (ParallelRun &r : plan->runs) {
+    if (plan->layers[r.layer].state_space) {
+      const StateSpaceShape &space = plan->layers[r.layer].space;
+      auto place = [&](uint64_t floats) {  // 16-byte pieces
+        const uint64_t at = plan->recurrent_floats;
+        plan->recurrent_floats += (floats + 3u) / 4u * 4u;
+        return at;
+      };
+      r.state_offset = place(static_cast<uint64_t>(space.heads) * space.state * space.v_dim);
+      r.history_offset = place(static_cast<uint64_t>(space.taps) * space.channels());
+      continue;
+    }
     const WindowAttentionShape &a = plan->layers[r.layer].shape;
     r.key_offset = plan->key_elems;
     r.value_offset = plan->value_elems;
@@ -220,6 +296,11 @@ cudaError_t pack_parallel_weights(Session *s) {
   };
   clear(plan.loop_vectors, static_cast<uint64_t>(std::max(plan.loop_times, 1u)) * pad * 2u);
   pack(s->layout.loop_vectors, plan.loop_times, width, plan.loop_vectors, pad, 1, 0);
+  if (plan.loop_input) {
+    // [out][stream | embedding], each half padded: as rows of one half, the halves of a matrix row follow each other
+    clear(plan.w_join, 2ull * pad * pad * 2u);
+    pack(s->layout.loop_input, 2u * width, width, plan.w_join, pad, 1, 0);
+  }
   for (size_t i = 0; i < plan.layers.size(); ++i) {
     const ParallelLayerPlan &l = plan.layers[i];
     const LayerLayout &L = s->layout.layers[i];
@@ -230,10 +311,27 @@ cudaError_t pack_parallel_weights(Session *s) {
     clear(l.norm, pad * 2u);
     clear(l.ls_attn, pad * 2u);
     clear(l.ls_mlp, pad * 2u);
-    const uint32_t q_rows = a.heads * a.qk_dim, k_rows = a.kv_heads * a.qk_dim, v_rows = a.kv_heads * a.v_dim;
-    pack(L.w_q, q_rows, width, l.w_in, pad, 1, 0);
-    pack(L.w_k, k_rows, width, l.w_in, pad, 1, q_rows);
-    pack(L.w_v, v_rows, width, l.w_in, pad, 1, q_rows + k_rows);
+    if (l.state_space) {
+      pack(L.w_space, l.qkv_rows, width, l.w_in, pad, 1, 0);
+      clear(l.group_norm, l.attn_pad * 2u);
+      pack(L.group_norm, 1, l.attn_width, l.group_norm, l.attn_pad, 1, 0);
+    } else {
+      const uint32_t q_rows = a.heads * a.qk_dim, k_rows = a.kv_heads * a.qk_dim, v_rows = a.kv_heads * a.v_dim;
+      pack(L.w_q, q_rows, width, l.w_in, pad, 1, 0);
+      pack(L.w_k, k_rows, width, l.w_in, pad, 1, q_rows);
+      pack(L.w_v, v_rows, width, l.w_in, pad, 1, q_rows + k_rows);
+      if (a.head_gate != 0) pack(L.w_head_gate, a.heads, width, l.w_in, pad, 1, q_rows + k_rows + v_rows);
+    }
+    if (plan.sandwich) {
+      clear(l.norm_after, pad * 2u);
+      clear(l.norm_mlp, pad * 2u);
+      clear(l.norm_mlp_after, pad * 2u);
+      pack(L.norm_after, 1, width, l.norm_after, pad, 1, 0);
+      if (l.intermediate != 0) {
+        pack(L.rms_mlp, 1, width, l.norm_mlp, pad, 1, 0);
+        pack(L.norm_mlp_after, 1, width, l.norm_mlp_after, pad, 1, 0);
+      }
+    }
     pack(L.w_o, width, l.attn_width, l.w_o, l.attn_pad, 1, 0);
     pack(L.rms_attn, 1, width, l.norm, pad, 1, 0);
     if (l.intermediate != 0) {
@@ -259,13 +357,60 @@ cudaError_t pack_parallel_weights(Session *s) {
 
 uint32_t parallel_attention_splits(const ParallelPlan &plan, uint32_t target_context) {
   uint32_t most = 1;
-  for (const ParallelLayerPlan &l : plan.layers)
-    most = std::max(most, window_attention_splits(target_context, l.shape.window));
+  for (const ParallelLayerPlan &l : plan.layers) {
+    if (!l.state_space) most = std::max(most, window_attention_splits(target_context, l.shape.window, l.shape.keep_first));
+  }
   return most;
 }
 
-cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launches, StepProfile *prof, ProfileMark mark) {
+cudaError_t enqueue_step_attention(Session *s, const ParallelLayerPlan &l, const ParallelRun &run, uint32_t splits,
+                                   uint64_t *launches) {
+  WindowAttentionParams a = layer_attention(*s->parallel, l, run);
+  a.pdl = s->use_pdl ? 1u : 0u;
+  a.qkv = s->qkv;
+  a.out = s->attn_bf16;
+  a.splits = std::min(splits, window_attention_splits(UINT32_MAX / 2u, l.shape.window, l.shape.keep_first));
+  a.partial_acc = s->partial_acc;
+  a.partial_m = s->partial_m;
+  a.partial_l = s->partial_l;
+  a.tickets = s->attn_tickets;
+  a.cursor = s->device_cursor;
+  a.max_context = s->max_context;
+  a.page_count = s->kv_pages;
+  a.keys = s->kv_keys;
+  a.values = s->kv_values;
+  a.page_table = s->page_table;
+  a.error_word = s->device_error;
+  *launches += 1;
+  return launch_window_attention(s->stream, a);
+}
+
+cudaError_t enqueue_block_attention(Session *s, const ParallelBlock &b, const ParallelLayerPlan &l, const ParallelRun &run,
+                                    uint64_t *launches) {
   const ParallelPlan &plan = *s->parallel;
+  const BlockWorkspace &ws = s->weights->block_ws;
+  WindowAttentionParams a = layer_attention(plan, l, run);
+  a.pdl = s->use_pdl ? 1u : 0u;
+  a.qkv = ws.qkv;
+  a.out = ws.attn;
+  a.partial_acc = ws.partial_acc;
+  a.partial_m = ws.partial_m;
+  a.partial_l = ws.partial_l;
+  a.tickets = ws.attn_tickets;
+  a.rows = ws.attn_rows;
+  a.row_count = b.rows;
+  *launches += 2;
+  const cudaError_t err = launch_window_publish(b.stream, a);
+  if (err != cudaSuccess) return err;
+  if (b.one_session && b.rows >= kPrefillTileMinRows && !plan.f32) return launch_window_prefill(b.stream, a);
+  a.splits = window_rows_splits(l.shape, b.rows, b.longest, s->sm_count);
+  return launch_window_attention(b.stream, a);
+}
+
+cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, ResidualStream *stream, uint64_t *launches, StepProfile *prof,
+                                    ProfileMark mark) {
+  const ParallelPlan &plan = *s->parallel;
+  if (plan.sandwich) return enqueue_sandwich_layers(s, splits, stream, launches, prof, mark);
   const uint32_t pdl = s->use_pdl ? 1u : 0u;
   uint64_t n = 0;
   cudaError_t err = cudaSuccess;
@@ -279,6 +424,7 @@ cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launc
     in.step = step;
     in.out_f32 = s->qkv;
     in.out_act = s->ff_bf16;
+    in.activation = plan.activation;
     ParallelProjectionParams out = layer_out(plan, l);
     out.pdl = pdl;
     out.error_word = s->device_error;
@@ -295,8 +441,9 @@ cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launc
       err = launch_parallel_projection(s->stream, kParallelIn, in, s->sm_count);
       n += 1;
     } else {
-      err = launch_stream_norm(s->stream, s->h_b, step, l.norm, s->rms_eps, plan.width, plan.width_pad, s->x_scratch,
-                               plan.f32, 1, nullptr, pdl != 0);
+      StreamNormParams norm = layer_stream_norm(s, s->h_b, l.norm, s->x_scratch);
+      norm.step = step;
+      err = launch_stream_norm(s->stream, norm, plan.f32, 1, pdl != 0);
       out.step = nullptr;  // it is part of the stream now
       in.x0 = s->x_scratch;
       if (err == cudaSuccess) err = launch_parallel_projection_plain(s->stream, kParallelIn, in, 1, plan.f32);
@@ -305,24 +452,7 @@ cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launc
     mark(s, prof, kBucketQkv);
     if (err != cudaSuccess) break;
 
-    WindowAttentionParams a = layer_attention(plan, l, run);
-    a.pdl = pdl;
-    a.qkv = s->qkv;
-    a.out = s->attn_bf16;
-    a.splits = std::min(splits, window_attention_splits(UINT32_MAX / 2u, l.shape.window));
-    a.partial_acc = s->partial_acc;
-    a.partial_m = s->partial_m;
-    a.partial_l = s->partial_l;
-    a.tickets = s->attn_tickets;
-    a.cursor = s->device_cursor;
-    a.max_context = s->max_context;
-    a.page_count = s->kv_pages;
-    a.keys = s->kv_keys;
-    a.values = s->kv_values;
-    a.page_table = s->page_table;
-    a.error_word = s->device_error;
-    err = launch_window_attention(s->stream, a);
-    n += 1;
+    err = enqueue_step_attention(s, l, run, splits, &n);
     mark(s, prof, kBucketAttention);
     if (err != cudaSuccess) break;
     if (streamed && gate) {
@@ -351,29 +481,37 @@ cudaError_t enqueue_parallel_layers(Session *s, uint32_t splits, uint64_t *launc
   return err;
 }
 
-cudaError_t enqueue_parallel_head(Session *s, uint32_t *partials, uint64_t *launches) {
+cudaError_t enqueue_parallel_head(Session *s, const ResidualStream &stream, uint32_t *partials, uint64_t *launches) {
   const ParallelPlan &plan = *s->parallel;
+  const uint32_t kind = plan.sandwich ? kSandwichHead : kParallelHead;
   ParallelProjectionParams p{};
   p.w0 = plan.head;
   p.rows0 = plan.vocab;
   p.cols0 = plan.width_pad;
-  p.h = s->h_b;
+  p.h = stream.h;
+  p.pending = stream.pending;
+  p.after = stream.after;
+  p.h_out = stream.h == s->h_a ? s->h_b : s->h_a;
+  p.layer_norm = plan.layer_norm;
   p.norm = plan.final_norm;
   p.width = plan.width;
   p.eps = s->rms_eps;
   p.out_f32 = s->logits;
+  p.scale = plan.logit_scale;
   p.softcap = plan.softcap;
   p.best_value = s->best_value;
   p.best_index = s->best_index;
   p.error_word = s->device_error;
   p.pdl = s->use_pdl ? 1u : 0u;
-  if (!plan.f32 && parallel_stream_eligible(kParallelHead, p, s->sm_count)) {
-    *partials = parallel_stream_blocks(kParallelHead, p, s->sm_count);
+  if (!plan.f32 && parallel_stream_eligible(kind, p, s->sm_count)) {
+    *partials = parallel_stream_blocks(kind, p, s->sm_count);
     if (launches != nullptr) *launches += 1;
-    return launch_parallel_projection(s->stream, kParallelHead, p, s->sm_count);
+    return launch_parallel_projection(s->stream, kind, p, s->sm_count);
   }
-  cudaError_t err = launch_stream_norm(s->stream, s->h_b, nullptr, plan.final_norm, s->rms_eps, plan.width,
-                                       plan.width_pad, s->x_scratch, plan.f32, 1, nullptr, p.pdl != 0);
+  StreamNormParams norm = layer_stream_norm(s, stream.h, plan.final_norm, s->x_scratch);
+  norm.pending = stream.pending;
+  norm.after = stream.after;
+  cudaError_t err = launch_stream_norm(s->stream, norm, plan.f32, 1, p.pdl != 0);
   p.x0 = s->x_scratch;
   if (err == cudaSuccess) err = launch_parallel_projection_plain(s->stream, kParallelHead, p, 1, plan.f32);
   *partials = std::min(kBlockArgmaxChunks, s->sm_count);
@@ -385,6 +523,7 @@ cudaError_t enqueue_parallel_head(Session *s, uint32_t *partials, uint64_t *laun
 
 cudaError_t enqueue_parallel_block_layers(Session *s, const ParallelBlock &b, uint64_t *launches) {
   const ParallelPlan &plan = *s->parallel;
+  if (plan.sandwich) return enqueue_sandwich_block_layers(s, b, launches);
   const BlockWorkspace &ws = s->weights->block_ws;
   const uint32_t pdl = s->use_pdl ? 1u : 0u;
   uint64_t n = 0;
@@ -392,13 +531,15 @@ cudaError_t enqueue_parallel_block_layers(Session *s, const ParallelBlock &b, ui
   for (size_t index = 0; err == cudaSuccess && index < plan.runs.size(); ++index) {
     const ParallelRun &run = plan.runs[index];
     const ParallelLayerPlan &l = plan.layers[run.layer];
-    err = launch_stream_norm(b.stream, ws.h_b, step_vector(plan, run), l.norm, s->rms_eps, plan.width, plan.width_pad,
-                             ws.x_bf16, plan.f32, b.rows, nullptr, pdl != 0);
+    StreamNormParams norm = layer_stream_norm(s, ws.h_b, l.norm, ws.x_bf16);
+    norm.step = step_vector(plan, run);
+    err = launch_stream_norm(b.stream, norm, plan.f32, b.rows, pdl != 0);
     ParallelProjectionParams in = layer_in(plan, l, s->rms_eps);
     if (err == cudaSuccess && plan.f32) {
       in.x0 = ws.x_bf16;
       in.out_f32 = ws.qkv;
       in.out_act = ws.ff;
+      in.activation = plan.activation;
       in.pdl = pdl;
       err = launch_parallel_projection_plain(b.stream, kParallelIn, in, b.rows, true);
     } else if (err == cudaSuccess) {
@@ -409,30 +550,12 @@ cudaError_t enqueue_parallel_block_layers(Session *s, const ParallelBlock &b, ui
       g.x = ws.x_bf16;
       g.epilogue = l.ff_pad != 0 ? kEpilogueStoreSwiglu : kEpilogueStore;
       g.split_row = l.qkv_pad;
+      g.activation = plan.activation;
       g.out_f32 = ws.qkv;
       g.out_bf16 = ws.ff;
-      err = block_gemm(s, b.stream, g, b.rows);
+      err = parallel_block_gemm(s, b.stream, g, b.rows);
     }
-
-    WindowAttentionParams a = layer_attention(plan, l, run);
-    a.pdl = pdl;
-    a.qkv = ws.qkv;
-    a.out = ws.attn;
-    a.partial_acc = ws.partial_acc;
-    a.partial_m = ws.partial_m;
-    a.partial_l = ws.partial_l;
-    a.tickets = ws.attn_tickets;
-    a.rows = ws.attn_rows;
-    a.row_count = b.rows;
-    if (err == cudaSuccess) err = launch_window_publish(b.stream, a);
-    if (err == cudaSuccess) {
-      if (b.one_session && b.rows >= kPrefillTileMinRows && !plan.f32) {
-        err = launch_window_prefill(b.stream, a);
-      } else {
-        a.splits = window_rows_splits(l.shape, b.rows, b.longest, s->sm_count);
-        err = launch_window_attention(b.stream, a);
-      }
-    }
+    if (err == cudaSuccess) err = enqueue_block_attention(s, b, l, run, &n);
 
     ParallelProjectionParams out = layer_out(plan, l);
     if (err == cudaSuccess && plan.f32) {
@@ -441,7 +564,7 @@ cudaError_t enqueue_parallel_block_layers(Session *s, const ParallelBlock &b, ui
       out.x1 = ws.ff;
       out.pdl = pdl;
       err = launch_parallel_projection_plain(b.stream, kParallelOut, out, b.rows, true);
-      n += 5;
+      n += 3;
     } else if (err == cudaSuccess) {
       GemmParams g{};
       g.rows = plan.width_pad;
@@ -451,22 +574,17 @@ cudaError_t enqueue_parallel_block_layers(Session *s, const ParallelBlock &b, ui
       g.cols = out.cols0;
       g.x = ws.attn;
       g.row_scale = out.scale0;
-      err = block_gemm(s, b.stream, g, b.rows);
+      err = parallel_block_gemm(s, b.stream, g, b.rows);
       if (err == cudaSuccess && l.ff_pad != 0) {
         g.weight = out.w1;
         g.cols = out.cols1;
         g.x = ws.ff;
         g.row_scale = out.scale1;
-        err = block_gemm(s, b.stream, g, b.rows);
+        err = parallel_block_gemm(s, b.stream, g, b.rows);
       }
-      n += l.ff_pad != 0 ? 6 : 5;
+      n += l.ff_pad != 0 ? 4 : 3;
     }
-    if (err == cudaSuccess && s->capture_stream != nullptr && b.one_session && b.capture_row < s->capture_rows) {
-      const uint32_t rows = std::min(b.rows, s->capture_rows - b.capture_row);
-      err = cudaMemcpy2DAsync(s->capture_stream + (index * s->capture_rows + b.capture_row) * plan.width,
-                              plan.width * sizeof(float), ws.h_b, plan.width_pad * sizeof(float),
-                              plan.width * sizeof(float), rows, cudaMemcpyDeviceToHost, b.stream);
-    }
+    if (err == cudaSuccess) err = capture_block_stream(s, b, index);
   }
   if (launches != nullptr) *launches += n;
   return err;
@@ -476,8 +594,9 @@ cudaError_t enqueue_parallel_block_head(Session *s, cudaStream_t stream, uint32_
                                         uint64_t *launches) {
   const ParallelPlan &plan = *s->parallel;
   const BlockWorkspace &ws = s->weights->block_ws;
-  cudaError_t err = launch_stream_norm(stream, ws.h_b, nullptr, plan.final_norm, s->rms_eps, plan.width, plan.width_pad,
-                                       ws.x_bf16, plan.f32, count, row_index, s->use_pdl);
+  StreamNormParams norm = layer_stream_norm(s, ws.h_b, plan.final_norm, ws.x_bf16);
+  norm.row_index = row_index;
+  cudaError_t err = launch_stream_norm(stream, norm, plan.f32, count, s->use_pdl);
   if (err == cudaSuccess && plan.f32) {
     ParallelProjectionParams p{};
     p.w0 = plan.head;
@@ -485,6 +604,7 @@ cudaError_t enqueue_parallel_block_head(Session *s, cudaStream_t stream, uint32_
     p.cols0 = plan.width_pad;
     p.x0 = ws.x_bf16;
     p.out_f32 = ws.logits;
+    p.scale = plan.logit_scale;
     p.softcap = plan.softcap;
     p.pdl = s->use_pdl ? 1u : 0u;
     err = launch_parallel_projection_plain(stream, kParallelHead, p, count, true);
@@ -495,9 +615,10 @@ cudaError_t enqueue_parallel_block_head(Session *s, cudaStream_t stream, uint32_
     g.cols = plan.width_pad;
     g.x = ws.x_bf16;
     g.epilogue = kEpilogueStore;
+    g.scale = plan.logit_scale;
     g.softcap = plan.softcap;
     g.out_f32 = ws.logits;
-    err = block_gemm(s, stream, g, count);
+    err = parallel_block_gemm(s, stream, g, count);
   }
   if (launches != nullptr) *launches += 2;
   return err;

@@ -123,21 +123,38 @@ ArenaLayout compute_arena_layout(const ModelDims &d, const NervaCudaHfDecodeChai
   out.scratch = push(c, hidden);
   out.layers.resize(d.layers);
   if (parallel != nullptr) {
+    if (parallel->loop_times != 0 && parallel->loop_input != 0) out.loop_input = push(c, 2u * hidden * hidden);
     if (parallel->loop_times != 0) out.loop_vectors = push(c, static_cast<uint64_t>(parallel->loop_times) * hidden);
     for (uint32_t i = 0; i < d.layers; ++i) {
       const NervaB200ParallelLayer &layer = parallel->layers[i];
       LayerLayout &l = out.layers[i];
       const uint64_t q = static_cast<uint64_t>(layer.heads) * layer.qk_dim, k = static_cast<uint64_t>(layer.kv_heads) * layer.qk_dim;
       const uint64_t v = static_cast<uint64_t>(layer.kv_heads) * layer.v_dim, a = static_cast<uint64_t>(layer.heads) * layer.v_dim;
+      const bool sandwich = parallel->block == NERVA_B200_BLOCK_SANDWICH;
       l.rms_attn = push(c, hidden);
-      l.w_q = push(c, q * hidden);
-      l.w_k = push(c, k * hidden);
-      l.w_v = push(c, v * hidden);
+      if (layer.mixer == NERVA_B200_MIXER_STATE_SPACE) {
+        const uint64_t channels = a + 2ull * layer.state_groups * layer.state_size;
+        l.w_space = push(c, (a + channels + layer.heads) * hidden);
+        l.conv = push(c, channels * layer.conv_taps);
+        l.conv_bias = push(c, channels);
+        l.step_bias = push(c, layer.heads);
+        l.a_log = push(c, layer.heads);
+        l.skip = push(c, layer.heads);
+        l.group_norm = push(c, a);
+      } else {
+        l.w_q = push(c, q * hidden);
+        l.w_k = push(c, k * hidden);
+        l.w_v = push(c, v * hidden);
+        if (layer.head_gate != 0) l.w_head_gate = push(c, layer.heads * hidden);
+      }
       l.w_o = push(c, hidden * a);
+      if (sandwich) l.norm_after = push(c, hidden);
       if (layer.intermediate != 0) {
+        if (sandwich) l.rms_mlp = push(c, hidden);
         l.w_gate = push(c, layer.intermediate * hidden);
         l.w_up = push(c, layer.intermediate * hidden);
         l.w_down = push(c, hidden * layer.intermediate);
+        if (sandwich) l.norm_mlp_after = push(c, hidden);
       }
       if (layer.layer_scale != 0) {
         l.ls_attn = push(c, hidden);
@@ -295,6 +312,7 @@ bool plan_weights(Session *s, StaticArena &arena, void *base, SharedWeights *w) 
     ParallelPlan &plan = *s->parallel;
     const uint64_t width = plan.width_pad;
     ok = ok && carve(arena, base, std::max<uint64_t>(plan.loop_times, 1u) * width, &plan.loop_vectors);
+    if (plan.loop_input) ok = ok && carve(arena, base, 2u * width * width, &plan.w_join);
     for (ParallelLayerPlan &l : plan.layers) {
       ok = ok && carve(arena, base, (l.qkv_pad + 2ull * l.ff_pad) * width, &l.w_in);
       ok = ok && carve(arena, base, width * l.attn_pad, &l.w_o);
@@ -302,6 +320,12 @@ bool plan_weights(Session *s, StaticArena &arena, void *base, SharedWeights *w) 
       ok = ok && carve(arena, base, width, &l.norm);
       ok = ok && carve(arena, base, width, &l.ls_attn);
       ok = ok && carve(arena, base, width, &l.ls_mlp);
+      if (plan.sandwich) {
+        ok = ok && carve(arena, base, width, &l.norm_after);
+        ok = ok && carve(arena, base, width, &l.norm_mlp);
+        ok = ok && carve(arena, base, width, &l.norm_mlp_after);
+      }
+      if (l.state_space) ok = ok && carve(arena, base, static_cast<uint64_t>(l.attn_pad), &l.group_norm);
       ok = ok && carve(arena, base, static_cast<uint64_t>(l.shape.rotary_pairs) + 1u, &l.frequency);
     }
     ok = ok && carve(arena, base, width, &plan.final_norm);
@@ -335,14 +359,14 @@ bool plan_state(Session *s, StaticArena &arena, void *base) {
     ParallelPlan &plan = *s->parallel;
     place_parallel_cache(&plan, s->kv_pages);
     const uint64_t words = plan.element_bytes() / 2u;
-    keys = plan.key_elems * words;
-    values = plan.value_elems * words;
+    keys = std::max<uint64_t>(plan.key_elems * words, 16u);
+    values = std::max<uint64_t>(plan.value_elems * words, 16u);
     hidden = plan.width_pad;
     qkv = plan.max_qkv_pad;
     attn = plan.max_attn_pad * words;
     ff = std::max<uint64_t>(plan.max_ff_pad, 8u) * words;
-    max_x = plan.width_pad * words;
-    partial_dim = plan.max_v_pad;
+    max_x = plan.x_width() * words;
+    partial_dim = std::max(plan.max_v_pad, 16u);
     s->kv_layer_elems = 0;
     s->max_splits = kWindowMaxSplits;
   }
@@ -353,8 +377,13 @@ bool plan_state(Session *s, StaticArena &arena, void *base) {
   ok = ok && carve(arena, base, hidden, &s->h_b);
   ok = ok && carve(arena, base, qkv, &s->qkv);
   ok = ok && carve(arena, base, std::max<uint64_t>(static_cast<uint64_t>(d.heads) * d.mla_rank, 4u), &s->mla_ql);
-  ok = ok && carve(arena, base, static_cast<uint64_t>(d.hidden), &s->o_out);
-  ok = ok && carve(arena, base, static_cast<uint64_t>(d.hidden), &s->down);
+  ok = ok && carve(arena, base, hidden, &s->o_out);
+  ok = ok && carve(arena, base, hidden, &s->down);
+  if (s->parallel) {
+    ok = ok && carve(arena, base, std::max<uint64_t>(s->parallel->recurrent_floats, 4u), &s->recurrent);
+    ok = ok && carve(arena, base, hidden, &s->first);
+    ok = ok && carve(arena, base, std::max<uint64_t>(s->parallel->max_space_pad, 4u), &s->mixed);
+  }
   ok = ok && carve(arena, base, static_cast<uint64_t>(d.vocab), &s->logits);
   // fused attention uses up to 16 spans, latent attention up to 64
   const uint64_t split_slots = std::max<uint32_t>(s->max_splits, d.mla() ? 64u : 16u);
@@ -664,13 +693,15 @@ cudaError_t enqueue_step(Session *s, uint32_t splits, uint32_t sample, uint64_t 
   if (!head_only) {
     if (s->parallel)
       err = launch_embed(s->stream, st, arena_at(s, s->layout.embeddings), d.hidden, s->h_b, s->parallel->embedding_scale,
-                         s->parallel->width_pad);
+                         s->parallel->width_pad, s->parallel->loop_input ? s->first : nullptr);
     else
       err = launch_embed(s->stream, st, arena_at(s, s->layout.embeddings), d.hidden, s->h_b);
     n += 1;
   }
   profile_mark(s, prof, kBucketEmbed);
-  if (s->parallel && !head_only && err == cudaSuccess) err = enqueue_parallel_layers(s, splits, &n, prof, profile_mark);
+  ResidualStream residual{s->h_b, nullptr, nullptr};
+  if (s->parallel && !head_only && err == cudaSuccess)
+    err = enqueue_parallel_layers(s, splits, &residual, &n, prof, profile_mark);
   for (uint32_t l = 0; !s->parallel && !head_only && err == cudaSuccess && l < d.layers; ++l) {
     const LayerLayout &L = s->layout.layers[l];
     ProjectionParams p{};
@@ -925,7 +956,7 @@ cudaError_t enqueue_step(Session *s, uint32_t splits, uint32_t sample, uint64_t 
   }
   uint32_t partials = 0;
   if (s->parallel && err == cudaSuccess && sample != 0) {
-    err = enqueue_parallel_head(s, &partials, &n);
+    err = enqueue_parallel_head(s, residual, &partials, &n);
     profile_mark(s, prof, kBucketLmHead);
   } else if (err == cudaSuccess && sample != 0) {
     ProjectionParams p{};
@@ -1115,7 +1146,9 @@ void fill_header(const Session *s, NervaCudaHfDecodeSequenceResult *out, uint32_
 }
 
 uint64_t resident_kv_bytes(const Session *s) {
-  if (s->parallel) return (s->parallel->key_elems + s->parallel->value_elems) * s->parallel->element_bytes();
+  if (s->parallel)
+    return (s->parallel->key_elems + s->parallel->value_elems) * s->parallel->element_bytes() +
+           s->parallel->recurrent_floats * sizeof(float);
   return (s->dims.mla() ? 1ull : 2ull) * s->dims.layers * s->kv_layer_elems * sizeof(uint16_t);
 }
 uint64_t device_footprint(const Session *s) {
@@ -1481,8 +1514,9 @@ cudaError_t allocate_state(Session *s, int32_t *stage) {
   // logical->physical table the identity, as the reference initialises it
   // (hf_decode_sequence/kernels.cu:732-739).
   // A page of a parallel-block session is 16 tokens of every layer run, K and V together.
-  const uint64_t page_bytes = s->parallel ? (s->parallel->key_elems + s->parallel->value_elems) / s->kv_pages *
-                                                s->parallel->element_bytes()
+  const uint64_t page_bytes = s->parallel ? std::max<uint64_t>((s->parallel->key_elems + s->parallel->value_elems) /
+                                                                   s->kv_pages * s->parallel->element_bytes(),
+                                                               16u)
                                           : NERVA_KV_CACHE_BLOCK_TOKENS * s->dims.kv_row() * 2u;
   StaticArena page_space(s->parallel ? page_bytes * s->kv_pages + 64u
                                      : 2ull * s->dims.layers * s->kv_layer_elems * 2u + 64u);
@@ -1737,6 +1771,7 @@ static int create_session(const NervaCudaHfDecodeSequenceSessionCreateRequest *r
   if (err == cudaSuccess) err = configure_mla_kernels();
   if (err == cudaSuccess && s->parallel) err = configure_parallel_projection();
   if (err == cudaSuccess && s->parallel) err = configure_window_attention();
+  if (err == cudaSuccess && s->parallel) err = configure_state_space();
   if (err != cudaSuccess) return create_fail(s, out, err, kStageSetDevice);
   if (d.mla() && !mla_session_supported(d.heads, d.mla_rank, d.mla_nope, d.mla_rope, d.head_dim)) {
     set_last_error("latent attention shape not supported: needs at most 16 heads, latent rank 128, 256 or 512, "

@@ -50,6 +50,11 @@ struct LayerLayout {
   uint64_t expert_stride = 0, expert_up_offset = 0;
   // parallel-block layers (rms_attn is the layer's one norm): per-channel scales of the two sublayers
   uint64_t ls_attn = kMissingOffset, ls_mlp = kMissingOffset;
+  // sandwich layers: the norms behind the sublayers (rms_attn, rms_mlp are those in front); attention's output
+  // gate; a state space's input projection (w_o is its output) and small tensors
+  uint64_t norm_after = kMissingOffset, norm_mlp_after = kMissingOffset, w_head_gate = kMissingOffset;
+  uint64_t w_space = kMissingOffset, conv = kMissingOffset, conv_bias = kMissingOffset, step_bias = kMissingOffset;
+  uint64_t a_log = kMissingOffset, skip = kMissingOffset, group_norm = kMissingOffset;
   // expert parallel: the experts whose matrices this arena holds (all of them otherwise)
   uint32_t expert_base = 0, expert_local = 0;
 };
@@ -57,6 +62,7 @@ struct LayerLayout {
 struct ArenaLayout {
   uint64_t embeddings = 0, input = 0, scratch = 0, final_norm = 0, lm_head = 0;
   uint64_t loop_vectors = kMissingOffset;  // [loop_times][hidden]
+  uint64_t loop_input = kMissingOffset;    // [hidden][2 hidden]
   uint64_t elements = 0;
   std::vector<LayerLayout> layers;
 };
@@ -88,14 +94,16 @@ bool layer_supported(const NervaCudaHfDecodeChainLayer &layer);
 ArenaLayout compute_arena_layout(const ModelDims &dims, const NervaCudaHfDecodeChainLayer *layers,
                                  const NervaB200ParallelModel *parallel = nullptr);
 
-// ---- parallel-block decoders (parallel_step.cu) ----
-// One layer: its attention shape and the padded copies of its weights the kernels read (every
+// ---- decoders described layer by layer (parallel_step.cu; sandwich blocks: sandwich_step.cu) ----
+// One layer: its mixer's shape and the padded copies of its weights the kernels read (every
 // dimension a projection sums over, and every output of the residual stream, rounded up to 64 with
 // zeros, so that neither TMA nor the norm prologue sees an odd size).
 struct ParallelLayerPlan {
-  WindowAttentionShape shape{};
+  bool state_space = false;
+  WindowAttentionShape shape{};               // attention
+  StateSpaceShape space{};                    // state space
   uint32_t intermediate = 0, ff_pad = 0;      // 0: no feed-forward
-  uint32_t qkv_rows = 0, qkv_pad = 0;         // [Q; K; V] rows, rounded up
+  uint32_t qkv_rows = 0, qkv_pad = 0;         // rows of the mixer's input projection ([Q; K; V; gates]), rounded up
   uint32_t attn_width = 0, attn_pad = 0;      // heads * v_dim
   bool layer_scale = false;
   std::vector<float> frequencies;
@@ -103,25 +111,41 @@ struct ParallelLayerPlan {
   uint16_t *w_o = nullptr;     // [width_pad][attn_pad]
   uint16_t *w_down = nullptr;  // [width_pad][ff_pad]
   uint16_t *norm = nullptr, *ls_attn = nullptr, *ls_mlp = nullptr;  // [width_pad]
+  uint16_t *norm_after = nullptr, *norm_mlp = nullptr, *norm_mlp_after = nullptr;  // [width_pad], sandwich blocks
+  uint16_t *group_norm = nullptr;             // [attn_pad], state space
   float *frequency = nullptr;
 };
-// One execution of a layer: a looped layer runs several times, each with its own part of the cache.
+// One execution of a layer: a looped layer runs several times, each with its own part of the cache or state.
 struct ParallelRun {
   uint32_t layer = 0;
   int32_t step = -1;  // row of the loop vectors added to the stream before this run, -1: none
   uint64_t key_offset = 0, value_offset = 0;  // elements from the start of a session's K / V array
+  uint64_t state_offset = 0, history_offset = 0;  // floats from the start of a session's recurrent state
 };
 struct ParallelPlan {
-  bool f32 = false;
+  bool f32 = false, sandwich = false;
+  uint32_t layer_norm = 0, activation = 0;
   uint32_t width = 0, width_pad = 0, vocab = 0, loop_times = 0;
-  float embedding_scale = 1.0f, softcap = 0.0f;
+  float embedding_scale = 1.0f, logit_scale = 0.0f, softcap = 0.0f;
   std::vector<ParallelLayerPlan> layers;
   std::vector<ParallelRun> runs;
   uint64_t key_elems = 0, value_elems = 0;    // per session, all runs
-  uint32_t max_heads = 0, max_qkv_pad = 0, max_attn_pad = 0, max_ff_pad = 0, max_v_pad = 0;
+  uint64_t recurrent_floats = 0;              // per session, all runs
+  uint32_t max_heads = 0, max_qkv_pad = 0, max_attn_pad = 0, max_ff_pad = 0, max_v_pad = 0;  // heads, v_pad: attention
+  uint32_t max_space_pad = 0, max_conv_width = 0;  // state-space layers: attn_pad, convolved row
   uint16_t *loop_vectors = nullptr;           // [loop_times][width_pad]
+  bool loop_input = false;
+  uint16_t *w_join = nullptr;                 // [width_pad][2 width_pad]: stream columns, embedding columns
   uint16_t *final_norm = nullptr, *head = nullptr;  // [width_pad], [vocab][width_pad]
   uint32_t element_bytes() const { return f32 ? 4u : 2u; }
+  uint32_t x_width() const { return loop_input ? 2u * width_pad : width_pad; }  // widest normalised activation row
+};
+// The residual stream of one token between two launches: h, and a sublayer output that has not joined it yet
+// (h + norm(pending) is the stream; sandwich blocks only).
+struct ResidualStream {
+  float *h = nullptr;
+  const float *pending = nullptr;
+  const uint16_t *after = nullptr;  // the weight of pending's norm
 };
 // Null (with the reason in last_error) when the description is inconsistent or beyond the kernels.
 std::shared_ptr<ParallelPlan> make_parallel_plan(const NervaB200ParallelModel &model, uint32_t width, uint32_t vocab,
@@ -131,10 +155,11 @@ void place_parallel_cache(ParallelPlan *plan, uint32_t pages);
 struct StepProfile;
 typedef void (*ProfileMark)(NervaCudaHfDecodeSequenceSession *, StepProfile *, uint32_t bucket);
 cudaError_t pack_parallel_weights(NervaCudaHfDecodeSequenceSession *s);
-// All layer runs of one decode step (s->h_b in and out), and its head; enqueue only.
-cudaError_t enqueue_parallel_layers(NervaCudaHfDecodeSequenceSession *s, uint32_t splits, uint64_t *launches,
-                                    StepProfile *prof, ProfileMark mark);
-cudaError_t enqueue_parallel_head(NervaCudaHfDecodeSequenceSession *s, uint32_t *partials, uint64_t *launches);
+// All layer runs of one decode step (stream: s->h_b in, what the head takes out), and its head; enqueue only.
+cudaError_t enqueue_parallel_layers(NervaCudaHfDecodeSequenceSession *s, uint32_t splits, ResidualStream *stream,
+                                    uint64_t *launches, StepProfile *prof, ProfileMark mark);
+cudaError_t enqueue_parallel_head(NervaCudaHfDecodeSequenceSession *s, const ResidualStream &stream, uint32_t *partials,
+                                  uint64_t *launches);
 uint32_t parallel_attention_splits(const ParallelPlan &plan, uint32_t target_context);
 uint64_t hash_tokens(const uint32_t *tokens, uint32_t count);
 uint64_t hash_weight_descriptors(const NervaCudaHfDecodeSequenceWeightBlock *blocks, uint32_t count);
@@ -159,7 +184,11 @@ struct BlockWorkspace {
   uint16_t *x_bf16 = nullptr;   // [max_rows][x_elems] normalised activations, the B operand of the next GEMM
   float *qkv = nullptr;         // [max_rows][A + 2 KV]
   uint16_t *attn = nullptr;     // [max_rows][A]
-  float *h_a = nullptr, *h_b = nullptr;  // [max_rows][hidden] residual stream, ping-pong
+  float *h_a = nullptr, *h_b = nullptr;  // [max_rows][hidden] residual stream, ping-pong; sandwich blocks keep
+                                         // the stream in h_b and a sublayer's output in h_a
+  float *first = nullptr;       // [max_rows][hidden] embedding output, where passes begin with it
+  float *mixed = nullptr;       // [max_rows][heads * v_dim] state-space output in front of its norm
+  void *convolved = nullptr;    // [max_rows][convolved row] of a state-space layer
   uint16_t *ff = nullptr;       // [max_rows][intermediate]
   float *logits = nullptr;      // [sample_rows][vocab]
   float *partial_acc = nullptr, *partial_m = nullptr, *partial_l = nullptr;  // split attention, per row
@@ -252,6 +281,20 @@ struct ParallelBlock {
   uint32_t capture_row;        // row of the capture buffer the first row of the block goes to
 };
 cudaError_t enqueue_parallel_block_layers(NervaCudaHfDecodeSequenceSession *s, const ParallelBlock &b, uint64_t *launches);
+// Pieces both kinds of block are made of: the norm between two projections, a projection of the block's rows, its attention (ws.qkv -> ws.attn),
+// the parameters of a layer run's attention, and the copy of the stream behind a layer run into the session's
+// capture buffer.
+StreamNormParams layer_stream_norm(const NervaCudaHfDecodeSequenceSession *s, float *h, const uint16_t *weight, void *x);
+cudaError_t parallel_block_gemm(NervaCudaHfDecodeSequenceSession *s, cudaStream_t stream, GemmParams g, uint32_t tokens);
+cudaError_t enqueue_block_attention(NervaCudaHfDecodeSequenceSession *s, const ParallelBlock &b, const ParallelLayerPlan &l,
+                                    const ParallelRun &run, uint64_t *launches);
+cudaError_t enqueue_step_attention(NervaCudaHfDecodeSequenceSession *s, const ParallelLayerPlan &l, const ParallelRun &run,
+                                   uint32_t splits, uint64_t *launches);
+cudaError_t capture_block_stream(NervaCudaHfDecodeSequenceSession *s, const ParallelBlock &b, size_t run);
+// Sandwich blocks (sandwich_step.cu).
+cudaError_t enqueue_sandwich_layers(NervaCudaHfDecodeSequenceSession *s, uint32_t splits, ResidualStream *stream,
+                                    uint64_t *launches, StepProfile *prof, ProfileMark mark);
+cudaError_t enqueue_sandwich_block_layers(NervaCudaHfDecodeSequenceSession *s, const ParallelBlock &b, uint64_t *launches);
 cudaError_t enqueue_parallel_block_head(NervaCudaHfDecodeSequenceSession *s, cudaStream_t stream, uint32_t count,
                                         const uint32_t *row_index, uint64_t *launches);
 
@@ -295,6 +338,9 @@ struct NervaCudaHfDecodeSequenceSession {
   uint32_t kv_pages = 0;
   uint32_t *page_table = nullptr;
   float *h_a = nullptr, *h_b = nullptr, *qkv = nullptr, *o_out = nullptr, *down = nullptr;
+  // decoders described layer by layer: recurrent state of all layer runs, the token's embedding output, and a
+  // state-space layer's output in front of its norm
+  float *recurrent = nullptr, *first = nullptr, *mixed = nullptr;
   float *logits = nullptr;
   float *partial_acc = nullptr, *partial_m = nullptr, *partial_l = nullptr;
   uint32_t max_splits = 1;

@@ -152,6 +152,65 @@ __device__ __forceinline__ void norm_single_finish(uint16_t *x, const NormValueR
   }
 }
 
+// Mean (zero for RMS norms) and 1 / sqrt(mean square deviation + eps) of the first `width` of the block's
+// values (zeros behind them), without cancellation: every warp takes the deviations from its own mean, and
+// the warps' results are merged.  One synchronisation; `scratch` holds 3 floats per warp and must not be in
+// use by an earlier call.
+struct NormMoments {
+  float mean, scale;
+};
+constexpr uint32_t kMomentsScratch = 3u * 32u;
+__device__ __forceinline__ NormMoments norm_moments(const float4 (&v)[kNormRegIters], uint32_t width, uint32_t layer_norm,
+                                                    float eps, float *scratch) {
+  const uint32_t lane = threadIdx.x & 31u, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  float sum = 0.0f;
+  uint32_t count = 0;
+#pragma unroll
+  for (uint32_t k = 0; k < kNormRegIters; ++k) {
+    const uint32_t first = 4u * (threadIdx.x + k * blockDim.x);
+    sum += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+    count += first >= width ? 0u : (width - first < 4u ? width - first : 4u);
+  }
+  const float n = static_cast<float>(__reduce_add_sync(0xffffffffu, count));
+  const float mean_w = layer_norm != 0 && n > 0.0f ? warp_sum(sum) / n : 0.0f;
+  float square = 0.0f;
+#pragma unroll
+  for (uint32_t k = 0; k < kNormRegIters; ++k) {
+    const uint32_t first = 4u * (threadIdx.x + k * blockDim.x);
+    const float d[4] = {v[k].x - mean_w, v[k].y - mean_w, v[k].z - mean_w, v[k].w - mean_w};
+#pragma unroll
+    for (uint32_t j = 0; j < 4u; ++j)
+      if (first + j < width) square = fmaf(d[j], d[j], square);
+  }
+  square = warp_sum(square);
+  if (lane == 0) {
+    scratch[3u * warp] = n;
+    scratch[3u * warp + 1u] = mean_w;
+    scratch[3u * warp + 2u] = square;
+  }
+  __syncthreads();
+  NormMoments m;
+  m.mean = 0.0f;
+  for (uint32_t w = 0; w < warps; ++w) m.mean = fmaf(scratch[3u * w], scratch[3u * w + 1u], m.mean);
+  m.mean /= static_cast<float>(width);
+  float total = 0.0f;
+  for (uint32_t w = 0; w < warps; ++w) {
+    const float d = scratch[3u * w + 1u] - m.mean;
+    total += fmaf(scratch[3u * w] * d, d, scratch[3u * w + 2u]);
+  }
+  m.scale = 1.0f / sqrtf(total / static_cast<float>(width) + eps);
+  return m;
+}
+// x = bf16((v - mean) * scale * w)
+__device__ __forceinline__ uint2 normed_bf16x4(const float4 &v, const uint2 &w, const NormMoments &m) {
+  uint2 out;
+  out.x = static_cast<uint32_t>(f32_to_bf16_bits((v.x - m.mean) * m.scale * bf16x2_lo(w.x))) |
+          (static_cast<uint32_t>(f32_to_bf16_bits((v.y - m.mean) * m.scale * bf16x2_hi(w.x))) << 16);
+  out.y = static_cast<uint32_t>(f32_to_bf16_bits((v.z - m.mean) * m.scale * bf16x2_lo(w.y))) |
+          (static_cast<uint32_t>(f32_to_bf16_bits((v.w - m.mean) * m.scale * bf16x2_hi(w.y))) << 16);
+  return out;
+}
+
 // Tensor-parallel form of the same prologue: `b` is the sum over the ranks of
 // partial vectors that arrive from the other GPUs while this runs.  recv holds
 // [world][cols] 8-byte entries, value bits in the low word and a tag in the high

@@ -2,6 +2,9 @@
 // separate query/key and value widths: a rotation of the leading dimensions of a head (its
 // frequencies and the factor on cos and sin come as a table, so plain and scaled rotations look
 // alike here), then an optional weightless RMS norm of q and k, softmax over the keys in the window.
+// Optionally the first positions stay visible behind the window (the kernels then walk the tiles that
+// hold them in front of the window's own), scores are soft-capped, and a sigmoid gate per head scales
+// the result.
 //
 //   window_attention_kernel   one query token per row.  The lone decode step (ROWS = false) prepares
 //                             q, appends the new K/V row and attends in one launch; block rows of an
@@ -76,6 +79,37 @@ __device__ __forceinline__ float dot_piece(const uint16_t *k, const float *q, fl
   return fmaf(bf16x2_hi(w.w), b.w, acc);
 }
 
+// The tiles of `size` tokens a query walks: those that hold kept first positions and lie in front of the
+// window, then the window's.
+struct TileWalk {
+  uint32_t kept, first;  // tiles in front; first tile of the window
+  __device__ __forceinline__ TileWalk(uint32_t keep_first, uint32_t lo, uint32_t size) {
+    first = lo / size;
+    kept = (keep_first + size - 1u) / size;
+    if (kept > first) kept = first;
+  }
+  __device__ __forceinline__ uint32_t count(uint32_t end, uint32_t size) const {  // tiles, for a window that ends at `end`
+    return kept + (end + size - 1u) / size - first;
+  }
+  __device__ __forceinline__ uint32_t tile(uint32_t i) const { return i < kept ? i : first + (i - kept); }
+};
+
+// Soft cap of a score that carries a factor log2(e).
+__device__ __forceinline__ float cap_score(float score, float cap2) { return cap2 * tanhf(score / cap2); }
+// The same through one exponential, absolute error a few 1e-7 of the cap.
+__device__ __forceinline__ float cap_score_fast(float score, float cap2, float inv_cap2) {
+  const float e = exp2f(score * inv_cap2 * (2.0f * kLog2e));
+  return cap2 - __fdividef(2.0f * cap2, e + 1.0f);
+}
+
+// Factor of a head's output.
+__device__ __forceinline__ float output_gate(const WindowAttentionParams &p, uint32_t row, uint32_t h) {
+  const WindowAttentionShape &s = p.s;
+  if (s.head_gate == 0) return 1.0f;
+  const uint32_t at = (s.heads + s.kv_heads) * s.qk_dim + s.kv_heads * s.v_dim + h;
+  return sigmoid(__ldcg(p.qkv + static_cast<uint64_t>(row) * p.qkv_stride + at));
+}
+
 // (sin, cos) of pair i at a position, with the magnitude of a scaled rotation.
 __device__ __forceinline__ float2 rotation(const WindowAttentionShape &s, uint32_t position, uint32_t i) {
   float2 t;
@@ -113,8 +147,9 @@ __device__ __forceinline__ uint64_t cache_row(uint32_t page, uint32_t token, uin
 }
 
 // Grid ((heads + kv_heads) / 8, rows), a warp per head: a query head is prepared in place, a KV head's K
-// and V go to the cache.
+// and V go to the cache.  Without rotation and norm there is nothing to prepare: KV heads only.
 constexpr uint32_t kPublishWarps = 8;
+__host__ __device__ inline bool queries_prepared(const WindowAttentionShape &s) { return s.rotary_pairs != 0 || s.qk_norm != 0; }
 template <class T>
 __global__ void __launch_bounds__(kPublishWarps * 32) window_publish_kernel(WindowAttentionParams p) {
   __shared__ float heads[kPublishWarps][256];
@@ -129,7 +164,8 @@ __global__ void __launch_bounds__(kPublishWarps * 32) window_publish_kernel(Wind
   for (uint32_t i = threadIdx.x; i < s.rotary_pairs; i += blockDim.x) turn[i] = rotation(s, r.position, i);
   __syncthreads();
   pdl_wait();
-  const uint32_t lane = threadIdx.x & 31u, unit = blockIdx.x * kPublishWarps + (threadIdx.x >> 5);
+  const uint32_t lane = threadIdx.x & 31u;
+  const uint32_t unit = (queries_prepared(s) ? 0u : s.heads) + blockIdx.x * kPublishWarps + (threadIdx.x >> 5);
   if (unit >= s.heads + s.kv_heads) return;
   float *head = heads[threadIdx.x >> 5];
   const bool query = unit < s.heads;
@@ -234,10 +270,11 @@ __device__ __forceinline__ void merge_spans(const WindowAttentionParams &p, uint
       }
     }
     T *out = reinterpret_cast<T *>(p.out) + static_cast<uint64_t>(row) * p.out_stride + h * s.v_dim;
+    const float gate = output_gate(p, row, h);
 #pragma unroll
     for (uint32_t i = 0; i < 2u * PAIRS; ++i) {
       const uint32_t d = 2u * lane + 64u * (i / 2u) + (i & 1u);
-      if (d < s.v_dim) to_cache(out + d, a[i]);
+      if (d < s.v_dim) to_cache(out + d, a[i] * gate);
     }
   }
   if (threadIdx.x == 0) *counter = 0;  // ready for the next launch
@@ -296,26 +333,27 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   const uint32_t head0 = kvh * group + sub * kHeadsPerBlock;
   const uint32_t left_heads = group - sub * kHeadsPerBlock;
   const uint32_t hb = left_heads < kHeadsPerBlock ? left_heads : kHeadsPerBlock;
-  // cached tokens [lo, hist) are seen; the lone step's own token comes from the projection
+  // cached tokens [lo, hist) and those below keep_first are seen; the lone step's own token comes from the projection
   const uint32_t hist = ROWS ? position + 1u : position;
   const uint32_t lo = s.window != 0 && position + 1u > s.window ? position + 1u - s.window : 0u;
-  const uint32_t first_chunk = lo / chunk_tokens;
-  const uint32_t chunks = (hist + chunk_tokens - 1u) / chunk_tokens - first_chunk;  // lo <= hist: never negative
-  const uint32_t chunk_begin = first_chunk + chunks * span / S;
-  const uint32_t chunk_end = first_chunk + chunks * (span + 1u) / S;
+  const TileWalk walk(s.keep_first, lo, chunk_tokens);
+  const uint32_t chunks = walk.count(hist, chunk_tokens);  // lo <= hist: never negative
+  const uint32_t chunk_begin = chunks * span / S, chunk_end = chunks * (span + 1u) / S;  // numbers in the walk
   const bool owns_current = !ROWS && span + 1u == S;
 
   const uint32_t k_pieces = s.qk_pad * static_cast<uint32_t>(sizeof(T)) / 16u;
   const uint32_t v_pieces = s.v_pad * static_cast<uint32_t>(sizeof(T)) / 16u;
   const uint32_t row_pieces = k_pieces + v_pieces;
-  auto issue = [&](uint32_t chunk, uint32_t stage) {
+  auto issue = [&](uint32_t number, uint32_t stage) {
+    const uint32_t chunk = walk.tile(number);
     uint8_t *k_stage = smem + stage * layout.stage;
     uint8_t *v_stage = k_stage + chunk_tokens * layout.k_row;
     const uint32_t first = chunk * chunk_tokens;
     // the chunk's page-table entries, one per lane, handed out by shuffle
     const uint32_t pages = chunk_tokens / kPageTokens;
     uint32_t my_page = 0;
-    if (lane < pages && first + lane * kPageTokens < hist && first + (lane + 1u) * kPageTokens > lo) {
+    const uint32_t page_token = first + lane * kPageTokens;
+    if (lane < pages && page_token < hist && (page_token + kPageTokens > lo || page_token / kTile * kTile < s.keep_first)) {
       my_page = table[first / kPageTokens + lane];
       if (my_page >= page_count) {
         report_error(error_word, kErrPageOutOfRange);
@@ -326,7 +364,8 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
     for (uint32_t t = warp; t < chunk_tokens; t += kWarps) {
       const uint32_t page = __shfl_sync(0xffffffffu, my_page, t / kPageTokens);
       const uint32_t token = first + t;
-      if (token < lo || token >= hist) continue;
+      // a tile with kept tokens is copied whole: its invisible rows meet probabilities of zero
+      if (token >= hist || (token < lo && token / kTile * kTile >= s.keep_first)) continue;
       const T *k_src = keys + cache_row(page, token, s.kv_heads, kvh, s.qk_pad);
       const T *v_src = values + cache_row(page, token, s.kv_heads, kvh, s.v_pad);
       for (uint32_t c = lane; c < row_pieces; c += 32u) {
@@ -349,7 +388,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   }
 
   const float *qkv = p.qkv + static_cast<uint64_t>(row) * p.qkv_stride;
-  const float qscale = s.scale * kLog2e;
+  const float qscale = s.scale * kLog2e, cap2 = s.softcap * kLog2e;
   for (uint32_t w = warp; w < hb; w += kWarps) {
     float *q = q_sh + w * s.qk_pad;
     const float *src = qkv + (head0 + w) * s.qk_dim;
@@ -410,13 +449,15 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
       const uint32_t item = warp + u * kWarps;
       if (item < items) {
         const uint32_t tile = item / hb, head = item - tile * hb;
-        const uint32_t first = chunk * chunk_tokens + tile * kTile;
-        // the tile's visible tokens [first + t0, first + t1)
-        const uint32_t t0 = lo > first ? lo - first : 0u;
-        const uint32_t t1 = hist > first ? (hist - first < kTile ? hist - first : kTile) : 0u;
+        const uint32_t first = walk.tile(chunk) * chunk_tokens + tile * kTile;
+        // the tile's visible tokens lie in [first + t0, first + t1)
+        const bool kept = first < s.keep_first;
+        const uint32_t t0 = lo > first && !kept ? lo - first : 0u;
+        const uint32_t end = kept && lo >= first + kTile && s.keep_first < hist ? s.keep_first : hist;
+        const uint32_t t1 = end > first ? (end - first < kTile ? end - first : kTile) : 0u;
         if (t0 < t1) {
           float score = -INFINITY;
-          if (lane >= t0 && lane < t1) {
+          if (lane >= t0 && lane < t1 && (first + lane >= lo || first + lane < s.keep_first)) {
             const T *k_row = reinterpret_cast<const T *>(k_stage + (tile * kTile + lane) * layout.k_row);
             const float *q = q_sh + head * s.qk_pad;
             constexpr uint32_t kElems = 16u / sizeof(T);
@@ -426,6 +467,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
               part[1] = dot_piece(k_row + (c + 1u) * kElems, q + (c + 1u) * kElems, part[1]);
             }
             score = part[0] + part[1];
+            if (s.softcap > 0.0f) score = cap_score(score, cap2);
           }
           const float m_new = fmaxf(m_run[u], warp_max(score));  // some token of the tile is visible: finite
           const float pr = exp2f(score - m_new);
@@ -497,6 +539,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
       float dot = 0.0f;
       for (uint32_t i = lane; i < s.qk_pad; i += 32u) dot = fmaf(q[i], k_new[i], dot);
       dot = warp_sum(dot);
+      if (s.softcap > 0.0f) dot = cap_score(dot, cap2);
       float v[2u * PAIRS];
 #pragma unroll
       for (uint32_t j = 0; j < PAIRS; ++j) {
@@ -507,7 +550,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
       fold(dot, 1.0f, v);
     }
     if (S == 1u) {
-      const float inv = 1.0f / l;
+      const float inv = output_gate(p, row, h) / l;
 #pragma unroll
       for (uint32_t i = 0; i < 2u * PAIRS; ++i) {
         const uint32_t d = 2u * lane + 64u * (i / 2u) + (i & 1u);
@@ -576,17 +619,18 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
   const uint32_t hb = left_heads < kHeadsPerBlock ? left_heads : kHeadsPerBlock;
   const uint32_t hist = r.position + 1u;
   const uint32_t lo = s.window != 0 && hist > s.window ? hist - s.window : 0u;
-  const uint32_t first_page = lo / kPageTokens;
-  const uint32_t pages = (hist + kPageTokens - 1u) / kPageTokens - first_page;
-  const uint32_t page_begin = first_page + pages * span / S, page_end = first_page + pages * (span + 1u) / S;
+  const TileWalk walk(s.keep_first, lo, kPageTokens);
+  const uint32_t pages = walk.count(hist, kPageTokens);
+  const uint32_t page_begin = pages * span / S, page_end = pages * (span + 1u) / S;  // numbers in the walk
   const uint32_t first = page_begin + warp;
+  auto visible = [&](uint32_t token) { return token < hist && (token >= lo || token < s.keep_first); };
   const uint32_t my_pages = first < page_end ? (page_end - first + kRowWarps - 1u) / kRowWarps : 0u;
 
   uint8_t *ring = smem + warp * L.ring;
   const uint32_t k_pieces = s.qk_pad / 8u, v_pieces = s.v_pad / 8u, row_pieces = k_pieces + v_pieces;
   auto issue = [&](uint32_t i) {  // one commit group per page, also when there is none left
     if (i < my_pages) {
-      const uint32_t logical = first + i * kRowWarps;
+      const uint32_t logical = walk.tile(first + i * kRowWarps);
       uint32_t page = r.page_table[logical];
       if (page >= r.page_count) {
         report_error(r.error_word, kErrPageOutOfRange);
@@ -609,7 +653,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
         } else {  // tokens outside the window are filled with zeros
 #pragma unroll
           for (uint32_t t = 0; t < kPageTokens; ++t)
-            cp_async_zfill<16>(dst + t * dst_step, src + t * src_step, token0 + t >= lo && token0 + t < hist);
+            cp_async_zfill<16>(dst + t * dst_step, src + t * src_step, visible(token0 + t));
         }
       }
     }
@@ -618,7 +662,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
   issue(0);
   issue(1);
 
-  const float qscale = s.scale * kLog2e;
+  const float qscale = s.scale * kLog2e, cap2 = s.softcap * kLog2e, inv_cap2 = cap2 > 0.0f ? 1.0f / cap2 : 0.0f;
   const float *q_in = p.qkv + static_cast<uint64_t>(row) * p.qkv_stride + head0 * s.qk_dim;
   const uint32_t q_pairs = s.qk_pad / 2u;
   for (uint32_t i = threadIdx.x; i < kHeadsPerBlock * q_pairs; i += blockDim.x) {
@@ -644,7 +688,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
     __syncwarp();
     const uint32_t k_base = smem_addr(ring + (i % kRowStages) * L.stage);
     const uint32_t v_base = k_base + kPageTokens * L.k_row;
-    const uint32_t token0 = (first + i * kRowWarps) * kPageTokens;
+    const uint32_t token0 = walk.tile(first + i * kRowWarps) * kPageTokens;
     float sc[2][4];
 #pragma unroll
     for (uint32_t n = 0; n < 2u; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.0f;
@@ -661,7 +705,8 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
 #pragma unroll
     for (uint32_t j = 0; j < 4u; ++j) {
       const uint32_t token = token0 + 8u * (j >> 1) + 2u * t4 + (j & 1u);
-      if (token < lo || token >= hist) v[j] = -INFINITY;
+      if (s.softcap > 0.0f) v[j] = cap_score_fast(v[j], cap2, inv_cap2);
+      if (!visible(token)) v[j] = -INFINITY;
     }
     float m_page = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
     m_page = fmaxf(m_page, __shfl_xor_sync(0xffffffffu, m_page, 1));
@@ -729,7 +774,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
     if (S == 1u) {
       if (d < s.v_dim)
         reinterpret_cast<uint16_t *>(p.out)[static_cast<uint64_t>(row) * p.out_stride + (head0 + h) * s.v_dim + d] =
-            f32_to_bf16_bits(a / l);
+            f32_to_bf16_bits(a / l * output_gate(p, row, head0 + h));
     } else {
       const uint64_t slot = (static_cast<uint64_t>(row) * s.heads + head0 + h) * S + span;
       p.partial_acc[slot * s.v_pad + d] = a;
@@ -795,12 +840,13 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
 
   const uint32_t kv_lo = s.window != 0 && pos_first + 1u > s.window ? pos_first + 1u - s.window : 0u;
   const uint32_t kv_end = pos_last + 1u;
-  const uint32_t tile_begin = kv_lo / kKeyTile + key_group, tile_end = (kv_end + kKeyTile - 1u) / kKeyTile;
+  const TileWalk walk(s.keep_first, kv_lo, kKeyTile);
+  const uint32_t tile_begin = key_group, tile_end = walk.count(kv_end, kKeyTile);  // numbers in the walk
   const uint32_t k_pieces = s.qk_pad / 8u, v_pieces = s.v_pad / 8u, row_pieces = k_pieces + v_pieces;
   auto issue = [&](uint32_t tile) {
     uint8_t *k_stage = stages + ((tile - tile_begin) / GROUPS & 1u) * L.stage;
     uint8_t *v_stage = k_stage + kKeyTile * L.k_row;
-    const uint32_t first = tile * kKeyTile;
+    const uint32_t first = walk.tile(tile) * kKeyTile;
     uint32_t my_page = 0;
     if (lane < kKeyTile / kPageTokens && first + lane * kPageTokens < kv_end) {
       my_page = r0.page_table[first / kPageTokens + lane];
@@ -828,7 +874,7 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
   if (tile_begin + GROUPS < tile_end) issue(tile_begin + GROUPS);
 
   // queries, scaled so that the softmax runs on exp2, as a bf16 rounding and its remainder
-  const float qscale = s.scale * kLog2e;
+  const float qscale = s.scale * kLog2e, cap2 = s.softcap * kLog2e, inv_cap2 = cap2 > 0.0f ? 1.0f / cap2 : 0.0f;
   const uint32_t q_pairs = s.qk_pad / 2u;
   for (uint32_t i = threadIdx.x; i < kTileRows * q_pairs; i += GROUPS * kPrefillThreads) {
     const uint32_t row = i / q_pairs, d = 2u * (i - row * q_pairs);
@@ -875,7 +921,7 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
     group_sync();
     const uint32_t k_base = smem_addr(stages + ((tile - tile_begin) / GROUPS & 1u) * L.stage);
     const uint32_t v_base = k_base + kKeyTile * L.k_row;
-    const uint32_t first = tile * kKeyTile;
+    const uint32_t first = walk.tile(tile) * kKeyTile;
     float sc[8][4];
 #pragma unroll
     for (uint32_t n = 0; n < 8u; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.0f;
@@ -893,7 +939,14 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
         mma_bf16(sc[2u * np + 1u], al, kb[2], kb[3]);
       }
     }
-    // visible: 0 <= pos - token < window
+    if (s.softcap > 0.0f) {
+#pragma unroll
+      for (uint32_t n = 0; n < 8u; ++n) {
+#pragma unroll
+        for (uint32_t j = 0; j < 4u; ++j) sc[n][j] = cap_score_fast(sc[n][j], cap2, inv_cap2);
+      }
+    }
+    // visible: 0 <= pos - token, and pos - token < window or token < keep_first
     float m_tile[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (uint32_t n = 0; n < 8u; ++n) {
@@ -901,7 +954,7 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
       for (uint32_t j = 0; j < 4u; ++j) {
         const uint32_t token = first + n * 8u + 2u * t4 + (j & 1u);
         const uint32_t i = j >> 1;
-        if (!(token <= pos[i] && pos[i] - token < window)) sc[n][j] = -INFINITY;
+        if (!(token <= pos[i] && (pos[i] - token < window || token < s.keep_first))) sc[n][j] = -INFINITY;
         m_tile[i] = fmaxf(m_tile[i], sc[n][j]);
       }
     }
@@ -1001,7 +1054,7 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
     const uint32_t f = f0 + warp * 16u + g + 8u * i;
     uint16_t *dst = reinterpret_cast<uint16_t *>(p.out) + static_cast<uint64_t>(f / group) * p.out_stride +
                     (kvh * group + f % group) * s.v_dim;
-    const float inv = 1.0f / l_run[i];
+    const float inv = output_gate(p, f / group, kvh * group + f % group) / l_run[i];
 #pragma unroll
     for (uint32_t n = 0; n < NT; ++n) {
       const uint32_t d = n * 8u + 2u * t4;
@@ -1063,14 +1116,14 @@ bool window_attention_supported(const WindowAttentionShape &s, bool f32) {
 
 // Spans for a step whose context is at most target_context: one 64-token chunk per block up to
 // kWindowMaxSplits, in powers of two so that a growing context re-captures the step rarely, but never
-// more than a full window (which may begin and end inside a chunk) needs.
-uint32_t window_attention_splits(uint32_t target_context, uint32_t window) {
+// more than a full window (which may begin and end inside a chunk) and the kept first positions need.
+uint32_t window_attention_splits(uint32_t target_context, uint32_t window, uint32_t keep_first) {
   constexpr uint32_t kChunk = 2u * kTile;
   const uint32_t chunks = target_context / kChunk + (target_context % kChunk != 0 ? 1u : 0u);
   uint32_t s = 1;
   while (s < chunks && s < kWindowMaxSplits) s <<= 1;
   if (window != 0) {
-    const uint32_t most = (window - 1u) / kChunk + 2u;
+    const uint32_t most = (window - 1u) / kChunk + 2u + keep_first / kChunk + (keep_first % kChunk != 0 ? 1u : 0u);
     if (s > most) s = most;
   }
   return s;
@@ -1081,7 +1134,8 @@ uint32_t window_attention_splits(uint32_t target_context, uint32_t window) {
 uint32_t window_rows_splits(const WindowAttentionShape &s, uint32_t rows, uint32_t longest_context, uint32_t sm_count) {
   const uint32_t group = s.heads / s.kv_heads;
   uint32_t keys = longest_context;
-  if (s.window != 0 && s.window + kPageTokens < keys) keys = s.window + kPageTokens;
+  const uint64_t seen = static_cast<uint64_t>(s.window) + kPageTokens + (s.keep_first != 0 ? s.keep_first + kPageTokens : 0u);
+  if (s.window != 0 && seen < keys) keys = static_cast<uint32_t>(seen);
   const uint32_t splits =
       attention_default_splits(keys, rows, s.kv_heads * ((group + kHeadsPerBlock - 1u) / kHeadsPerBlock), sm_count);
   return splits > kWindowMaxSplits ? kWindowMaxSplits : splits;
@@ -1111,7 +1165,8 @@ cudaError_t configure_window_attention() {
 
 cudaError_t launch_window_publish(cudaStream_t stream, const WindowAttentionParams &p) {
   if (p.rows == nullptr || p.row_count == 0 || p.row_count > 65535u) return cudaErrorInvalidValue;
-  const dim3 grid((p.s.heads + p.s.kv_heads + kPublishWarps - 1u) / kPublishWarps, p.row_count);
+  const uint32_t units = p.s.kv_heads + (queries_prepared(p.s) ? p.s.heads : 0u);
+  const dim3 grid((units + kPublishWarps - 1u) / kPublishWarps, p.row_count);
   return launch_with_pdl(p.f32 != 0 ? window_publish_kernel<float> : window_publish_kernel<uint16_t>, grid,
                          dim3(kPublishWarps * 32), 0, stream, p.pdl != 0, p);
 }

@@ -34,6 +34,32 @@ class ParallelLayer:
     scaling: dict | None = None  # factor, original, fast, slow
     qk_norm: bool = True
     layer_scale: bool = True
+    keep_first: int = 0     # positions below this stay visible behind the window
+    score_softcap: float = 0.0
+    head_gate: bool = False
+
+    def fill(self, out) -> None:
+        """This layer as a NervaB200ParallelLayer."""
+        out.heads, out.kv_heads, out.qk_dim, out.v_dim = self.heads, self.kv_heads, self.qk_dim, self.v_dim
+        out.intermediate, out.window, out.rotary_dims = self.intermediate, self.window, self.rotary_dims
+        out.qk_norm, out.layer_scale, out.score_scale = int(self.qk_norm), int(self.layer_scale), self.score_scale
+        out.keep_first, out.score_softcap, out.head_gate = self.keep_first, self.score_softcap, int(self.head_gate)
+        out.rotary_base = self.rotary_base
+        if self.scaling:
+            out.yarn_factor, out.yarn_original = self.scaling["factor"], self.scaling["original"]
+            out.yarn_fast, out.yarn_slow = self.scaling["fast"], self.scaling["slow"]
+
+
+def native_model(cfg, compute: str, **fields):
+    """The NervaB200ParallelModel of a configuration's layer_specs and loop; fields: the model's own."""
+    layers = (ffi.structs["NervaB200ParallelLayer"] * cfg.layers)()
+    for out, spec in zip(layers, cfg.layer_specs):
+        spec.fill(out)
+    model = ffi.structs["NervaB200ParallelModel"](
+        layer_count=cfg.layers, compute=COMPUTE[compute], loop_start=cfg.loop_start, loop_stop=cfg.loop_stop,
+        loop_times=cfg.loop_times, layers=C.cast(layers, C.c_void_p), **fields)
+    model._keep = layers
+    return model
 
 
 @dataclass(frozen=True)
@@ -109,6 +135,9 @@ class ParallelConfig:
         looped = sum(per_layer[self.loop_start:self.loop_stop]) if self.loop_times else 0
         return sum(per_layer) + (self.loop_times - 1 if self.loop_times else 0) * looped + 2 * self.vocab * self.hidden
 
+    def native_model(self, compute: str):
+        return native_model(self, compute, embedding_scale=self.embedding_scale, logit_softcap=self.logit_softcap)
+
     @classmethod
     def from_json(cls, config: dict, name: str = ARCHITECTURE) -> "ParallelConfig":
         """From a parsed config.json (sizes that only tensor shapes carry come from there: see load)."""
@@ -135,7 +164,8 @@ class ParallelConfig:
 
 @dataclass
 class ParallelCheckpoint:
-    """A configuration and its tensors: uint16 arrays of bf16 bits, or FileTensor ranges of a file."""
+    """A configuration (this module's, or one of the same interface) and its tensors: uint16 arrays of bf16
+    bits, or FileTensor ranges of a file."""
     config: ParallelConfig
     tensors: dict
 
@@ -154,22 +184,7 @@ class ParallelCheckpoint:
 
     def native_model(self, compute: str):
         """The NervaB200ParallelModel of the create call."""
-        cfg = self.config
-        layers = (ffi.structs["NervaB200ParallelLayer"] * cfg.layers)()
-        for out, s in zip(layers, cfg.layer_specs):
-            out.heads, out.kv_heads, out.qk_dim, out.v_dim = s.heads, s.kv_heads, s.qk_dim, s.v_dim
-            out.intermediate, out.window, out.rotary_dims = s.intermediate, s.window, s.rotary_dims
-            out.qk_norm, out.layer_scale, out.score_scale = int(s.qk_norm), int(s.layer_scale), s.score_scale
-            out.rotary_base = s.rotary_base
-            if s.scaling:
-                out.yarn_factor, out.yarn_original = s.scaling["factor"], s.scaling["original"]
-                out.yarn_fast, out.yarn_slow = s.scaling["fast"], s.scaling["slow"]
-        model = ffi.structs["NervaB200ParallelModel"](
-            layer_count=cfg.layers, compute=COMPUTE[compute], loop_start=cfg.loop_start, loop_stop=cfg.loop_stop,
-            loop_times=cfg.loop_times, embedding_scale=cfg.embedding_scale, logit_softcap=cfg.logit_softcap,
-            layers=C.cast(layers, C.c_void_p))
-        model._keep = layers
-        return model
+        return self.config.native_model(compute)
 
 
 def random_checkpoint(cfg: ParallelConfig, seed: int = 0, std: float = 0.02, fill=None) -> ParallelCheckpoint:

@@ -10,10 +10,11 @@ from __future__ import annotations
 import json
 import os
 
-from . import parallel_model
+from . import parallel_model, sandwich_model
 
 LOADERS = {
     parallel_model.ARCHITECTURE: parallel_model.load,
+    sandwich_model.ARCHITECTURE: sandwich_model.load,
 }
 
 
