@@ -778,13 +778,29 @@ def vuvolix_config(size: str, window: int):
                              loop_times=2)
 
 
-def run_vuvolix_workload(args) -> None:
-    """Prefill and decode of the Vuvolix design (parallel blocks, windowed attention, a looped range of layers)
-    beside the dense model of equal layer shapes: per size one JSON line with both models' prefill tok/s at
-    several prompt lengths, batch-1 decode tok/s after the longest prompt, and the packed step of 16 forks.
-    Device time (CUDA events inside the library) for prefill and decode; wall clock around the calls for the
-    packed step.  Every timed decode step streams more weight bytes than the L2 holds."""
-    from nerva_b200 import build, ops, parallel_model, synth
+# The Vamidra design at the same widths: attention and state-space layers in turn (inner width twice the hidden
+# size, heads of 64, a state of 128), the middle third of the layers run twice.  Beside it Vuvolix.
+def vamidra_config(size: str, window: int):
+    from nerva_b200 import sandwich_model as sm
+    hidden, heads, kv_heads, dim, inter, vocab, runs = VUVOLIX_SIZES[size]
+    layers = runs - runs // 3
+    attention = sm.attention_layer(heads=heads, kv_heads=kv_heads, qk_dim=dim, v_dim=dim, intermediate=inter, window=window,
+                                   keep_first=4, score_scale=dim ** -0.5, score_softcap=50.0)
+    space = sm.StateSpaceLayer(heads=hidden // 32, v_dim=64, state=128, groups=8, conv=4, norm_groups=8, intermediate=inter)
+    start = (layers - runs // 3) // 2
+    return sm.SandwichConfig(name=f"vamidra-{size}", hidden=hidden, vocab=vocab, rms_eps=1e-5,
+                             layer_specs=tuple(space if i % 2 else attention for i in range(layers)), logit_scale=0.5,
+                             loop_start=start, loop_stop=start + runs // 3, loop_times=2)
+
+
+def run_layered_workload(args) -> None:
+    """Prefill and decode of a design described layer by layer beside its closest relative at equal sizes: Vuvolix
+    (parallel blocks, windowed attention, a looped range of layers) beside the dense model of the same layer shapes,
+    Vamidra (sandwich blocks, attention and state-space mixers in turn) beside Vuvolix.  Per size one JSON line with
+    both models' prefill tok/s at several prompt lengths, batch-1 decode tok/s after the longest prompt, and the
+    packed step of 16 forks.  Device time (CUDA events inside the library) for prefill and decode; wall clock around
+    the calls for the packed step.  Every timed decode step streams more weight bytes than the L2 holds."""
+    from nerva_b200 import build, ops, parallel_model, sandwich_model, synth
     from nerva_b200.session import CudaHfDecodeSequenceLoop, CudaHfDecodeSequenceSession, SmokeStatus
     build.build()
     prompts = [args.prompt_tokens] if args.prompt_tokens else [256, 512, 2048]
@@ -792,20 +808,28 @@ def run_vuvolix_workload(args) -> None:
     peaks = measured_peaks()
     for size in [args.shape] if args.shape else list(VUVOLIX_SIZES):
         hidden, heads, kv_heads, dim, inter, vocab, runs = VUVOLIX_SIZES[size]
-        cfg = vuvolix_config(size, window)
         dense = synth.DecoderConfig(f"dense-{size}", layers=runs, hidden=hidden, heads=heads, kv_heads=kv_heads, head_dim=dim,
                                     intermediate=inter, vocab=vocab)
-        line = {"workload": "vuvolix beside the dense model of equal layer shapes", "size": size, "steps": args.steps,
+        relative = vuvolix_config(size, window)
+        models = {"vuvolix": (relative, lambda: parallel_model.random_checkpoint(relative, fill=ops.synth_normal_bf16),
+                              relative.streamed_bytes_per_token())}
+        cfg = relative
+        if args.workload == "vuvolix":
+            what = "vuvolix beside the dense model of equal layer shapes"
+            models["dense"] = (dense, lambda: synth.dense_checkpoint(dense, fill=ops.synth_normal_bf16),
+                               dense.projection_bytes_per_token())
+        else:
+            what = "vamidra beside vuvolix at equal widths"
+            cfg = vamidra_config(size, window)
+            models = {"vamidra": (cfg, lambda: sandwich_model.random_checkpoint(cfg, fill=ops.synth_normal_bf16),
+                                  cfg.streamed_bytes_per_token()), **models}
+        line = {"workload": what, "size": size, "steps": args.steps,
                 "config": {"hidden": hidden, "heads": heads, "kv_heads": kv_heads, "head_size": dim, "intermediate": inter,
                            "vocab": vocab, "layer_runs": runs, "window": window, "layers": cfg.layers,
                            "loop": [cfg.loop_start, cfg.loop_stop, cfg.loop_times], "weights": "random-init bf16 (synthetic)",
                            "l2": "every step streams more weight bytes than the L2 holds"}}
-        for name, model, nbytes in (("vuvolix", cfg, cfg.streamed_bytes_per_token()),
-                                    ("dense", dense, dense.projection_bytes_per_token())):
-            if name == "vuvolix":
-                ck = parallel_model.random_checkpoint(cfg, fill=ops.synth_normal_bf16)
-            else:
-                ck = synth.dense_checkpoint(dense, fill=ops.synth_normal_bf16)
+        for name, (model, make, nbytes) in models.items():
+            ck = make()
             context = max(prompts) + max(args.warmup, 3) + args.steps + 48 + MAX_EXTRA_CLOCK_STEPS
             session = CudaHfDecodeSequenceSession(ck, context, use_descriptors=True)
             del ck
@@ -976,13 +1000,13 @@ def main() -> None:
     ap.add_argument("--layers", type=int, default=0,
                     help="cut the model to this many layers (profiler captures only; not a bench line)")
     ap.add_argument("--prompt-tokens", type=int, default=0, help="override the prompt length")
-    ap.add_argument("--workload", default="decode", choices=["decode", "linear", "attention", "reference-gpu", "batch", "deepseek", "vuvolix"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "linear", "attention", "reference-gpu", "batch", "deepseek", "vuvolix", "vamidra"],
                     help="decode: the bench line; linear / attention: per-operator sweeps of the isolated "
                          "projection shapes and of long-context attention (one JSON line per case)")
-    ap.add_argument("--shape", default="", help="vuvolix: only this size (0.6b, 1.7b, 8b); linear sweep: only this projection (qkv, o, gate_up, down, lm_head)")
+    ap.add_argument("--shape", default="", help="vuvolix and vamidra: only this size (0.6b, 1.7b, 8b); linear sweep: only this projection (qkv, o, gate_up, down, lm_head)")
     ap.add_argument("--tokens", type=int, default=0, help="linear sweep: only this block size")
     ap.add_argument("--batch", type=int, default=0, help="attention sweep: only this batch size")
-    ap.add_argument("--context", type=int, default=0, help="attention sweep: only this context length; vuvolix: the window")
+    ap.add_argument("--context", type=int, default=0, help="attention sweep: only this context length; vuvolix and vamidra: the window")
     ap.add_argument("--shard-of", type=int, default=0, choices=[0, 2, 4, 8],
                     help="attention sweep on one GPU: measure one rank's shard of an N-way split by KV head")
     ap.add_argument("--timeline", action="store_true",
@@ -1008,9 +1032,9 @@ def main() -> None:
         if rank == 0:
             run_operator_workloads(args.workload, args.shape, args.tokens, args.batch, args.context)
         return
-    if args.workload == "vuvolix":
+    if args.workload in ("vuvolix", "vamidra"):
         if rank == 0:
-            run_vuvolix_workload(args)
+            run_layered_workload(args)
         return
     cfg = workload(args.config, args.layers, args.prompt_tokens)
     if args.workload == "reference-gpu":

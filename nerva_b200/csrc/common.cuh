@@ -218,14 +218,13 @@ __device__ __forceinline__ uint4 lds128(const void *p) {
 __device__ __forceinline__ float silu(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
 __device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
-__device__ __forceinline__ float gelu_tanh(float v) {
-  return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * v * v, v, v)));
-}
 
-// Activation of the gate in a gated feed-forward.
+// Activation of the gate in a gated feed-forward.  With (1 + tanh u) / 2 = sigmoid(2 u) the tanh form of
+// gelu is v * sigmoid(2 sqrt(2 / pi) (v + 0.044715 v^3)): both are v times a sigmoid.
 enum Activation : uint32_t { kActivationSilu = 0, kActivationGeluTanh = 1 };
 __device__ __forceinline__ float activate(uint32_t activation, float v) {
-  return activation == kActivationGeluTanh ? gelu_tanh(v) : silu(v);
+  const float u = activation == kActivationGeluTanh ? 1.5957691216057308f * fmaf(0.044715f * v * v, v, v) : v;
+  return v / (1.0f + expf(-u));
 }
 
 }  // namespace nb

@@ -233,26 +233,29 @@ __device__ __forceinline__ void row_epilogue(const GemmKernelParams &p, const fl
     // rows interleaved (gate, up): the neighbouring lane holds the other half of the pair
     const uint32_t base = p.epilogue == kEpilogueStoreSwiglu ? p.split_row : 0u;
     const uint32_t width = (p.rows - base) / 2u;
+    auto store = [&](auto act) {  // one loop per activation: the epilogue's last tile is not hidden behind anything
 #pragma unroll
-    for (uint32_t j = 0; j < N; ++j) {
-      const float other = __shfl_xor_sync(0xffffffffu, v[j], 1);
-      const uint32_t m = m0 + j;
-      if ((lane & 1u) == 0 && row + 1u < p.rows && m < p.tokens)
-        p.out_bf16[static_cast<uint64_t>(m) * width + (row - base) / 2u] = f32_to_bf16_bits(activate(p.activation, v[j]) * other);
-    }
+      for (uint32_t j = 0; j < N; ++j) {
+        const float other = __shfl_xor_sync(0xffffffffu, v[j], 1);
+        const uint32_t m = m0 + j;
+        if ((lane & 1u) == 0 && row + 1u < p.rows && m < p.tokens)
+          p.out_bf16[static_cast<uint64_t>(m) * width + (row - base) / 2u] = f32_to_bf16_bits(act(v[j]) * other);
+      }
+    };
+    if (p.activation == kActivationSilu)
+      store([](float x) { return silu(x); });
+    else
+      store([](float x) { return activate(kActivationGeluTanh, x); });
   } else if (row < p.rows) {
     const uint32_t width = p.epilogue == kEpilogueStoreSwiglu ? p.split_row : p.rows;
-    const float scale = p.row_scale != nullptr ? bf16_bits_to_f32(p.row_scale[row]) : 1.0f;
+    const float scale = (p.row_scale != nullptr ? bf16_bits_to_f32(p.row_scale[row]) : 1.0f) * (p.scale != 0.0f ? p.scale : 1.0f);
     const float add = p.row_add != nullptr ? bf16_bits_to_f32(p.row_add[row]) : 0.0f;
 #pragma unroll
     for (uint32_t j = 0; j < N; ++j) {
       const uint32_t m = m0 + j;
       if (m < p.tokens) {
         const uint64_t at = static_cast<uint64_t>(m) * width + row;
-        float y = v[j];
-        if (p.row_scale != nullptr) y *= scale;
-        if (p.row_add != nullptr) y += add;
-        if (p.scale != 0.0f) y *= p.scale;
+        float y = fmaf(v[j], scale, add);
         if (p.softcap > 0.0f) y = p.softcap * tanhf(y / p.softcap);
         p.out_f32[at] = p.resid_in != nullptr ? y + __ldcg(p.resid_in + at) : y;
       }
@@ -547,10 +550,10 @@ uint32_t gemm_smem_bytes(uint32_t n_pad, uint32_t stages) {
 uint32_t gemm_blocks(uint32_t rows, uint32_t cols, uint32_t sm_count) {
   const Partition p = make_partition(rows, cols, 1);
   const uint32_t want = 2u * sm_count;
-  // Between one and two row tiles per SM (gate/up of the 8B shapes: 192 tiles): one block per tile.
-  // Nothing is split, so no fix-up launch follows; the SMs that hold two blocks stream twice the
+  // Between (about) one and two row tiles per SM (gate/up of the 8B shapes: 192 tiles): one block per
+  // tile.  Nothing is split, so no fix-up launch follows; the SMs that hold two blocks stream twice the
   // bytes of the others, which the memory system evens out better than a second launch costs.
-  if (p.tiles >= sm_count && p.tiles <= want) return p.tiles;
+  if (p.tiles * 8u >= sm_count * 7u && p.tiles <= want) return p.tiles;
   return p.total < want ? static_cast<uint32_t>(p.total) : want;
 }
 

@@ -114,9 +114,9 @@ struct GemmParams {
                            // kEpilogueStoreSwiglu: out_f32[token][split_row], out_bf16[token][(rows - split_row)/2]
   uint32_t split_row;
   const uint16_t *row_scale;  // optional bf16 [rows], kEpilogueStore: y * row_scale[row] is what is stored / added
-  const uint16_t *row_add;    // optional bf16 [rows], kEpilogueStore: added to what is stored
+  const uint16_t *row_add;    // optional bf16 [rows], kEpilogueStore: added to y
   uint32_t activation;     // of the gate in gate/up pairs (common.cuh Activation)
-  float scale;             // kEpilogueStore: 0, or a factor on y (in front of the soft cap)
+  float scale;             // kEpilogueStore: 0, or a factor on y like row_scale (in front of row_add and the soft cap)
   float softcap;           // kEpilogueStore: 0, or softcap * tanh(y / softcap) is stored
   const float *resid_in;   // optional [tokens][rows]; may be out_f32
   float *out_f32;          // [tokens][rows]

@@ -30,12 +30,16 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// Two fp32 values -> one register of two bf16 roundings (low half first), and what the rounding lost.
+// Two fp32 values -> one register of two bf16 roundings (low half first; to nearest, ties to even), and
+// what the rounding lost.
 __device__ __forceinline__ uint32_t pack_bf16_hi(float x, float y) {
-  return static_cast<uint32_t>(f32_to_bf16_bits(x)) | (static_cast<uint32_t>(f32_to_bf16_bits(y)) << 16);
+  uint32_t r;
+  asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r) : "f"(y), "f"(x));
+  return r;
 }
 __device__ __forceinline__ uint32_t pack_bf16_lo(float x, float y) {
-  return pack_bf16_hi(x - bf16_round(x), y - bf16_round(y));
+  const uint32_t hi = pack_bf16_hi(x, y);
+  return pack_bf16_hi(x - bf16x2_lo(hi), y - bf16x2_hi(hi));
 }
 
 }  // namespace nb

@@ -433,6 +433,45 @@ __device__ __forceinline__ NormMoments row_moments(const float *row, const Strea
   return m;
 }
 
+// A row's pending output and norm with every value read once: the sandwich prologue for a block of rows.
+template <class X>
+__device__ __forceinline__ void norm_in_registers(const StreamNormParams &p, float *row, uint32_t source) {
+  __shared__ float scratch[2u * kMomentsScratch];
+  const uint32_t vecs = p.padded / 4u;
+  NormValueRegs h, y;
+  norm_single_load(h, row, p.padded);
+  if (p.pending != nullptr) {
+    norm_single_load(y, p.pending + static_cast<uint64_t>(source) * p.padded, p.padded);
+    const NormMoments m = norm_moments(y.v, p.width, p.layer_norm, p.eps, scratch);
+#pragma unroll
+    for (uint32_t k = 0; k < kNormRegIters; ++k) {
+      const uint32_t i = threadIdx.x + k * kNormThreads;
+      if (i < vecs) {
+        const uint2 w = reinterpret_cast<const uint2 *>(p.after)[i];
+        h.v[k].x += (y.v[k].x - m.mean) * m.scale * bf16x2_lo(w.x);
+        h.v[k].y += (y.v[k].y - m.mean) * m.scale * bf16x2_hi(w.x);
+        h.v[k].z += (y.v[k].z - m.mean) * m.scale * bf16x2_lo(w.y);
+        h.v[k].w += (y.v[k].w - m.mean) * m.scale * bf16x2_hi(w.y);
+        reinterpret_cast<float4 *>(row)[i] = h.v[k];
+      }
+    }
+  }
+  if (p.x == nullptr) return;
+  const NormMoments m = norm_moments(h.v, p.width, p.layer_norm, p.eps, scratch + kMomentsScratch);
+  X *out = reinterpret_cast<X *>(p.x) + static_cast<uint64_t>(blockIdx.x) * p.padded;
+#pragma unroll
+  for (uint32_t k = 0; k < kNormRegIters; ++k) {
+    const uint32_t i = threadIdx.x + k * kNormThreads;
+    if (i < vecs) {
+      const uint2 w = reinterpret_cast<const uint2 *>(p.norm)[i];
+      store_act(out + 4u * i, (h.v[k].x - m.mean) * m.scale * bf16x2_lo(w.x));
+      store_act(out + 4u * i + 1u, (h.v[k].y - m.mean) * m.scale * bf16x2_hi(w.x));
+      store_act(out + 4u * i + 2u, (h.v[k].z - m.mean) * m.scale * bf16x2_lo(w.y));
+      store_act(out + 4u * i + 3u, (h.v[k].w - m.mean) * m.scale * bf16x2_hi(w.y));
+    }
+  }
+}
+
 // One block per row.
 template <class X>
 __global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(StreamNormParams p) {
@@ -441,6 +480,10 @@ __global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(StreamNormPar
   pdl_wait();
   const uint32_t source = p.row_index != nullptr ? p.row_index[blockIdx.x] : blockIdx.x;
   float *row = p.h + static_cast<uint64_t>(source) * p.padded;
+  if (p.layer_norm != 0 && p.step == nullptr && p.first == nullptr && p.padded <= 4u * kNormRegIters * kNormThreads) {
+    norm_in_registers<X>(p, row, source);
+    return;
+  }
   if (p.step != nullptr) {
     for (uint32_t i = threadIdx.x * 4u; i < p.padded; i += kNormThreads * 4u) {
       float4 v = *reinterpret_cast<const float4 *>(row + i);

@@ -32,21 +32,26 @@ constexpr uint32_t kStepThreads = 256;
 constexpr uint32_t kStepWarps = kStepThreads / 32;
 
 // ---------------------------------------------------------------- one token per row ----
-// Lane = value column, warp w = state rows w, w + 8, ...; ROWS_PER: of them a thread holds.
-template <uint32_t ROWS_PER>
+// A thread holds four neighbouring columns of state rows r, r + 32, ...: eight threads span a block's 32
+// columns.  ROWS_PER: rows a thread holds.  VECTOR: v_dim is a multiple of 4, so that the four columns are
+// one 16-byte access.
+template <uint32_t ROWS_PER, bool VECTOR>
 __global__ void __launch_bounds__(kStepThreads) state_space_step_kernel(StateSpaceParams p) {
-  constexpr uint32_t kChannels = (kColumns + 2u * kStepWarps * ROWS_PER + kStepThreads - 1u) / kStepThreads;
-  __shared__ float values[kColumns + 2u * kStepWarps * ROWS_PER];  // x | B | C behind convolution and silu
-  __shared__ float part[kStepWarps][kColumns];
+  constexpr uint32_t kRowStep = kStepThreads / 8u;
+  constexpr uint32_t kMaxValues = kColumns + 2u * kRowStep * ROWS_PER;
+  constexpr uint32_t kChannels = (kMaxValues + kStepThreads - 1u) / kStepThreads;
+  __shared__ __align__(16) float values[kMaxValues];  // x | B | C behind convolution and silu
+  __shared__ __align__(16) float part[kStepWarps][kColumns];
   const StateSpaceShape &s = p.s;
   const uint32_t lane = threadIdx.x & 31u, warp = threadIdx.x >> 5;
   const uint32_t tiles = (s.v_dim + kColumns - 1u) / kColumns;
   const uint32_t head = blockIdx.x / tiles, column0 = (blockIdx.x - head * tiles) * kColumns;
   const uint32_t group = head / (s.heads / s.groups);
+  const bool several = p.rows != nullptr;
   pdl_trigger();
   uint32_t position, max_context;
   float *recurrent;
-  if (p.rows != nullptr) {
+  if (several) {
     const FusedAttentionRow &r = p.rows[blockIdx.y];
     position = r.position;
     max_context = r.max_context;
@@ -60,83 +65,131 @@ __global__ void __launch_bounds__(kStepThreads) state_space_step_kernel(StateSpa
     pdl_wait();
     return;
   }
-  const uint32_t column = column0 + lane;
-  const bool live = column < s.v_dim;
-  float *state = recurrent + p.state_offset + static_cast<uint64_t>(head) * s.state * s.v_dim + column;
-  float held[ROWS_PER];
+  const uint32_t quad = 4u * (threadIdx.x & 7u), row0 = threadIdx.x >> 3;  // columns column0 + quad .. + 3
+  float *state = recurrent + p.state_offset + static_cast<uint64_t>(head) * s.state * s.v_dim + column0 + quad;
+  float held[ROWS_PER][4];
 #pragma unroll
   for (uint32_t i = 0; i < ROWS_PER; ++i) {
-    const uint32_t n = warp + i * kStepWarps;
-    held[i] = live && n < s.state && position != 0 ? __ldcg(state + static_cast<uint64_t>(n) * s.v_dim) : 0.0f;
+    const uint32_t n = row0 + i * kRowStep;
+    const float *src = state + static_cast<uint64_t>(n) * s.v_dim;
+#pragma unroll
+    for (uint32_t j = 0; j < 4u; ++j) held[i][j] = 0.0f;
+    if (n < s.state && position != 0) {
+      if (VECTOR) {
+        if (column0 + quad < s.v_dim) {
+          const float4 v = __ldcg(reinterpret_cast<const float4 *>(src));
+          held[i][0] = v.x;
+          held[i][1] = v.y;
+          held[i][2] = v.z;
+          held[i][3] = v.w;
+        }
+      } else {
+#pragma unroll
+        for (uint32_t j = 0; j < 4u; ++j)
+          if (column0 + quad + j < s.v_dim) held[i][j] = __ldcg(src + j);
+      }
+    }
   }
 
-  // the convolution of this block's x columns and of its group's B and C, up to the current token
+  // the convolution of this block's x columns and of its group's B and C
   const uint32_t inner = s.inner(), channels = s.channels(), shared = s.groups * s.state;
   float *history = recurrent + p.history_offset;
   const float *in = p.in + static_cast<uint64_t>(blockIdx.y) * p.in_stride;
   const uint32_t wanted = kColumns + 2u * s.state;
   auto channel_of = [&](uint32_t i) {  // channels: none
+    if (i >= wanted) return channels;
     if (i < kColumns) return column0 + i < s.v_dim ? head * s.v_dim + column0 + i : channels;
     const uint32_t n = i - kColumns;
     return n < s.state ? inner + group * s.state + n : inner + shared + group * s.state + (n - s.state);
   };
-  float sum[kChannels], newest[kChannels];
+  const uint32_t column = column0 + lane;
+  const bool live = column < s.v_dim;
+  float sum[kChannels], newest[kChannels], u[kChannels], step_in = 0.0f, z = 0.0f;
+  auto load_inputs = [&]() {
+#pragma unroll
+    for (uint32_t k = 0; k < kChannels; ++k) {
+      const uint32_t ch = channel_of(threadIdx.x + k * kStepThreads);
+      u[k] = ch < channels ? __ldcg(in + inner + ch) : 0.0f;
+    }
+    step_in = __ldcg(in + inner + channels + head);
+    if (live && warp == 0) z = __ldcg(in + head * s.v_dim + column);
+  };
+  // Alone, what the earlier tokens left is summed while the projection still runs.  With many rows most blocks
+  // start after it has ended, and all loads travel together.
+  if (several) {
+    pdl_wait();
+    load_inputs();
+  }
 #pragma unroll
   for (uint32_t k = 0; k < kChannels; ++k) {
-    const uint32_t i = threadIdx.x + k * kStepThreads;
-    const uint32_t ch = i < wanted ? channel_of(i) : channels;
+    const uint32_t ch = channel_of(threadIdx.x + k * kStepThreads);
     sum[k] = newest[k] = 0.0f;
     if (ch < channels) {
       const uint16_t *w = p.conv + static_cast<uint64_t>(ch) * s.taps;
       sum[k] = bf16_bits_to_f32(p.conv_bias[ch]);
       newest[k] = bf16_bits_to_f32(w[s.taps - 1u]);
-      for (uint32_t back = 1; back < s.taps && back <= position; ++back)
-        sum[k] = fmaf(bf16_bits_to_f32(w[s.taps - 1u - back]),
-                      __ldcg(history + static_cast<uint64_t>((position - back) % s.taps) * channels + ch), sum[k]);
+#pragma unroll 3
+      for (uint32_t back = 1; back < s.taps; ++back) {
+        if (back <= position)
+          sum[k] = fmaf(bf16_bits_to_f32(w[s.taps - 1u - back]),
+                        __ldcg(history + static_cast<uint64_t>((position - back) % s.taps) * channels + ch), sum[k]);
+      }
     }
   }
   const float rate = expf(bf16_bits_to_f32(p.a_log[head])), bias = bf16_bits_to_f32(p.step_bias[head]);
   const float skip = bf16_bits_to_f32(p.skip[head]);
+  if (!several) {
+    pdl_wait();
+    load_inputs();
+  }
 
-  pdl_wait();
   const bool owns_shared = column0 == 0 && head % (s.heads / s.groups) == 0;
 #pragma unroll
   for (uint32_t k = 0; k < kChannels; ++k) {
-    const uint32_t i = threadIdx.x + k * kStepThreads;
-    if (i < wanted) {
-      const uint32_t ch = channel_of(i);
-      float v = 0.0f;
-      if (ch < channels) {
-        const float u = __ldcg(in + inner + ch);
-        v = silu(fmaf(newest[k], u, sum[k]));
-        if (i < kColumns || owns_shared) history[static_cast<uint64_t>(position % s.taps) * channels + ch] = u;
-      }
-      values[i] = v;
-    }
+    const uint32_t i = threadIdx.x + k * kStepThreads, ch = channel_of(i);
+    if (i < wanted) values[i] = ch < channels ? silu(fmaf(newest[k], u[k], sum[k])) : 0.0f;
+    if (ch < channels && (i < kColumns || owns_shared)) history[static_cast<uint64_t>(position % s.taps) * channels + ch] = u[k];
   }
-  const float step = softplus(__ldcg(in + inner + channels + head) + bias);
+  const float step = softplus(step_in + bias);
   const float decay = expf(-rate * step);
-  const float z = live && warp == 0 ? __ldcg(in + head * s.v_dim + column) : 0.0f;
   __syncthreads();
-  const float x = values[lane], fed = step * x;
+  const float4 x4 = *reinterpret_cast<const float4 *>(values + quad);
+  const float fed[4] = {step * x4.x, step * x4.y, step * x4.z, step * x4.w};
   const float *b = values + kColumns, *c = b + s.state;
-  float y = 0.0f;
+  float y[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
   for (uint32_t i = 0; i < ROWS_PER; ++i) {
-    const uint32_t n = warp + i * kStepWarps;
+    const uint32_t n = row0 + i * kRowStep;
     if (n < s.state) {
-      held[i] = fmaf(decay, held[i], fed * b[n]);
-      y = fmaf(held[i], c[n], y);
-      if (live) state[static_cast<uint64_t>(n) * s.v_dim] = held[i];
+      const float bn = b[n], cn = c[n];
+#pragma unroll
+      for (uint32_t j = 0; j < 4u; ++j) {
+        held[i][j] = fmaf(decay, held[i][j], fed[j] * bn);
+        y[j] = fmaf(held[i][j], cn, y[j]);
+      }
+      float *dst = state + static_cast<uint64_t>(n) * s.v_dim;
+      if (VECTOR) {
+        if (column0 + quad < s.v_dim)
+          *reinterpret_cast<float4 *>(dst) = make_float4(held[i][0], held[i][1], held[i][2], held[i][3]);
+      } else {
+#pragma unroll
+        for (uint32_t j = 0; j < 4u; ++j)
+          if (column0 + quad + j < s.v_dim) dst[j] = held[i][j];
+      }
     }
   }
-  part[warp][lane] = y;
+#pragma unroll
+  for (uint32_t j = 0; j < 4u; ++j) {  // the warp's four rows
+    y[j] += __shfl_xor_sync(0xffffffffu, y[j], 8);
+    y[j] += __shfl_xor_sync(0xffffffffu, y[j], 16);
+  }
+  if (lane < 8u) *reinterpret_cast<float4 *>(&part[warp][quad]) = make_float4(y[0], y[1], y[2], y[3]);
   __syncthreads();
   if (warp != 0 || !live) return;
-  y = skip * x;
+  float total = skip * values[lane];
 #pragma unroll
-  for (uint32_t w = 0; w < kStepWarps; ++w) y += part[w][lane];
-  p.out[static_cast<uint64_t>(blockIdx.y) * p.out_stride + head * s.v_dim + column] = y * silu(z);
+  for (uint32_t w = 0; w < kStepWarps; ++w) total += part[w][lane];
+  p.out[static_cast<uint64_t>(blockIdx.y) * p.out_stride + head * s.v_dim + column] = total * silu(z);
 }
 
 // ---------------------------------------------------------------- a block of one session ----
@@ -322,7 +375,10 @@ __global__ void __launch_bounds__(kStepThreads) state_space_rows_kernel(StateSpa
 
 // ------------------------------------------------------------------ chunks on the tensor pipe ----
 constexpr uint32_t kChunk = 64;
-constexpr uint32_t kScanThreads = 128;
+constexpr uint32_t kScanThreads = 256;
+constexpr uint32_t kScanWarps = kScanThreads / 32u;
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr uint32_t kScanMaxRows = 256;  // rows of a block
 
 __device__ __forceinline__ void cp_async_16(void *dst, const void *src, bool valid) {  // zeros when not valid
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(valid ? 16u : 0u)
@@ -346,17 +402,20 @@ struct ScanLayout {  // bytes; rows are an odd number of 16-byte pieces apart (l
   }
 };
 
-// Grid (value columns / 32, heads).  MT: m-tiles of 16 state rows a warp holds (state <= 64 MT).
+// Grid (value columns / 32, heads).  MT: m-tiles of 16 state rows a warp holds (state <= 128 MT).  Outputs: warps
+// 0..3 take 16 columns of the token tiles 0..3, warps 4..7 the other 16 columns of the tiles 3..0, so that the
+// two warps of an SM partition share the triangle of earlier tokens evenly.
 template <uint32_t MT>
 __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpaceParams p) {
-  constexpr uint32_t NT = kColumns / 8u;
+  constexpr uint32_t NT = kColumns / 8u, YT = NT / 2u;
   extern __shared__ __align__(128) uint8_t smem[];
-  __shared__ float log_decay[kChunk], steps[kChunk], to_end[kChunk];
+  __shared__ float log_decay_all[kScanMaxRows], steps_all[kScanMaxRows], to_end_all[kScanMaxRows];
   const StateSpaceShape &s = p.s;
   const ScanLayout L(s);
   uint8_t *fed_hi = smem + 2u * L.stage, *fed_lo = fed_hi + L.fed;
   uint8_t *state_hi = fed_lo + L.fed, *state_lo = state_hi + L.states;
   const uint32_t lane = threadIdx.x & 31u, warp = threadIdx.x >> 5, g = lane >> 2, t4 = lane & 3u;
+  const uint32_t token_tile = warp < 4u ? warp : kScanWarps - 1u - warp, y_first = warp < 4u ? 0u : kColumns / 2u;
   const uint32_t head = blockIdx.y, column0 = blockIdx.x * kColumns;
   const uint32_t group = head / (s.heads / s.groups);
   const uint32_t n_pad = s.state_pad(), m_tiles = n_pad / 16u;
@@ -364,7 +423,7 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
   const FusedAttentionRow &r0 = p.rows[0];
   const uint32_t base = r0.position;
   float *state = r0.recurrent + p.state_offset + static_cast<uint64_t>(head) * s.state * s.v_dim + column0;
-  // held[m][n]: state rows 16 (warp + 4 m) + g (+ 8), columns 8 n + 2 t (+ 1); written by an earlier block step
+  // held[m][n]: state rows 16 (warp + 8 m) + g (+ 8), columns 8 n + 2 t (+ 1); written by an earlier block step
   float held[MT][NT][4];
 #pragma unroll
   for (uint32_t m = 0; m < MT; ++m) {
@@ -372,15 +431,15 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
     for (uint32_t n = 0; n < NT; ++n) {
 #pragma unroll
       for (uint32_t j = 0; j < 4u; ++j) {
-        const uint32_t row = 16u * (warp + 4u * m) + g + 8u * (j >> 1), col = 8u * n + 2u * t4 + (j & 1u);
+        const uint32_t row = 16u * (warp + kScanWarps * m) + g + 8u * (j >> 1), col = 8u * n + 2u * t4 + (j & 1u);
         held[m][n][j] = base != 0 && row < s.state && column0 + col < s.v_dim
                             ? __ldcg(state + static_cast<uint64_t>(row) * s.v_dim + col)
                             : 0.0f;
       }
     }
   }
-  const float rate = expf(bf16_bits_to_f32(p.a_log[head])), bias = bf16_bits_to_f32(p.step_bias[head]);
-  const float skip = bf16_bits_to_f32(p.skip[head]);
+  const float rate = kLog2e * expf(bf16_bits_to_f32(p.a_log[head]));  // decays are powers of two here
+  const float bias = bf16_bits_to_f32(p.step_bias[head]), skip = bf16_bits_to_f32(p.skip[head]);
   pdl_wait();
   if (base + p.row_count > r0.max_context) return;
 
@@ -393,18 +452,27 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
   const uint32_t pieces = 2u * n_pieces + x_pieces;
   auto issue = [&](uint32_t chunk) {  // one commit group per chunk
     uint8_t *b = smem + (chunk & 1u) * L.stage, *c = b + kChunk * L.n_row, *x = c + kChunk * L.n_row;
-    for (uint32_t i = threadIdx.x; i < kChunk * pieces; i += kScanThreads) {
-      const uint32_t t = i / pieces, piece = i - t * pieces, r = chunk * kChunk + t;
-      const bool inside = r < p.row_count;
-      const uint64_t at = static_cast<uint64_t>(inside ? r : 0u) * width;
-      if (piece < n_pieces) {
-        cp_async_16(b + t * L.n_row + piece * 16u, b_src + at + piece * 8u, inside);
-      } else if (piece < 2u * n_pieces) {
-        cp_async_16(c + t * L.n_row + (piece - n_pieces) * 16u, c_src + at + (piece - n_pieces) * 8u, inside);
-      } else {
+    const uint32_t first = chunk * kChunk;
+    // a lane takes one 16-byte piece of the B, C or x row of every eighth token
+    for (uint32_t piece = lane; piece < pieces; piece += 32u) {
+      const uint16_t *src = b_src + piece * 8u;
+      uint8_t *dst = b + piece * 16u;
+      uint32_t dst_step = L.n_row;
+      bool used = true;
+      if (piece >= 2u * n_pieces) {
         const uint32_t e = piece - 2u * n_pieces;
-        const bool valid = inside && e < x_valid;
-        cp_async_16(x + t * L.x_row + e * 16u, x_src + at + (valid ? e * 8u : 0u), valid);
+        used = e < x_valid;
+        src = x_src + (used ? e * 8u : 0u);
+        dst = x + e * 16u;
+        dst_step = L.x_row;
+      } else if (piece >= n_pieces) {
+        src = c_src + (piece - n_pieces) * 8u;
+        dst = c + (piece - n_pieces) * 16u;
+      }
+#pragma unroll
+      for (uint32_t t = warp; t < kChunk; t += kScanWarps) {
+        const bool inside = first + t < p.row_count;
+        cp_async_16(dst + t * dst_step, src + static_cast<uint64_t>(inside ? first + t : 0u) * width, inside && used);
       }
     }
     cp_async_commit();
@@ -417,51 +485,55 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
 
   const uint32_t chunks = (p.row_count + kChunk - 1u) / kChunk;
   issue(0);
+  for (uint32_t chunk = warp; chunk < chunks; chunk += kScanWarps) {
+    // step sizes and their running sums, a chunk per warp: tokens 2 lane, 2 lane + 1; rows behind the block change nothing
+    float d[2], sum[2];
+#pragma unroll
+    for (uint32_t i = 0; i < 2u; ++i) {
+      const uint32_t r = chunk * kChunk + 2u * lane + i;
+      d[i] = r < p.row_count
+                 ? softplus(__ldcg(p.in + static_cast<uint64_t>(r) * p.in_stride + s.inner() + s.channels() + head) + bias)
+                 : 0.0f;
+    }
+    sum[0] = d[0];
+    sum[1] = d[0] + d[1];
+    float through = sum[1], from = sum[1];  // sums up to and from this lane's tokens
+#pragma unroll
+    for (uint32_t o = 1; o < 32u; o <<= 1) {
+      const float left = __shfl_up_sync(0xffffffffu, through, o), right = __shfl_down_sync(0xffffffffu, from, o);
+      if (lane >= o) through += left;
+      if (lane + o < 32u) from += right;
+    }
+    float before = __shfl_up_sync(0xffffffffu, through, 1), behind = __shfl_down_sync(0xffffffffu, from, 1);
+    if (lane == 0) before = 0.0f;
+    if (lane == 31) behind = 0.0f;
+#pragma unroll
+    for (uint32_t i = 0; i < 2u; ++i) {
+      const uint32_t t = chunk * kChunk + 2u * lane + i;
+      steps_all[t] = d[i];
+      log_decay_all[t] = -rate * (before + sum[i]);
+      // not a difference of the running sums: the last token's factor is exactly one
+      to_end_all[t] = exp2f(-rate * (i == 0 ? behind + d[1] : behind)) * d[i];
+    }
+  }
   for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
     const uint32_t first = chunk * kChunk;
-    if (warp == 0) {
-      // step sizes and their running sum: tokens 2 lane, 2 lane + 1; rows behind the block change nothing
-      float d[2], sum[2];
-#pragma unroll
-      for (uint32_t i = 0; i < 2u; ++i) {
-        const uint32_t r = first + 2u * lane + i;
-        d[i] = r < p.row_count
-                   ? softplus(__ldcg(p.in + static_cast<uint64_t>(r) * p.in_stride + s.inner() + s.channels() + head) + bias)
-                   : 0.0f;
-      }
-      sum[0] = d[0];
-      sum[1] = d[0] + d[1];
-      float before = sum[1];
-#pragma unroll
-      for (uint32_t o = 1; o < 32u; o <<= 1) {
-        const float left = __shfl_up_sync(0xffffffffu, before, o);
-        if (lane >= o) before += left;
-      }
-      const float end = __shfl_sync(0xffffffffu, before, 31);
-      before -= sum[1];
-#pragma unroll
-      for (uint32_t i = 0; i < 2u; ++i) {
-        const uint32_t t = 2u * lane + i;
-        steps[t] = d[i];
-        log_decay[t] = -rate * (before + sum[i]);
-        to_end[t] = expf(-rate * (end - (before + sum[i]))) * d[i];
-      }
-    }
+    const float *log_decay = log_decay_all + first, *steps = steps_all + first, *to_end = to_end_all + first;
     cp_async_wait<0>();
     __syncthreads();  // this chunk's rows and steps are in place; the other stage is free
     if (chunk + 1u < chunks) issue(chunk + 1u);
     uint8_t *b_sh = smem + (chunk & 1u) * L.stage, *c_sh = b_sh + kChunk * L.n_row, *x_sh = c_sh + kChunk * L.n_row;
 
     // z of this thread's outputs, on its way while the products run
-    float z[2][NT][2];
+    float z[2][YT][2];
 #pragma unroll
     for (uint32_t i = 0; i < 2u; ++i) {
-      const uint32_t r = first + 16u * warp + g + 8u * i;
+      const uint32_t r = first + 16u * token_tile + g + 8u * i;
 #pragma unroll
-      for (uint32_t n = 0; n < NT; ++n) {
+      for (uint32_t n = 0; n < YT; ++n) {
 #pragma unroll
         for (uint32_t j = 0; j < 2u; ++j) {
-          const uint32_t col = column0 + 8u * n + 2u * t4 + j;
+          const uint32_t col = column0 + y_first + 8u * n + 2u * t4 + j;
           z[i][n][j] = r < p.row_count && col < s.v_dim
                            ? __ldcg(p.in + static_cast<uint64_t>(r) * p.in_stride + head * s.v_dim + col)
                            : 0.0f;
@@ -471,7 +543,7 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
     // state at the chunk's start and x scaled for its end, both as two bf16 parts
 #pragma unroll
     for (uint32_t m = 0; m < MT; ++m) {
-      const uint32_t tile = warp + 4u * m;
+      const uint32_t tile = warp + kScanWarps * m;
       if (tile < m_tiles) {
 #pragma unroll
         for (uint32_t n = 0; n < NT; ++n) {
@@ -493,42 +565,40 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
     }
     __syncthreads();
 
-    // what the state gives: rows 16 warp + g (+ 8) of the chunk
-    float y[NT][4];
+    // what the state gives: rows 16 token_tile + g (+ 8) of the chunk
+    float y[YT][4];
 #pragma unroll
-    for (uint32_t n = 0; n < NT; ++n) y[n][0] = y[n][1] = y[n][2] = y[n][3] = 0.0f;
-    const uint32_t c_addr = smem_addr(c_sh) + (16u * warp + a_row) * L.n_row + a_off;
+    for (uint32_t n = 0; n < YT; ++n) y[n][0] = y[n][1] = y[n][2] = y[n][3] = 0.0f;
+    const uint32_t c_addr = smem_addr(c_sh) + (16u * token_tile + a_row) * L.n_row + a_off;
+#pragma unroll 4
     for (uint32_t ks = 0; ks < n_pad / 16u; ++ks) {
-      uint32_t ca[4];
+      uint32_t ca[4], hi[4], lo[4];
       ldmatrix_x4(ca, c_addr + ks * 32u);
-#pragma unroll
-      for (uint32_t np = 0; np < NT / 2u; ++np) {
-        uint32_t hi[4], lo[4];
-        const uint32_t at = (ks * 16u + kn_row) * L.x_row + np * 32u + kn_off;
-        ldmatrix_x4_trans(hi, smem_addr(state_hi) + at);
-        ldmatrix_x4_trans(lo, smem_addr(state_lo) + at);
-        mma_bf16(y[2u * np], ca, hi[0], hi[1]);
-        mma_bf16(y[2u * np], ca, lo[0], lo[1]);
-        mma_bf16(y[2u * np + 1u], ca, hi[2], hi[3]);
-        mma_bf16(y[2u * np + 1u], ca, lo[2], lo[3]);
-      }
+      const uint32_t at = (ks * 16u + kn_row) * L.x_row + y_first * 2u + kn_off;
+      ldmatrix_x4_trans(hi, smem_addr(state_hi) + at);
+      ldmatrix_x4_trans(lo, smem_addr(state_lo) + at);
+      mma_bf16(y[0], ca, hi[0], hi[1]);
+      mma_bf16(y[1], ca, hi[2], hi[3]);
+      mma_bf16(y[0], ca, lo[0], lo[1]);
+      mma_bf16(y[1], ca, lo[2], lo[3]);
     }
-    const uint32_t row[2] = {16u * warp + g, 16u * warp + g + 8u};
+    const uint32_t row[2] = {16u * token_tile + g, 16u * token_tile + g + 8u};
     const float here[2] = {log_decay[row[0]], log_decay[row[1]]};
-    const float from_start[2] = {expf(here[0]), expf(here[1])};
+    const float from_start[2] = {exp2f(here[0]), exp2f(here[1])};
 #pragma unroll
-    for (uint32_t n = 0; n < NT; ++n) {
+    for (uint32_t n = 0; n < YT; ++n) {
       y[n][0] *= from_start[0];
       y[n][1] *= from_start[0];
       y[n][2] *= from_start[1];
       y[n][3] *= from_start[1];
     }
     // what the chunk's own tokens give: 16 of them at a time, up to the diagonal
-    for (uint32_t kb = 0; kb <= warp; ++kb) {
+    for (uint32_t kb = 0; kb <= token_tile; ++kb) {
       float sc[2][4];
 #pragma unroll
       for (uint32_t n = 0; n < 2u; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.0f;
       const uint32_t b_addr = smem_addr(b_sh) + (16u * kb + nk_row) * L.n_row + nk_off;
+#pragma unroll 4
       for (uint32_t ks = 0; ks < n_pad / 16u; ++ks) {
         uint32_t ca[4], bb[4];
         ldmatrix_x4(ca, c_addr + ks * 32u);
@@ -541,22 +611,19 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
 #pragma unroll
         for (uint32_t j = 0; j < 4u; ++j) {
           const uint32_t from = 16u * kb + 8u * n + 2u * t4 + (j & 1u), i = j >> 1;
-          sc[n][j] = from <= row[i] ? sc[n][j] * expf(here[i] - log_decay[from]) * steps[from] : 0.0f;
+          sc[n][j] = from <= row[i] ? sc[n][j] * exp2f(here[i] - log_decay[from]) * steps[from] : 0.0f;
         }
       }
       const uint32_t hi[4] = {pack_bf16_hi(sc[0][0], sc[0][1]), pack_bf16_hi(sc[0][2], sc[0][3]),
                               pack_bf16_hi(sc[1][0], sc[1][1]), pack_bf16_hi(sc[1][2], sc[1][3])};
       const uint32_t lo[4] = {pack_bf16_lo(sc[0][0], sc[0][1]), pack_bf16_lo(sc[0][2], sc[0][3]),
                               pack_bf16_lo(sc[1][0], sc[1][1]), pack_bf16_lo(sc[1][2], sc[1][3])};
-#pragma unroll
-      for (uint32_t np = 0; np < NT / 2u; ++np) {
-        uint32_t xb[4];
-        ldmatrix_x4_trans(xb, smem_addr(x_sh) + (16u * kb + kn_row) * L.x_row + np * 32u + kn_off);
-        mma_bf16(y[2u * np], hi, xb[0], xb[1]);
-        mma_bf16(y[2u * np], lo, xb[0], xb[1]);
-        mma_bf16(y[2u * np + 1u], hi, xb[2], xb[3]);
-        mma_bf16(y[2u * np + 1u], lo, xb[2], xb[3]);
-      }
+      uint32_t xb[4];
+      ldmatrix_x4_trans(xb, smem_addr(x_sh) + (16u * kb + kn_row) * L.x_row + y_first * 2u + kn_off);
+      mma_bf16(y[0], hi, xb[0], xb[1]);
+      mma_bf16(y[1], hi, xb[2], xb[3]);
+      mma_bf16(y[0], lo, xb[0], xb[1]);
+      mma_bf16(y[1], lo, xb[2], xb[3]);
     }
 #pragma unroll
     for (uint32_t i = 0; i < 2u; ++i) {
@@ -564,19 +631,19 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
       if (r < p.row_count) {
         float *out = p.out + static_cast<uint64_t>(r) * p.out_stride + head * s.v_dim;
 #pragma unroll
-        for (uint32_t n = 0; n < NT; ++n) {
-          const uint32_t x = *reinterpret_cast<const uint32_t *>(x_sh + row[i] * L.x_row + (8u * n + 2u * t4) * 2u);
-          const uint32_t col = column0 + 8u * n + 2u * t4;
+        for (uint32_t n = 0; n < YT; ++n) {
+          const uint32_t x = *reinterpret_cast<const uint32_t *>(x_sh + row[i] * L.x_row + (y_first + 8u * n + 2u * t4) * 2u);
+          const uint32_t col = column0 + y_first + 8u * n + 2u * t4;
           if (col < s.v_dim) out[col] = fmaf(skip, bf16x2_lo(x), y[n][2u * i]) * silu(z[i][n][0]);
           if (col + 1u < s.v_dim) out[col + 1u] = fmaf(skip, bf16x2_hi(x), y[n][2u * i + 1u]) * silu(z[i][n][1]);
         }
       }
     }
     // the state at the chunk's end
-    const float whole = expf(log_decay[kChunk - 1u]);
+    const float whole = exp2f(log_decay[kChunk - 1u]);
 #pragma unroll
     for (uint32_t m = 0; m < MT; ++m) {
-      const uint32_t tile = warp + 4u * m;
+      const uint32_t tile = warp + kScanWarps * m;
       if (tile < m_tiles) {
 #pragma unroll
         for (uint32_t n = 0; n < NT; ++n) {
@@ -601,7 +668,7 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
         }
       }
     }
-    __syncthreads();  // steps, state and scaled x may be overwritten
+    __syncthreads();  // state and scaled x may be overwritten
   }
 #pragma unroll
   for (uint32_t m = 0; m < MT; ++m) {
@@ -609,7 +676,7 @@ __global__ void __launch_bounds__(kScanThreads) state_space_scan_kernel(StateSpa
     for (uint32_t n = 0; n < NT; ++n) {
 #pragma unroll
       for (uint32_t j = 0; j < 4u; ++j) {
-        const uint32_t row = 16u * (warp + 4u * m) + g + 8u * (j >> 1), col = 8u * n + 2u * t4 + (j & 1u);
+        const uint32_t row = 16u * (warp + kScanWarps * m) + g + 8u * (j >> 1), col = 8u * n + 2u * t4 + (j & 1u);
         if (row < s.state && column0 + col < s.v_dim) state[static_cast<uint64_t>(row) * s.v_dim + col] = held[m][n][j];
       }
     }
@@ -652,7 +719,7 @@ cudaError_t launch_block(cudaStream_t stream, const StateSpaceParams &p) {
                                     conv_grid, dim3(kConvThreads), 0, stream, p.pdl != 0, p);
   if (err != cudaSuccess) return err;
   if (sizeof(T) == 2u && p.row_count >= kScanMinRows)
-    return launch_with_pdl(s.state <= 128u ? state_space_scan_kernel<2> : state_space_scan_kernel<4>,
+    return launch_with_pdl(s.state <= 128u ? state_space_scan_kernel<1> : state_space_scan_kernel<2>,
                            dim3(column_tiles(s), s.heads), dim3(kScanThreads), ScanLayout(s).total, stream, p.pdl != 0, p);
   return launch_with_pdl(s.state <= 128u ? state_space_rows_kernel<T, 16> : state_space_rows_kernel<T, 32>,
                          dim3(column_tiles(s) * s.heads), dim3(kStepThreads), 0, stream, p.pdl != 0, p);
@@ -668,8 +735,8 @@ bool state_space_supported(const StateSpaceShape &s) {
 
 cudaError_t configure_state_space() {
   cudaError_t err = cudaSuccess;
-  for (const void *kernel : {reinterpret_cast<const void *>(state_space_scan_kernel<2>),
-                             reinterpret_cast<const void *>(state_space_scan_kernel<4>)})
+  for (const void *kernel : {reinterpret_cast<const void *>(state_space_scan_kernel<1>),
+                             reinterpret_cast<const void *>(state_space_scan_kernel<2>)})
     if (err == cudaSuccess) err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
   return err;
 }
@@ -677,13 +744,17 @@ cudaError_t configure_state_space() {
 cudaError_t launch_state_space_step(cudaStream_t stream, const StateSpaceParams &p) {
   if (!state_space_supported(p.s) || (p.rows != nullptr && (p.row_count == 0 || p.row_count > 65535u)))
     return cudaErrorInvalidValue;
-  return launch_with_pdl(p.s.state <= 128u ? state_space_step_kernel<16> : state_space_step_kernel<32>,
-                         dim3(column_tiles(p.s) * p.s.heads, p.rows != nullptr ? p.row_count : 1u), dim3(kStepThreads), 0,
-                         stream, p.pdl != 0, p);
+  void (*kernel)(StateSpaceParams);
+  if (p.s.v_dim % 4u == 0)
+    kernel = p.s.state <= 128u ? state_space_step_kernel<4, true> : state_space_step_kernel<8, true>;
+  else
+    kernel = p.s.state <= 128u ? state_space_step_kernel<4, false> : state_space_step_kernel<8, false>;
+  return launch_with_pdl(kernel, dim3(column_tiles(p.s) * p.s.heads, p.rows != nullptr ? p.row_count : 1u), dim3(kStepThreads), 0, stream,
+                         p.pdl != 0, p);
 }
 
 cudaError_t launch_state_space_block(cudaStream_t stream, const StateSpaceParams &p) {
-  if (!state_space_supported(p.s) || p.rows == nullptr || p.row_count == 0 || p.convolved == nullptr)
+  if (!state_space_supported(p.s) || p.rows == nullptr || p.row_count == 0 || p.row_count > kScanMaxRows || p.convolved == nullptr)
     return cudaErrorInvalidValue;
   return p.f32 != 0 ? launch_block<float>(stream, p) : launch_block<uint16_t>(stream, p);
 }

@@ -94,6 +94,12 @@ struct TileWalk {
   __device__ __forceinline__ uint32_t tile(uint32_t i) const { return i < kept ? i : first + (i - kept); }
 };
 
+// EXTRAS of the kernels below: kept first positions, score cap and output gates.  Without them the code
+// is the plain window's.
+__host__ __device__ inline bool has_extras(const WindowAttentionShape &s) {
+  return s.keep_first != 0 || s.softcap > 0.0f || s.head_gate != 0;
+}
+
 // Soft cap of a score that carries a factor log2(e).
 __device__ __forceinline__ float cap_score(float score, float cap2) { return cap2 * tanhf(score / cap2); }
 // The same through one exponential, absolute error a few 1e-7 of the cap.
@@ -103,9 +109,10 @@ __device__ __forceinline__ float cap_score_fast(float score, float cap2, float i
 }
 
 // Factor of a head's output.
+template <bool EXTRAS>
 __device__ __forceinline__ float output_gate(const WindowAttentionParams &p, uint32_t row, uint32_t h) {
   const WindowAttentionShape &s = p.s;
-  if (s.head_gate == 0) return 1.0f;
+  if (!EXTRAS || s.head_gate == 0) return 1.0f;
   const uint32_t at = (s.heads + s.kv_heads) * s.qk_dim + s.kv_heads * s.v_dim + h;
   return sigmoid(__ldcg(p.qkv + static_cast<uint64_t>(row) * p.qkv_stride + at));
 }
@@ -212,7 +219,7 @@ uint32_t chunk_tiles(const WindowAttentionShape &s) {
 // After every thread's partials of its block are stored: the block that draws the last ticket of its
 // heads merges their spans (one acquire-release atomic between the block's barriers orders the
 // partials).  Called by the whole block.
-template <class T, uint32_t PAIRS>
+template <class T, uint32_t PAIRS, bool EXTRAS>
 __device__ __forceinline__ void merge_spans(const WindowAttentionParams &p, uint32_t row, uint32_t head0, uint32_t hb,
                                             uint32_t *ticket) {
   const WindowAttentionShape &s = p.s;
@@ -270,7 +277,7 @@ __device__ __forceinline__ void merge_spans(const WindowAttentionParams &p, uint
       }
     }
     T *out = reinterpret_cast<T *>(p.out) + static_cast<uint64_t>(row) * p.out_stride + h * s.v_dim;
-    const float gate = output_gate(p, row, h);
+    const float gate = output_gate<EXTRAS>(p, row, h);
 #pragma unroll
     for (uint32_t i = 0; i < 2u * PAIRS; ++i) {
       const uint32_t d = 2u * lane + 64u * (i / 2u) + (i & 1u);
@@ -283,7 +290,7 @@ __device__ __forceinline__ void merge_spans(const WindowAttentionParams &p, uint
 // PAIRS: value pairs (2 lane + 64 j, +1) a lane accumulates; v_pad <= 64 PAIRS.
 // A warp has at most two work items: heads x tiles <= 2 kWarps.  Two stages of two 128-dim bf16 tiles take
 // 75 KB, which fits beside a weight-streaming block with two ring slots per warp on the same SM.
-template <class T, uint32_t PAIRS, bool ROWS>
+template <class T, uint32_t PAIRS, bool ROWS, bool EXTRAS>
 __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAttentionParams p, uint32_t tiles) {
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ uint32_t ticket;
@@ -336,7 +343,9 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
   // cached tokens [lo, hist) and those below keep_first are seen; the lone step's own token comes from the projection
   const uint32_t hist = ROWS ? position + 1u : position;
   const uint32_t lo = s.window != 0 && position + 1u > s.window ? position + 1u - s.window : 0u;
-  const TileWalk walk(s.keep_first, lo, chunk_tokens);
+  const uint32_t keep_first = EXTRAS ? s.keep_first : 0u;
+  const bool capped = EXTRAS && s.softcap > 0.0f;
+  const TileWalk walk(keep_first, lo, chunk_tokens);
   const uint32_t chunks = walk.count(hist, chunk_tokens);  // lo <= hist: never negative
   const uint32_t chunk_begin = chunks * span / S, chunk_end = chunks * (span + 1u) / S;  // numbers in the walk
   const bool owns_current = !ROWS && span + 1u == S;
@@ -353,7 +362,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
     const uint32_t pages = chunk_tokens / kPageTokens;
     uint32_t my_page = 0;
     const uint32_t page_token = first + lane * kPageTokens;
-    if (lane < pages && page_token < hist && (page_token + kPageTokens > lo || page_token / kTile * kTile < s.keep_first)) {
+    if (lane < pages && page_token < hist && (page_token + kPageTokens > lo || page_token / kTile * kTile < keep_first)) {
       my_page = table[first / kPageTokens + lane];
       if (my_page >= page_count) {
         report_error(error_word, kErrPageOutOfRange);
@@ -365,7 +374,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
       const uint32_t page = __shfl_sync(0xffffffffu, my_page, t / kPageTokens);
       const uint32_t token = first + t;
       // a tile with kept tokens is copied whole: its invisible rows meet probabilities of zero
-      if (token >= hist || (token < lo && token / kTile * kTile >= s.keep_first)) continue;
+      if (token >= hist || (token < lo && token / kTile * kTile >= keep_first)) continue;
       const T *k_src = keys + cache_row(page, token, s.kv_heads, kvh, s.qk_pad);
       const T *v_src = values + cache_row(page, token, s.kv_heads, kvh, s.v_pad);
       for (uint32_t c = lane; c < row_pieces; c += 32u) {
@@ -451,13 +460,13 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
         const uint32_t tile = item / hb, head = item - tile * hb;
         const uint32_t first = walk.tile(chunk) * chunk_tokens + tile * kTile;
         // the tile's visible tokens lie in [first + t0, first + t1)
-        const bool kept = first < s.keep_first;
+        const bool kept = first < keep_first;
         const uint32_t t0 = lo > first && !kept ? lo - first : 0u;
-        const uint32_t end = kept && lo >= first + kTile && s.keep_first < hist ? s.keep_first : hist;
+        const uint32_t end = kept && lo >= first + kTile && keep_first < hist ? keep_first : hist;
         const uint32_t t1 = end > first ? (end - first < kTile ? end - first : kTile) : 0u;
         if (t0 < t1) {
           float score = -INFINITY;
-          if (lane >= t0 && lane < t1 && (first + lane >= lo || first + lane < s.keep_first)) {
+          if (lane >= t0 && lane < t1 && (first + lane >= lo || first + lane < keep_first)) {
             const T *k_row = reinterpret_cast<const T *>(k_stage + (tile * kTile + lane) * layout.k_row);
             const float *q = q_sh + head * s.qk_pad;
             constexpr uint32_t kElems = 16u / sizeof(T);
@@ -467,7 +476,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
               part[1] = dot_piece(k_row + (c + 1u) * kElems, q + (c + 1u) * kElems, part[1]);
             }
             score = part[0] + part[1];
-            if (s.softcap > 0.0f) score = cap_score(score, cap2);
+            if (capped) score = cap_score(score, cap2);
           }
           const float m_new = fmaxf(m_run[u], warp_max(score));  // some token of the tile is visible: finite
           const float pr = exp2f(score - m_new);
@@ -539,7 +548,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
       float dot = 0.0f;
       for (uint32_t i = lane; i < s.qk_pad; i += 32u) dot = fmaf(q[i], k_new[i], dot);
       dot = warp_sum(dot);
-      if (s.softcap > 0.0f) dot = cap_score(dot, cap2);
+      if (capped) dot = cap_score(dot, cap2);
       float v[2u * PAIRS];
 #pragma unroll
       for (uint32_t j = 0; j < PAIRS; ++j) {
@@ -550,7 +559,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
       fold(dot, 1.0f, v);
     }
     if (S == 1u) {
-      const float inv = output_gate(p, row, h) / l;
+      const float inv = output_gate<EXTRAS>(p, row, h) / l;
 #pragma unroll
       for (uint32_t i = 0; i < 2u * PAIRS; ++i) {
         const uint32_t d = 2u * lane + 64u * (i / 2u) + (i & 1u);
@@ -571,7 +580,7 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WindowAtt
     }
   }
   if (S == 1u) return;
-  merge_spans<T, PAIRS>(p, row, head0, hb, &ticket);
+  merge_spans<T, PAIRS, EXTRAS>(p, row, head0, hb, &ticket);
 }
 
 // ------------------------------------------------------- block rows on the tensor pipe ----
@@ -594,7 +603,7 @@ struct RowLayout {
   }
 };
 
-template <uint32_t PAIRS>
+template <uint32_t PAIRS, bool EXTRAS>
 __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAttentionParams p) {
   constexpr uint32_t NT = 8u * PAIRS;  // value n-tiles of 8 dims: v_pad <= 64 PAIRS
   extern __shared__ __align__(128) uint8_t smem[];
@@ -619,11 +628,13 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
   const uint32_t hb = left_heads < kHeadsPerBlock ? left_heads : kHeadsPerBlock;
   const uint32_t hist = r.position + 1u;
   const uint32_t lo = s.window != 0 && hist > s.window ? hist - s.window : 0u;
-  const TileWalk walk(s.keep_first, lo, kPageTokens);
+  const uint32_t keep_first = EXTRAS ? s.keep_first : 0u;
+  const bool capped = EXTRAS && s.softcap > 0.0f;
+  const TileWalk walk(keep_first, lo, kPageTokens);
   const uint32_t pages = walk.count(hist, kPageTokens);
   const uint32_t page_begin = pages * span / S, page_end = pages * (span + 1u) / S;  // numbers in the walk
   const uint32_t first = page_begin + warp;
-  auto visible = [&](uint32_t token) { return token < hist && (token >= lo || token < s.keep_first); };
+  auto visible = [&](uint32_t token) { return token < hist && (token >= lo || token < keep_first); };
   const uint32_t my_pages = first < page_end ? (page_end - first + kRowWarps - 1u) / kRowWarps : 0u;
 
   uint8_t *ring = smem + warp * L.ring;
@@ -705,7 +716,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
 #pragma unroll
     for (uint32_t j = 0; j < 4u; ++j) {
       const uint32_t token = token0 + 8u * (j >> 1) + 2u * t4 + (j & 1u);
-      if (s.softcap > 0.0f) v[j] = cap_score_fast(v[j], cap2, inv_cap2);
+      if (capped) v[j] = cap_score_fast(v[j], cap2, inv_cap2);
       if (!visible(token)) v[j] = -INFINITY;
     }
     float m_page = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
@@ -774,7 +785,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
     if (S == 1u) {
       if (d < s.v_dim)
         reinterpret_cast<uint16_t *>(p.out)[static_cast<uint64_t>(row) * p.out_stride + (head0 + h) * s.v_dim + d] =
-            f32_to_bf16_bits(a / l * output_gate(p, row, head0 + h));
+            f32_to_bf16_bits(a / l * output_gate<EXTRAS>(p, row, head0 + h));
     } else {
       const uint64_t slot = (static_cast<uint64_t>(row) * s.heads + head0 + h) * S + span;
       p.partial_acc[slot * s.v_pad + d] = a;
@@ -784,7 +795,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) window_rows_kernel(WindowAtten
       }
     }
   }
-  if (S != 1u) merge_spans<uint16_t, PAIRS>(p, row, head0, hb, &ticket);
+  if (S != 1u) merge_spans<uint16_t, PAIRS, EXTRAS>(p, row, head0, hb, &ticket);
 }
 
 uint32_t rows_smem(const WindowAttentionShape &s) {
@@ -813,7 +824,7 @@ struct PrefillLayout {
 };
 
 // NT: value n-tiles of 8 dims held in registers (v_pad <= 8 NT).
-template <uint32_t NT, uint32_t GROUPS>
+template <uint32_t NT, uint32_t GROUPS, bool EXTRAS>
 __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kernel(WindowAttentionParams p) {
   extern __shared__ __align__(128) uint8_t smem[];
   const WindowAttentionShape &s = p.s;
@@ -840,7 +851,9 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
 
   const uint32_t kv_lo = s.window != 0 && pos_first + 1u > s.window ? pos_first + 1u - s.window : 0u;
   const uint32_t kv_end = pos_last + 1u;
-  const TileWalk walk(s.keep_first, kv_lo, kKeyTile);
+  const uint32_t keep_first = EXTRAS ? s.keep_first : 0u;
+  const bool capped = EXTRAS && s.softcap > 0.0f;
+  const TileWalk walk(keep_first, kv_lo, kKeyTile);
   const uint32_t tile_begin = key_group, tile_end = walk.count(kv_end, kKeyTile);  // numbers in the walk
   const uint32_t k_pieces = s.qk_pad / 8u, v_pieces = s.v_pad / 8u, row_pieces = k_pieces + v_pieces;
   auto issue = [&](uint32_t tile) {
@@ -939,7 +952,7 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
         mma_bf16(sc[2u * np + 1u], al, kb[2], kb[3]);
       }
     }
-    if (s.softcap > 0.0f) {
+    if (capped) {
 #pragma unroll
       for (uint32_t n = 0; n < 8u; ++n) {
 #pragma unroll
@@ -954,7 +967,7 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
       for (uint32_t j = 0; j < 4u; ++j) {
         const uint32_t token = first + n * 8u + 2u * t4 + (j & 1u);
         const uint32_t i = j >> 1;
-        if (!(token <= pos[i] && (pos[i] - token < window || token < s.keep_first))) sc[n][j] = -INFINITY;
+        if (!(token <= pos[i] && (pos[i] - token < window || token < keep_first))) sc[n][j] = -INFINITY;
         m_tile[i] = fmaxf(m_tile[i], sc[n][j]);
       }
     }
@@ -1054,7 +1067,7 @@ __global__ void __launch_bounds__(GROUPS * kPrefillThreads) window_prefill_kerne
     const uint32_t f = f0 + warp * 16u + g + 8u * i;
     uint16_t *dst = reinterpret_cast<uint16_t *>(p.out) + static_cast<uint64_t>(f / group) * p.out_stride +
                     (kvh * group + f % group) * s.v_dim;
-    const float inv = output_gate(p, f / group, kvh * group + f % group) / l_run[i];
+    const float inv = output_gate<EXTRAS>(p, f / group, kvh * group + f % group) / l_run[i];
 #pragma unroll
     for (uint32_t n = 0; n < NT; ++n) {
       const uint32_t d = n * 8u + 2u * t4;
@@ -1071,11 +1084,28 @@ uint32_t prefill_groups(const WindowAttentionShape &s) {
   return s.v_pad <= 128u && L.total <= kMaxSmem - 2048u && hand <= 4u * L.stage ? 2u : 1u;
 }
 
-template <class T, bool ROWS>
+template <class T, bool ROWS, bool EXTRAS>
 void (*decode_kernel(uint32_t v_pad))(WindowAttentionParams, uint32_t) {
-  if (v_pad <= 64u) return window_attention_kernel<T, 1, ROWS>;
-  if (v_pad <= 128u) return window_attention_kernel<T, 2, ROWS>;
-  return window_attention_kernel<T, 4, ROWS>;
+  if (v_pad <= 64u) return window_attention_kernel<T, 1, ROWS, EXTRAS>;
+  if (v_pad <= 128u) return window_attention_kernel<T, 2, ROWS, EXTRAS>;
+  return window_attention_kernel<T, 4, ROWS, EXTRAS>;
+}
+template <class T, bool ROWS>
+void (*decode_kernel(const WindowAttentionShape &s))(WindowAttentionParams, uint32_t) {
+  return has_extras(s) ? decode_kernel<T, ROWS, true>(s.v_pad) : decode_kernel<T, ROWS, false>(s.v_pad);
+}
+template <bool EXTRAS>
+void (*rows_kernel(uint32_t v_pad))(WindowAttentionParams) {
+  if (v_pad <= 64u) return window_rows_kernel<1, EXTRAS>;
+  if (v_pad <= 128u) return window_rows_kernel<2, EXTRAS>;
+  return window_rows_kernel<4, EXTRAS>;
+}
+template <bool EXTRAS>
+void (*prefill_kernel(uint32_t v_pad, uint32_t groups))(WindowAttentionParams) {
+  if (groups == 2u) return v_pad <= 64u ? window_prefill_kernel<8, 2, EXTRAS> : window_prefill_kernel<16, 2, EXTRAS>;
+  if (v_pad <= 64u) return window_prefill_kernel<8, 1, EXTRAS>;
+  if (v_pad <= 128u) return window_prefill_kernel<16, 1, EXTRAS>;
+  return window_prefill_kernel<32, 1, EXTRAS>;
 }
 
 // The hand-off of the items' states reuses the stages; both must fit.
@@ -1098,7 +1128,7 @@ cudaError_t launch_decode(cudaStream_t stream, const WindowAttentionParams &p) {
   const uint32_t subs = (group + kHeadsPerBlock - 1u) / kHeadsPerBlock;
   const bool rows = p.rows != nullptr;
   const dim3 grid(p.s.kv_heads * subs * p.splits, rows ? p.row_count : 1u);
-  return launch_with_pdl(rows && kHasRows ? decode_kernel<float, true>(p.s.v_pad) : decode_kernel<T, false>(p.s.v_pad), grid,
+  return launch_with_pdl(rows && kHasRows ? decode_kernel<float, true>(p.s) : decode_kernel<T, false>(p.s), grid,
                          dim3(kWarps * 32), bytes, stream, p.pdl != 0, p,
                          tiles);
 }
@@ -1148,18 +1178,19 @@ cudaError_t configure_window_attention() {
       err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kMaxSmem - 2048u));
   };
   for (uint32_t v : {64u, 128u, 256u}) {
-    set(reinterpret_cast<const void *>(decode_kernel<uint16_t, false>(v)));
-    set(reinterpret_cast<const void *>(decode_kernel<float, false>(v)));
-    set(reinterpret_cast<const void *>(decode_kernel<float, true>(v)));
+    set(reinterpret_cast<const void *>(decode_kernel<uint16_t, false, false>(v)));
+    set(reinterpret_cast<const void *>(decode_kernel<uint16_t, false, true>(v)));
+    set(reinterpret_cast<const void *>(decode_kernel<float, false, false>(v)));
+    set(reinterpret_cast<const void *>(decode_kernel<float, false, true>(v)));
+    set(reinterpret_cast<const void *>(decode_kernel<float, true, false>(v)));
+    set(reinterpret_cast<const void *>(decode_kernel<float, true, true>(v)));
+    set(reinterpret_cast<const void *>(rows_kernel<false>(v)));
+    set(reinterpret_cast<const void *>(rows_kernel<true>(v)));
+    for (uint32_t groups : {1u, 2u}) {
+      set(reinterpret_cast<const void *>(prefill_kernel<false>(v, groups)));
+      set(reinterpret_cast<const void *>(prefill_kernel<true>(v, groups)));
+    }
   }
-  set(reinterpret_cast<const void *>(window_rows_kernel<1>));
-  set(reinterpret_cast<const void *>(window_rows_kernel<2>));
-  set(reinterpret_cast<const void *>(window_rows_kernel<4>));
-  set(reinterpret_cast<const void *>(window_prefill_kernel<8, 1>));
-  set(reinterpret_cast<const void *>(window_prefill_kernel<16, 1>));
-  set(reinterpret_cast<const void *>(window_prefill_kernel<32, 1>));
-  set(reinterpret_cast<const void *>(window_prefill_kernel<8, 2>));
-  set(reinterpret_cast<const void *>(window_prefill_kernel<16, 2>));
   return err;
 }
 
@@ -1176,9 +1207,7 @@ cudaError_t launch_window_attention(cudaStream_t stream, const WindowAttentionPa
     return cudaErrorInvalidValue;
   if (p.rows != nullptr && p.f32 == 0) {
     const uint32_t subs = (p.s.heads / p.s.kv_heads + kHeadsPerBlock - 1u) / kHeadsPerBlock;
-    void (*kernel)(WindowAttentionParams) = p.s.v_pad <= 64u    ? window_rows_kernel<1>
-                                            : p.s.v_pad <= 128u ? window_rows_kernel<2>
-                                                                : window_rows_kernel<4>;
+    void (*kernel)(WindowAttentionParams) = has_extras(p.s) ? rows_kernel<true>(p.s.v_pad) : rows_kernel<false>(p.s.v_pad);
     return launch_with_pdl(kernel, dim3(p.s.kv_heads * subs * p.splits, p.row_count), dim3(kRowWarps * 32),
                            rows_smem(p.s), stream, p.pdl != 0, p);
   }
@@ -1191,11 +1220,8 @@ cudaError_t launch_window_prefill(cudaStream_t stream, const WindowAttentionPara
   const dim3 grid((rows + kTileRows - 1u) / kTileRows, p.s.kv_heads);
   const uint32_t groups = prefill_groups(p.s);
   const uint32_t bytes = PrefillLayout(p.s, groups).total;
-  void (*kernel)(WindowAttentionParams);
-  if (groups == 2u)
-    kernel = p.s.v_pad <= 64u ? window_prefill_kernel<8, 2> : window_prefill_kernel<16, 2>;
-  else
-    kernel = p.s.v_pad <= 64u ? window_prefill_kernel<8, 1> : (p.s.v_pad <= 128u ? window_prefill_kernel<16, 1> : window_prefill_kernel<32, 1>);
+  void (*kernel)(WindowAttentionParams) =
+      has_extras(p.s) ? prefill_kernel<true>(p.s.v_pad, groups) : prefill_kernel<false>(p.s.v_pad, groups);
   return launch_with_pdl(kernel, grid, dim3(groups * kPrefillThreads), bytes, stream, p.pdl != 0, p);
 }
 
