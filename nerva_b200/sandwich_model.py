@@ -167,7 +167,7 @@ class SandwichConfig:
                 raise ValueError(f"layer {i}: unknown mixer type {entry['type']!r}")
         loop = config.get("loop") or {"start": 0, "stop": 0, "times": 0}
         return cls(name=name, hidden=config["width"], vocab=config["vocab"], rms_eps=config["norm"]["eps"],
-                   layer_specs=tuple(specs), logit_scale=config.get("logit_scale", 1.0), loop_start=loop["start"],
+                   layer_specs=tuple(specs), logit_scale=config.get("logit_scale") or 1.0, loop_start=loop["start"],
                    loop_stop=loop["stop"], loop_times=loop["times"])
 
 
