@@ -985,7 +985,7 @@ int nerva_b200_session_append(NervaCudaHfDecodeSequenceSession *session, const u
 
 /* The residual stream after each layer run of the next appended blocks (a diagnostic): `stream`
  * is host memory of [layer runs][capacity_rows][hidden] floats, filled for the rows of the append
- * calls that follow until it is set to NULL.  Parallel-block sessions only. */
+ * calls that follow until it is set to NULL.  Sessions of nerva_b200_session_create_parallel only. */
 int nerva_b200_session_capture_stream(NervaCudaHfDecodeSequenceSession *session, float *stream,
                                       uint32_t capacity_rows);
 

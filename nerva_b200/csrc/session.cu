@@ -1513,7 +1513,7 @@ cudaError_t allocate_state(Session *s, int32_t *stage) {
   // KV pages come out of the pool in FIFO order, which makes the initial
   // logical->physical table the identity, as the reference initialises it
   // (hf_decode_sequence/kernels.cu:732-739).
-  // A page of a parallel-block session is 16 tokens of every layer run, K and V together.
+  // A page of a session with a layer-by-layer plan is 16 tokens of every layer run, K and V together.
   const uint64_t page_bytes = s->parallel ? std::max<uint64_t>((s->parallel->key_elems + s->parallel->value_elems) /
                                                                    s->kv_pages * s->parallel->element_bytes(),
                                                                16u)

@@ -48,9 +48,9 @@ struct LayerLayout {
   // (expert_up_offset = moe_intermediate * hidden inside a stride of twice that); DeepSeek layers
   // hold all gate matrices, then all up matrices (weights_pack.inc.cu:303-312).
   uint64_t expert_stride = 0, expert_up_offset = 0;
-  // parallel-block layers (rms_attn is the layer's one norm): per-channel scales of the two sublayers
+  // parallel blocks (rms_attn is the layer's one norm): per-channel scales of the two sublayers
   uint64_t ls_attn = kMissingOffset, ls_mlp = kMissingOffset;
-  // sandwich layers: the norms behind the sublayers (rms_attn, rms_mlp are those in front); attention's output
+  // sandwich blocks: the norms behind the sublayers (rms_attn, rms_mlp are those in front); attention's output
   // gate; a state space's input projection (w_o is its output) and small tensors
   uint64_t norm_after = kMissingOffset, norm_mlp_after = kMissingOffset, w_head_gate = kMissingOffset;
   uint64_t w_space = kMissingOffset, conv = kMissingOffset, conv_bias = kMissingOffset, step_bias = kMissingOffset;
@@ -272,7 +272,7 @@ struct WantedLogits {
 // norm, lm_head and the sampler for the last position.  Leaves the cursor at prompt_count.
 cudaError_t enqueue_chunked_prefill(NervaCudaHfDecodeSequenceSession *s, uint32_t begin, uint32_t prompt_count,
                                     const WantedLogits &wanted, uint64_t *launches);
-// The layer runs of a parallel-block model over the block's rows (ws.h_b in and out) and the head of
+// The layer runs of a decoder described layer by layer over the block's rows (ws.h_b in and out) and the head of
 // `count` rows (row_index: device array of block rows, null: the first `count`) into ws.logits.
 struct ParallelBlock {
   cudaStream_t stream;
@@ -320,7 +320,7 @@ struct NervaCudaHfDecodeSequenceSession {
   uint64_t planned_weight_descriptor_hash = 0;
 
   std::shared_ptr<nb::SharedWeights> weights;
-  std::shared_ptr<nb::ParallelPlan> parallel;  // parallel-block models only
+  std::shared_ptr<nb::ParallelPlan> parallel;  // decoders described layer by layer only
   float *capture_stream = nullptr;             // host buffer of nerva_b200_session_capture_stream
   uint32_t capture_rows = 0;
   nb::StaticArena weight_arena, state_arena;

@@ -115,6 +115,8 @@ class ParallelConfig:
             shapes[p + "mix.q"] = (s.heads * s.qk_dim, self.hidden)
             shapes[p + "mix.k"] = (s.kv_heads * s.qk_dim, self.hidden)
             shapes[p + "mix.v"] = (s.kv_heads * s.v_dim, self.hidden)
+            if s.head_gate:
+                shapes[p + "mix.g"] = (s.heads, self.hidden)
             shapes[p + "mix.o"] = (self.hidden, s.heads * s.v_dim)
             if s.intermediate:
                 shapes[p + "mlp.gate"] = (s.intermediate, self.hidden)

@@ -3,7 +3,7 @@
 A loader gets (folder, parsed config.json) and returns a checkpoint object that
 nerva_b200.session.CudaHfDecodeSequenceSession takes: `.config` with the create request's scalars,
 and either the dense tensors of nerva_b200.synth.DenseCheckpoint or `upload_order()` and
-`native_model(compute)` (nerva_b200.parallel_model).
+`native_model(compute)` (nerva_b200.parallel_model, nerva_b200.sandwich_model).
 """
 from __future__ import annotations
 

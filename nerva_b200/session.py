@@ -186,7 +186,7 @@ class CudaHfDecodeSequenceSession:
         """library: a handle from ffi.load_abi_library for another implementation of the same C ABI
         (default: this package's libnerva_b200.so).  weight_file: upload through descriptors that
         name byte ranges of this file (see write_weight_file) instead of host pointers.
-        compute: "bfloat16", or "float32" for models that also run in true fp32 (parallel_model)."""
+        compute: "bfloat16", or "float32" for models that also run in true fp32 (parallel_model, sandwich_model)."""
         cfg = checkpoint.config
         self._lib = library if library is not None else ffi.lib()
         self._own_library = library is None
@@ -316,7 +316,7 @@ class CudaHfDecodeSequenceSession:
 
     def append_with_stream(self, tokens, reset: bool = False) -> np.ndarray:
         """append of at least two tokens; returns the residual stream after every layer run, [runs, tokens, hidden]
-        (parallel-block models)."""
+        (models described layer by layer: parallel_model, sandwich_model)."""
         stream = np.zeros((self.config.layer_runs, len(tokens), self.config.hidden), dtype=np.float32)
         if ffi.lib().nerva_b200_session_capture_stream(self._handle, _ptr(stream), len(tokens)) != 0:
             raise RuntimeError("no stream capture for this model")

@@ -2,6 +2,7 @@
 together, in fp32 and in bf16; prompts, portions, token-by-token decoding, packed batches; page, state and
 session re-use; window and kept-position edges with a key that stands out; a state that has to last; sizes
 of all kinds; generation and replay through the entry points a user calls."""
+import dataclasses
 import json
 import os
 import subprocess
@@ -10,10 +11,12 @@ import sys
 import numpy as np
 import pytest
 
-from nerva_b200 import generate, registry, synth
+from nerva_b200 import generate, parallel_model, registry, sandwich_model, synth
 from nerva_b200.session import CudaHfDecodeSequenceLoop, CudaHfDecodeSequenceSession, SmokeStatus, sampler_config
 from tests import vamidra_models as M
 from tests import vamidra_oracle as O
+from tests import vuvolix_models as V
+from tests import vuvolix_oracle as VO
 from tests.conftest import ROOT
 
 pytestmark = pytest.mark.gpu
@@ -102,6 +105,77 @@ def test_mechanism(built_lib, name, dtype):
     assert M.distance(s.append(tokens, range(45), reset=True), want) < M.TOLERANCE[dtype]
     assert M.distance(run_portions(s, tokens, [1]), want) < M.TOLERANCE[dtype]
     assert M.distance(run_portions(s, tokens, [2, 5, 3, 9, 17, 2]), want) < M.TOLERANCE[dtype]
+
+
+@dataclasses.dataclass(frozen=True)
+class PlainSandwich(sandwich_model.SandwichConfig):
+    """Sandwich blocks with RMS norms, silu and passes that begin with their vector alone."""
+
+    def tensor_shapes(self):
+        return {k: v for k, v in super().tensor_shapes().items() if k != "loop.in"}
+
+    def native_model(self, compute):
+        return parallel_model.native_model(self, compute, embedding_scale=2.0, logit_softcap=3.0, block=sandwich_model.BLOCK_SANDWICH)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_sandwich_blocks_of_another_design(built_lib, monkeypatch, dtype):
+    """The other norm, activation and loop entry, rotated and normalised q and k, a scaled embedding, capped logits."""
+    cfg = M.config([M.attention(kv_heads=4), M.space(), M.attention(window=9)], loop=(1, 3, 2))
+    w = M.weights(cfg)
+    parsed = sandwich_model.SandwichConfig.from_json(cfg)
+    specs = tuple(dataclasses.replace(s, rotary_dims=16, qk_norm=True) if isinstance(s, parallel_model.ParallelLayer) else s
+                  for s in parsed.layer_specs)
+    plain = PlainSandwich(**{**{f.name: getattr(parsed, f.name) for f in dataclasses.fields(parsed)}, "layer_specs": specs})
+    s = CudaHfDecodeSequenceSession(parallel_model.ParallelCheckpoint(
+        plain, {k: synth.f32_to_bf16(v).reshape(v.shape) for k, v in w.items()}), 64, compute=dtype)
+    assert s.status == SmokeStatus.OK, s.error
+
+    capped = O.capped_attention
+
+    def rotated(q, k, v, scale, cap, mask):
+        at = np.arange(len(q))
+        freq, magnitude = VO.rotary_frequencies(16, 10000.0)
+        return capped(*(VO.rms_norm(VO.rotate(t, at, freq, magnitude), cfg["norm"]["eps"]) for t in (q, k)), v, scale, cap, mask)
+
+    monkeypatch.setattr(O, "capped_attention", rotated)
+    monkeypatch.setattr(O, "layer_norm", lambda x, eps, weight: VO.rms_norm(x, eps, weight))
+    monkeypatch.setattr(O, "gelu_tanh", O.silu)
+    monkeypatch.setattr(O, "begin_pass", lambda x, first, weights, number: (x + weights["loop.step"][number]).astype(np.float32))
+    tokens = M.tokens(cfg, 50)
+    want = VO.soft_cap(O.forward({**cfg, "logit_scale": 1.0}, {**w, "embed": 2.0 * w["embed"]}, tokens), 3.0)
+    assert M.distance(s.append(tokens, range(50), reset=True), want) < M.TOLERANCE[dtype]
+    assert M.distance(run_portions(s, tokens, [1, 1, 20, 3, 1]), want) < M.TOLERANCE[dtype]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_parallel_blocks_with_kept_positions_cap_and_gates(built_lib, monkeypatch, dtype):
+    cfg = V.config([V.layer(window=9), V.layer(heads=6, kv_heads=3, window=20, ff=0)])
+    parsed = parallel_model.ParallelConfig.from_json(cfg)
+    parsed = dataclasses.replace(parsed, layer_specs=tuple(
+        dataclasses.replace(s, keep_first=4, score_softcap=1.5, head_gate=True) for s in parsed.layer_specs))
+    w = V.weights(cfg)
+    rng = np.random.default_rng(3)
+    for i, heads in enumerate((4, 6)):
+        w[f"l{i}.mix.g"] = M.round_bf16(rng.standard_normal((heads, cfg["width"])) * 0.2)
+    s = CudaHfDecodeSequenceSession(parallel_model.ParallelCheckpoint(
+        parsed, {k: synth.f32_to_bf16(v).reshape(v.shape) for k, v in w.items()}), 64, compute=dtype)
+    assert s.status == SmokeStatus.OK, s.error
+
+    def attention_mixer(h, m, get, eps, positions):
+        tokens, heads, groups = len(h), m["heads"], m["kv_heads"]
+        freq, magnitude = VO.rotary_frequencies(m["rot"]["dims"], m["rot"]["base"])
+        q, k = (VO.rms_norm(VO.rotate(VO.linear(get(n), h).reshape(tokens, c, m["dim"]), positions, freq, magnitude), eps)
+                for n, c in (("q", heads), ("k", groups)))
+        v = VO.linear(get("v"), h).reshape(tokens, groups, m["vdim"])
+        a = O.capped_attention(q, k, v, m["scale"], 1.5, O.visible(positions, positions, m["mask"]["size"], 4))
+        return VO.linear(get("o"), O.head_gate(a, get("g"), h).reshape(tokens, heads * m["vdim"]))
+
+    monkeypatch.setattr(VO, "attention_mixer", attention_mixer)
+    tokens = M.tokens(cfg, 50)
+    want = VO.forward(cfg, w, tokens)
+    assert M.distance(s.append(tokens, range(50), reset=True), want) < M.TOLERANCE[dtype]
+    assert M.distance(run_portions(s, tokens, [1, 1, 20, 3, 1]), want) < M.TOLERANCE[dtype]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
